@@ -127,7 +127,7 @@ def build_library(name: str, sources, defines: dict | None = None, extra_flags=(
         name = name + "_trc"
     nvcc = _nvcc()
     tmp = path.with_suffix(f".tmp{os.getpid()}.so")
-    cmd = [nvcc] + flags + ["-I", str(CSRC), "-o", str(tmp)] + [str(CSRC / s) for s in sources]
+    cmd = [nvcc, "-t", "0"] + flags + ["-I", str(CSRC), "-o", str(tmp)] + [str(CSRC / s) for s in sources]
     if verbose:
         print(f"[tensorline_b200] compiling {name} ({', '.join(sources)}) for sm_100a ...", file=sys.stderr, flush=True)
     t0 = time.time()

@@ -3,13 +3,16 @@
 //   S_t = a_t S_{t-1} + b_t k_t v_t^T        S: [d, dv] per (request, head), float, kept in the request's state slot
 //   o_t = S_t^T q_t
 //
-// Two kinds of (a_t, b_t), one kernel:
+// Three kinds of (a_t, b_t), one kernel:
 //   fixed decay    a_t = decay[h], b_t = 1                                   (retention: no normaliser)
 //   gated          log gates i_t = cap tanh(x_i / cap), f_t = logsigmoid(cap tanh(x_f / cap)) from the
 //                  pre-activations x_i, x_f; running maximum m_t = max(f_t + m_{t-1}, i_t), m_0 = 0;
 //                  a_t = exp(f_t + m_{t-1} - m_t), b_t = exp(i_t - m_t); a normaliser n_t = a_t n_{t-1} + b_t k_t
 //                  rides along as one more column of S (v = 1), and
 //                  o_t = S_t^T q_t / (max(|n_t . q_t|, exp(-m_t)) + den_eps)   (the matrix memory of the xLSTM)
+//   channel gates  a_t is a vector over the d rows: f_t = lower + (1 - lower) sigmoid(x_f + bias) from pre-activations x_f [H, d]
+//                  of the projection, b_t k_t = 1 - f_t (the gate decides what is written, there is no key), and q_t = silu(x_q)
+//                  (HGRN2: Qin et al., "HGRN2: Gated Linear RNNs with State Expansion").  No rotation.
 // q and k may be rotated by position first (either pairing of dimensions, the first `rot` of a head) and scaled.
 // Everything is float: angles, gates, exponentials, the state and the sums; only q, k, v come in the
 // activation type, as the projection left them.
@@ -41,10 +44,15 @@ struct ScanArgs {
     float* out;                            // [T, H * dv]
     int H, d, dv;
     float den_eps;
+    const float* lower; const float* bias;  // channel gates: [H, d] each; k_off is then where x_f lies
 };
 
+// KIND of the templates below
+constexpr int SCAN_FIXED = 0, SCAN_GATED = 1, SCAN_CHANNEL = 2;
+
 // A head's d rows are dealt out to IS threads a column, R consecutive rows each (R * IS >= d; the rows beyond d are zeros).
-template <int R, int IS, bool GATED> struct ScanShape {
+template <int R, int IS, int KIND> struct ScanShape {
+    static constexpr bool GATED = KIND == SCAN_GATED;
     static constexpr int JW = SCAN_JS + (GATED ? 1 : 0);
     static constexpr int NT = (IS * JW + 31) / 32 * 32;
     static constexpr int PB = R * NT + (GATED ? 4 : 0);          // floats of state a (head, column slice)
@@ -52,11 +60,14 @@ template <int R, int IS, bool GATED> struct ScanShape {
     static constexpr int TS = IS * RS;                           // 16-byte reads of the IS threads of a column hit different banks
 };
 
+__device__ __forceinline__ float scan_sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
+__device__ __forceinline__ float channel_gate(float x, float bias, float lower) { return fmaf(1.0f - lower, scan_sigmoid(x + bias), lower); }
 __device__ __forceinline__ float log_sigmoid(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
 
-template <typename TA, int R, int IS, bool GATED>
-__global__ void __launch_bounds__(ScanShape<R, IS, GATED>::NT) linear_scan_kernel(const ScanArgs A) {
-    using Sh = ScanShape<R, IS, GATED>;
+template <typename TA, int R, int IS, int KIND>
+__global__ void __launch_bounds__(ScanShape<R, IS, KIND>::NT) linear_scan_kernel(const ScanArgs A) {
+    using Sh = ScanShape<R, IS, KIND>;
+    constexpr bool GATED = KIND == SCAN_GATED, CHANNEL = KIND == SCAN_CHANNEL;
     constexpr int NT = Sh::NT, PB = Sh::PB, RS = Sh::RS, TS = Sh::TS;
     constexpr int PF = (SCAN_C * R * IS + NT - 1) / NT;           // q (and k) elements of a chunk a thread fetches
     constexpr int PV = (SCAN_C * SCAN_JS + NT - 1) / NT;          // v elements
@@ -80,7 +91,7 @@ __global__ void __launch_bounds__(ScanShape<R, IS, GATED>::NT) linear_scan_kerne
     const int jcol = z * SCAN_JS + j;
     const bool ones = GATED && j == SCAN_JS;
     const bool live = j < SCAN_JS && jcol < A.dv;
-    const float dec = GATED ? 0.f : A.decay[h];
+    const float dec = KIND == SCAN_FIXED ? A.decay[h] : 0.f;
     const TA* proj = (const TA*)A.proj;
     const int rhalf = A.rot >> 1;
     // rows beyond d and the padding stay zero; a step of single tokens uses (and clears) the first token's part only
@@ -92,9 +103,11 @@ __global__ void __launch_bounds__(ScanShape<R, IS, GATED>::NT) linear_scan_kerne
     int g_off[PF], s_off[PF], v_goff[PV];
     unsigned in_rot = 0, v_ok = 0;                         // bit it: the element is rotated / the v element exists
     int tok_of[PF];
+    float lo[CHANNEL ? PF : 1], bi[CHANNEL ? PF : 1];      // channel gates: lower bound and bias of each element
 #pragma unroll
     for (int it = 0; it < PF; ++it) {
         const int idx = tid + it * NT, t = idx / d, e = idx - t * d;
+        if (CHANNEL) { lo[it] = A.lower[h * d + e]; bi[it] = A.bias[h * d + e]; }
         tok_of[it] = t < SCAN_C ? t : SCAN_C;              // SCAN_C: beyond every chunk
         g_off[it] = t * A.stride + h * d + e;
         s_off[it] = t * TS + (e / R) * RS + (e % R);
@@ -140,6 +153,12 @@ __global__ void __launch_bounds__(ScanShape<R, IS, GATED>::NT) linear_scan_kerne
 #pragma unroll
         for (int it = 0; it < PF; ++it) {
             if (tok_of[it] < n) {
+                if (CHANNEL) {
+                    const float x = to_f<TA>(fq[it]);
+                    qs[s_off[it]] = x * scan_sigmoid(x);
+                    ks[s_off[it]] = channel_gate(to_f<TA>(fk[it]), bi[it], lo[it]);
+                    continue;
+                }
                 const bool rt = (in_rot >> it) & 1u;
                 qs[s_off[it]] = rt ? to_f<TA>(fq[it]) : to_f<TA>(fq[it]) * A.q_scale;
                 ks[s_off[it]] = rt ? to_f<TA>(fk[it]) : to_f<TA>(fk[it]) * A.k_scale;
@@ -201,6 +220,13 @@ __global__ void __launch_bounds__(ScanShape<R, IS, GATED>::NT) linear_scan_kerne
                 for (int r = 0; r < R; r += 4) {
                     const float4 kk = *reinterpret_cast<const float4*>(kt + t * TS + r);
                     const float4 qq = *reinterpret_cast<const float4*>(qt + t * TS + r);
+                    if (CHANNEL) {                       // f S + (1 - f) v as v + f (S - v)
+                        S[r] = fmaf(kk.x, S[r] - v, v);         acc = fmaf(S[r], qq.x, acc);
+                        S[r + 1] = fmaf(kk.y, S[r + 1] - v, v); acc = fmaf(S[r + 1], qq.y, acc);
+                        S[r + 2] = fmaf(kk.z, S[r + 2] - v, v); acc = fmaf(S[r + 2], qq.z, acc);
+                        S[r + 3] = fmaf(kk.w, S[r + 3] - v, v); acc = fmaf(S[r + 3], qq.w, acc);
+                        continue;
+                    }
                     S[r] = fmaf(a, S[r], kk.x * bv);         acc = fmaf(S[r], qq.x, acc);
                     S[r + 1] = fmaf(a, S[r + 1], kk.y * bv); acc = fmaf(S[r + 1], qq.y, acc);
                     S[r + 2] = fmaf(a, S[r + 2], kk.z * bv); acc = fmaf(S[r + 2], qq.z, acc);
@@ -243,9 +269,10 @@ __global__ void __launch_bounds__(ScanShape<R, IS, GATED>::NT) linear_scan_kerne
 // kernel's own arithmetic, so a token decoded alone gets the bits it gets inside a portion), works the token in and
 // stores the state.  Few registers: several blocks share an SM and the loads and stores of the state, which are all
 // the step moves, overlap.
-template <typename TA, int R, int IS, bool GATED>
-__global__ void __launch_bounds__(ScanShape<R, IS, GATED>::NT) linear_step_kernel(const ScanArgs A) {
-    using Sh = ScanShape<R, IS, GATED>;
+template <typename TA, int R, int IS, int KIND>
+__global__ void __launch_bounds__(ScanShape<R, IS, KIND>::NT) linear_step_kernel(const ScanArgs A) {
+    using Sh = ScanShape<R, IS, KIND>;
+    constexpr bool GATED = KIND == SCAN_GATED, CHANNEL = KIND == SCAN_CHANNEL;
     constexpr int NT = Sh::NT, PB = Sh::PB, RS = Sh::RS, TS = Sh::TS;
     __shared__ __align__(16) float qs[TS];
     __shared__ __align__(16) float ks[TS];
@@ -271,7 +298,8 @@ __global__ void __launch_bounds__(ScanShape<R, IS, GATED>::NT) linear_step_kerne
         float qv = 0.f, kv = 0.f;
         if (e < d) {
             qv = to_f<TA>(row[A.q_off + (size_t)h * d + e]); kv = to_f<TA>(row[A.k_off + (size_t)h * d + e]);
-            if (e >= A.rot) { qv *= A.q_scale; kv *= A.k_scale; }
+            if (CHANNEL) { qv *= scan_sigmoid(qv); kv = channel_gate(kv, A.bias[h * d + e], A.lower[h * d + e]); }
+            else if (e >= A.rot) { qv *= A.q_scale; kv *= A.k_scale; }
         }
         qs[(e / R) * RS + (e % R)] = qv; ks[(e / R) * RS + (e % R)] = kv;
     }
@@ -298,7 +326,7 @@ __global__ void __launch_bounds__(ScanShape<R, IS, GATED>::NT) linear_step_kerne
         }
         __syncthreads();
     }
-    const float a = GATED ? sc[0] : A.decay[h];
+    const float a = GATED ? sc[0] : CHANNEL ? 0.f : A.decay[h];
     const float v = ones ? 1.f : vraw;
     const float bv = GATED ? sc[1] * v : v;
     float acc = 0.f;
@@ -306,6 +334,13 @@ __global__ void __launch_bounds__(ScanShape<R, IS, GATED>::NT) linear_step_kerne
     for (int r = 0; r < R; r += 4) {
         const float4 kk = *reinterpret_cast<const float4*>(ks + islice * RS + r);
         const float4 qq = *reinterpret_cast<const float4*>(qs + islice * RS + r);
+        if (CHANNEL) {
+            S[r] = fmaf(kk.x, S[r] - v, v);         acc = fmaf(S[r], qq.x, acc);
+            S[r + 1] = fmaf(kk.y, S[r + 1] - v, v); acc = fmaf(S[r + 1], qq.y, acc);
+            S[r + 2] = fmaf(kk.z, S[r + 2] - v, v); acc = fmaf(S[r + 2], qq.z, acc);
+            S[r + 3] = fmaf(kk.w, S[r + 3] - v, v); acc = fmaf(S[r + 3], qq.w, acc);
+            continue;
+        }
         S[r] = fmaf(a, S[r], kk.x * bv);         acc = fmaf(S[r], qq.x, acc);
         S[r + 1] = fmaf(a, S[r + 1], kk.y * bv); acc = fmaf(S[r + 1], qq.y, acc);
         S[r + 2] = fmaf(a, S[r + 2], kk.z * bv); acc = fmaf(S[r + 2], qq.z, acc);
@@ -330,21 +365,21 @@ static int scan_shape(int d) { return d <= 32 ? 0 : d <= 64 ? 1 : d <= 128 ? 2 :
 // Floats of state per (head, column slice) for a head of d rows; 0: d is too large.
 TL_EXPORT int tl_scan_state_floats(int d, int gated) {
     switch (scan_shape(d)) {
-        case 0: return gated ? ScanShape<4, 8, true>::PB : ScanShape<4, 8, false>::PB;
-        case 1: return gated ? ScanShape<8, 8, true>::PB : ScanShape<8, 8, false>::PB;
-        case 2: return gated ? ScanShape<8, 16, true>::PB : ScanShape<8, 16, false>::PB;
-        case 3: return gated ? ScanShape<8, 32, true>::PB : ScanShape<8, 32, false>::PB;
+        case 0: return gated ? ScanShape<4, 8, SCAN_GATED>::PB : ScanShape<4, 8, SCAN_FIXED>::PB;
+        case 1: return gated ? ScanShape<8, 8, SCAN_GATED>::PB : ScanShape<8, 8, SCAN_FIXED>::PB;
+        case 2: return gated ? ScanShape<8, 16, SCAN_GATED>::PB : ScanShape<8, 16, SCAN_FIXED>::PB;
+        case 3: return gated ? ScanShape<8, 32, SCAN_GATED>::PB : ScanShape<8, 32, SCAN_FIXED>::PB;
     }
     return 0;
 }
 TL_EXPORT int tl_scan_columns() { return SCAN_JS; }
 
-template <typename TA, int R, int IS, bool GATED>
+template <typename TA, int R, int IS, int KIND>
 static int launch_scan_shape(const ScanArgs& A, int B, bool single, cudaStream_t stream) {
-    using Sh = ScanShape<R, IS, GATED>;
+    using Sh = ScanShape<R, IS, KIND>;
     const int nz = (A.dv + SCAN_JS - 1) / SCAN_JS;
     if (single) {
-        return launch_after_wait(linear_step_kernel<TA, R, IS, GATED>, dim3(B, A.H, nz), dim3(Sh::NT), 0, stream, A);
+        return launch_after_wait(linear_step_kernel<TA, R, IS, KIND>, dim3(B, A.H, nz), dim3(Sh::NT), 0, stream, A);
     }
     const size_t smem = (size_t)(2 * SCAN_C * Sh::TS + SCAN_C * SCAN_JS + 4 * SCAN_C + A.rot / 2) * sizeof(float);
     if (smem > 48 * 1024) {                              // the widest heads: more dynamic shared memory than a kernel has by default
@@ -352,22 +387,22 @@ static int launch_scan_shape(const ScanArgs& A, int B, bool single, cudaStream_t
         const int dev = tl_device_index();
         if (dev < 0) return 1;
         if (!raised[dev]) {
-            const cudaError_t e = cudaFuncSetAttribute(linear_scan_kernel<TA, R, IS, GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+            const cudaError_t e = cudaFuncSetAttribute(linear_scan_kernel<TA, R, IS, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
             if (e != cudaSuccess) return (int)e;
             raised[dev] = true;
         }
     }
-    linear_scan_kernel<TA, R, IS, GATED><<<dim3(B, A.H, nz), Sh::NT, smem, stream>>>(A);
+    linear_scan_kernel<TA, R, IS, KIND><<<dim3(B, A.H, nz), Sh::NT, smem, stream>>>(A);
     return tl_launch_status();
 }
 
-template <typename TA, bool GATED>
+template <typename TA, int KIND>
 static int launch_scan(const ScanArgs& A, int B, bool single, cudaStream_t stream) {
     switch (scan_shape(A.d)) {
-        case 0: return launch_scan_shape<TA, 4, 8, GATED>(A, B, single, stream);
-        case 1: return launch_scan_shape<TA, 8, 8, GATED>(A, B, single, stream);
-        case 2: return launch_scan_shape<TA, 8, 16, GATED>(A, B, single, stream);
-        case 3: return launch_scan_shape<TA, 8, 32, GATED>(A, B, single, stream);
+        case 0: return launch_scan_shape<TA, 4, 8, KIND>(A, B, single, stream);
+        case 1: return launch_scan_shape<TA, 8, 8, KIND>(A, B, single, stream);
+        case 2: return launch_scan_shape<TA, 8, 16, KIND>(A, B, single, stream);
+        case 3: return launch_scan_shape<TA, 8, 32, KIND>(A, B, single, stream);
     }
     return 1;
 }
@@ -376,16 +411,19 @@ TL_EXPORT int tl_linear_scan(const void* proj, int act_dtype, int stride, int q_
                              const float* gates, float cap, const float* decay, const float* inv_freq, int rot,
                              int interleaved, const int* pos, float q_scale, float k_scale, float* state,
                              long long slot_stride, const int* q_start, const int* slots, float* out, int B, int H,
-                             int d, int dv, float den_eps, int single_tokens, cudaStream_t stream) {
+                             int d, int dv, float den_eps, int single_tokens, const float* lower, const float* bias,
+                             cudaStream_t stream) {
     // single_tokens: every request of the step brings exactly one token (the caller knows; the step kernel takes it)
     if (B <= 0 || H <= 0) return 0;
     if (H > 65535 || (rot & 1) || rot > d) return 1;
     const ScanArgs A{proj, stride, q_off, k_off, v_off, gates, cap, decay, inv_freq, rot, interleaved, pos, q_scale, k_scale,
-                     state, slot_stride, q_start, slots, out, H, d, dv, den_eps};
+                     state, slot_stride, q_start, slots, out, H, d, dv, den_eps, lower, bias};
     const bool gated = gates != nullptr;
+    if ((lower == nullptr) != (bias == nullptr) || (lower && (gated || decay || rot))) return 1;
     const bool single = single_tokens != 0;
-    if (act_dtype == TL_F32) return gated ? launch_scan<float, true>(A, B, single, stream) : launch_scan<float, false>(A, B, single, stream);
-    return gated ? launch_scan<bf16, true>(A, B, single, stream) : launch_scan<bf16, false>(A, B, single, stream);
+    if (lower) return act_dtype == TL_F32 ? launch_scan<float, SCAN_CHANNEL>(A, B, single, stream) : launch_scan<bf16, SCAN_CHANNEL>(A, B, single, stream);
+    if (act_dtype == TL_F32) return gated ? launch_scan<float, SCAN_GATED>(A, B, single, stream) : launch_scan<float, SCAN_FIXED>(A, B, single, stream);
+    return gated ? launch_scan<bf16, SCAN_GATED>(A, B, single, stream) : launch_scan<bf16, SCAN_FIXED>(A, B, single, stream);
 }
 
 // ------------------------------------------------------------------ per-head RMS norm, weight, gate

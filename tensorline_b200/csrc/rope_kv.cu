@@ -13,7 +13,8 @@
 // the rotated dimensions (`interleaved`: pair i is dimensions (2i, 2i + 1) instead of (i, i + rot/2)), and an
 // RMS norm of every q and k head over its d dimensions with a weight of its own (`q_norm`, `k_norm`, `norm_eps`),
 // applied after the bias and before the rotation, statistics in float.  `norm_dim` (0: d) is the number of dimensions the
-// mean of squares is taken over: a head padded with zeros to d is normalised over its own size.
+// mean of squares is taken over: a head padded with zeros to d is normalised over its own size.  `norm_cast` 0: x * rstd * w in
+// float with one rounding at the end, instead of a rounding to the activation type before the weight.
 #include "common.cuh"
 
 // grid (T, heads): one block per (token, head), one thread per pair of dimensions, so that all loads
@@ -25,7 +26,7 @@ __global__ void rope_kv_kernel(TA* __restrict__ qkv, const TW* __restrict__ bias
                                const float* __restrict__ inv_freq, int rot, int nq, int nkv, int d,
                                TA* __restrict__ k_pages, TA* __restrict__ v_pages, int interleaved,
                                const float* __restrict__ q_norm, const float* __restrict__ k_norm, float norm_eps,
-                               int norm_dim, const TlLimits L) {
+                               int norm_dim, int norm_cast, const TlLimits L) {
     __shared__ float red[33];
     const int t = blockIdx.x, hh = blockIdx.y;
     const int p = pos[t];
@@ -60,9 +61,10 @@ __global__ void rope_kv_kernel(TA* __restrict__ qkv, const TW* __restrict__ bias
         float a = to_f<TA>(row[e1]);
         float b = to_f<TA>(row[e2]);
         if (bias) { a += to_f<TW>(bias[hh * d + e1]); b += to_f<TW>(bias[hh * d + e2]); }
-        if (nw) {                                                // cast before the weight, as the layer norms do
-            a = to_f<TA>(from_f<TA>(a * rstd)) * nw[e1];
-            b = to_f<TA>(from_f<TA>(b * rstd)) * nw[e2];
+        if (nw) {                                                // `norm_cast`: rounded before the weight, as the layer norms do
+            a *= rstd; b *= rstd;
+            if (norm_cast) { a = to_f<TA>(from_f<TA>(a)); b = to_f<TA>(from_f<TA>(b)); }
+            a *= nw[e1]; b *= nw[e2];
         }
         if (rotate_head && i < rhalf) {
             float s, c;
@@ -188,7 +190,7 @@ TL_EXPORT int tl_rope_kv_write(void* qkv, int act_dtype, const void* bias, int b
                                int page_size, const float* inv_freq, int rot, int nq, int nkv, int d,
                                void* k_pages, void* v_pages, int write_kv, int T, const float* pieces, int splits,
                                long long plane, int interleaved, const float* q_norm, const float* k_norm,
-                               float norm_eps, int norm_dim, int table_rows, int total_pages, int* fault, cudaStream_t stream) {
+                               float norm_eps, int norm_dim, int norm_cast, int table_rows, int total_pages, int* fault, cudaStream_t stream) {
     const TlLimits L{table_rows, total_pages, fault};
     if (T <= 0) return 0;
     if (rot < 0 || rot > d || (rot & 1) || (d & 1)) return 1;     // cudaErrorInvalidValue
@@ -213,7 +215,7 @@ TL_EXPORT int tl_rope_kv_write(void* qkv, int act_dtype, const void* bias, int b
     const int threads = half < 256 ? ((half + 31) / 32) * 32 : 256;
 #define LAUNCH(TA, TW) rope_kv_kernel<TA, TW><<<grid, threads, 0, stream>>>( \
         (TA*)qkv, (const TW*)bias, pos, req_slot, table, max_pages, page_size, inv_freq, rot, nq, nkv, d, \
-        (TA*)k_pages, (TA*)v_pages, interleaved, q_norm, k_norm, norm_eps, norm_dim, L)
+        (TA*)k_pages, (TA*)v_pages, interleaved, q_norm, k_norm, norm_eps, norm_dim, norm_cast, L)
     if (act_dtype == TL_F32) { if (bias_dtype == TL_F32) LAUNCH(float, float); else LAUNCH(float, bf16); }
     else                     { if (bias_dtype == TL_F32) LAUNCH(bf16, float);  else LAUNCH(bf16, bf16); }
 #undef LAUNCH

@@ -1,0 +1,285 @@
+// The residual sum with several waiting addends, the norm behind it and the token shift, one kernel, all float arithmetic.
+//
+//   v[t]  = x[t] (+ base[t]) (+ row) + sum_i scale_i * a_i[t]      a_i of the activation type, scale_i a vector over the width
+//                                                                  (a layer scale; null: ones), base float [T, W], row [W]
+//   n[t]  = v[t] / sqrt(mean(v[t]^2) + eps) * w
+//   h[t]  = n[t] + (n[t-1] - n[t]) * shift                         shift [W]; null: h = n
+// n[t-1] is the row of the request's token in front of t: the row in front in the step, or, for the first row of a request's
+// portion, what the request's slot of `prev` (float [slots, W]) holds, or zeros at position 0.  The block that owns a
+// portion's first row leaves n of the portion's LAST row in the slot after it has read the slot, so a launch both reads and
+// renews the state and no two blocks touch the same slot.
+// A row's neighbour is normalised again by the block that needs it (NR rows a block, NR + 1 norms), from the same inputs in
+// the same order of additions, so the result does not depend on how a step was cut.  With a shift x is therefore left as it
+// is (the addends stay with the caller until a norm without a shift writes them); without one x takes v (`write_x`).
+// `rows` picks rows (no shift; x is left alone); `h` null: only the sum.
+#include "common.cuh"
+
+constexpr int SUM_ADDENDS = 3;
+
+struct SumNormArgs {
+    float* x; int W;
+    const void* add[SUM_ADDENDS]; const float* scale[SUM_ADDENDS]; int n_add;
+    const float* base; const float* row;
+    const void* w; float eps;
+    void* h;
+    const int* rows; int T; int write_x;
+    const float* shift; float* prev; long long prev_stride;
+    const int* pos; const int* req_slot; const int* q_start; int B; int single;
+};
+
+template <int VEC> struct Pack;
+template <> struct Pack<4> {
+    static __device__ __forceinline__ void load(const float* p, float (&v)[4]) {
+        const float4 t = *reinterpret_cast<const float4*>(p); v[0] = t.x; v[1] = t.y; v[2] = t.z; v[3] = t.w;
+    }
+    static __device__ __forceinline__ void load(const bf16* p, float (&v)[4]) {
+        const uint2 t = *reinterpret_cast<const uint2*>(p);
+        const __nv_bfloat162 a = *reinterpret_cast<const __nv_bfloat162*>(&t.x), b = *reinterpret_cast<const __nv_bfloat162*>(&t.y);
+        v[0] = __low2float(a); v[1] = __high2float(a); v[2] = __low2float(b); v[3] = __high2float(b);
+    }
+    static __device__ __forceinline__ void store(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+    static __device__ __forceinline__ void store(bf16* p, const float (&v)[4]) {
+        __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+        uint2 t; t.x = *reinterpret_cast<uint32_t*>(&a); t.y = *reinterpret_cast<uint32_t*>(&b);
+        *reinterpret_cast<uint2*>(p) = t;
+    }
+};
+template <> struct Pack<1> {
+    template <typename T> static __device__ __forceinline__ void load(const T* p, float (&v)[1]) { v[0] = to_f<T>(*p); }
+    template <typename T> static __device__ __forceinline__ void store(T* p, const float (&v)[1]) { *p = from_f<T>(v[0]); }
+};
+
+// v of one row in this thread's columns, and the thread's share of the sum of its squares
+template <typename TA, int VEC, int NV>
+__device__ __forceinline__ float sum_row(const SumNormArgs& A, size_t t, int nvec, float (&v)[NV][VEC]) {
+    using P = Pack<VEC>;
+    const size_t base = t * (size_t)A.W;
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        const int c = threadIdx.x + k * blockDim.x;
+        if (c < nvec) P::load(A.x + base + (size_t)c * VEC, v[k]);
+    }
+    if (A.base) {
+#pragma unroll
+        for (int k = 0; k < NV; ++k) {
+            const int c = threadIdx.x + k * blockDim.x;
+            if (c < nvec) {
+                float b[VEC]; P::load(A.base + base + (size_t)c * VEC, b);
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) v[k][e] += b[e];
+            }
+        }
+    }
+    if (A.row) {
+#pragma unroll
+        for (int k = 0; k < NV; ++k) {
+            const int c = threadIdx.x + k * blockDim.x;
+            if (c < nvec) {
+                float b[VEC]; P::load(A.row + (size_t)c * VEC, b);
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) v[k][e] += b[e];
+            }
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < SUM_ADDENDS; ++i) {
+        if (i < A.n_add) {
+            const TA* a = (const TA*)A.add[i] + base;
+#pragma unroll
+            for (int k = 0; k < NV; ++k) {
+                const int c = threadIdx.x + k * blockDim.x;
+                if (c < nvec) {
+                    float av[VEC], sv[VEC];
+                    P::load(a + (size_t)c * VEC, av);
+                    if (A.scale[i]) P::load(A.scale[i] + (size_t)c * VEC, sv);
+                    else {
+#pragma unroll
+                        for (int e = 0; e < VEC; ++e) sv[e] = 1.0f;
+                    }
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) v[k][e] = fmaf(sv[e], av[e], v[k][e]);
+                }
+            }
+        }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < NV; ++k)
+        if (threadIdx.x + k * blockDim.x < nvec)
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) ss = fmaf(v[k][e], v[k][e], ss);
+    return ss;
+}
+
+// L sums over the block at once; the order of additions is that of one sum alone.  red: [L][33] floats.
+template <int L>
+__device__ __forceinline__ void block_sums(float (&s)[L], float (*red)[33]) {
+    const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;
+#pragma unroll
+    for (int j = 0; j < L; ++j) s[j] = warp_sum(s[j]);
+    __syncthreads();
+    if (lane == 0) {
+#pragma unroll
+        for (int j = 0; j < L; ++j) red[j][wid] = s[j];
+    }
+    __syncthreads();
+    for (int j = wid; j < L; j += nw) {
+        float t = lane < nw ? red[j][lane] : 0.f;
+        t = warp_sum(t);
+        if (lane == 0) red[j][32] = t;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int j = 0; j < L; ++j) s[j] = red[j][32];
+}
+
+template <typename TA, typename TW, int VEC, int NV, int NR, bool SHIFT>
+__global__ void sum_norm_kernel(const SumNormArgs A) {
+    using P = Pack<VEC>;
+    constexpr int L = NR + (SHIFT ? 1 : 0);
+    __shared__ float red[L][33];
+    const int nvec = A.W / VEC;
+    const int t0 = blockIdx.x * NR;
+    float wv[NV][VEC];
+    const bool early = gridDim.x <= 128;                     // few rows: the weights, nobody's output, come before the wait
+    auto load_w = [&]() {
+        if (A.h == nullptr) return;
+#pragma unroll
+        for (int k = 0; k < NV; ++k) {
+            const int c = threadIdx.x + k * blockDim.x;
+            if (c < nvec) P::load((const TW*)A.w + (size_t)c * VEC, wv[k]);
+        }
+    };
+    if (early) load_w();
+    grid_dependency_wait();
+    grid_dependency_trigger();
+    if (!early) load_w();
+    float v[L][NV][VEC], ss[L];
+#pragma unroll
+    for (int j = 0; j < L; ++j) {
+        const int t = t0 + j - (SHIFT ? 1 : 0);
+        ss[j] = 0.f;
+        if (t >= 0 && t < A.T && !(SHIFT && j == 0 && A.single)) ss[j] = sum_row<TA, VEC, NV>(A, A.rows ? (size_t)A.rows[t] : (size_t)t, nvec, v[j]);
+    }
+    if (!SHIFT && A.write_x) {
+#pragma unroll
+        for (int j = 0; j < L; ++j)
+            if (t0 + j < A.T)
+#pragma unroll
+                for (int k = 0; k < NV; ++k) {
+                    const int c = threadIdx.x + k * blockDim.x;
+                    if (c < nvec) P::store(A.x + (size_t)(t0 + j) * A.W + (size_t)c * VEC, v[j][k]);
+                }
+    }
+    if (A.h == nullptr) return;
+    block_sums<L>(ss, red);
+#pragma unroll
+    for (int j = 0; j < L; ++j) {
+        const float rstd = 1.0f / sqrtf(ss[j] / (float)A.W + A.eps);
+#pragma unroll
+        for (int k = 0; k < NV; ++k)
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) v[j][k][e] = v[j][k][e] * rstd * wv[k][e];
+    }
+    TA* h = (TA*)A.h;
+    if (!SHIFT) {
+#pragma unroll
+        for (int j = 0; j < L; ++j)
+            if (t0 + j < A.T)
+#pragma unroll
+                for (int k = 0; k < NV; ++k) {
+                    const int c = threadIdx.x + k * blockDim.x;
+                    if (c < nvec) P::store(h + (size_t)(t0 + j) * A.W + (size_t)c * VEC, v[j][k]);
+                }
+        return;
+    }
+    unsigned firsts = 0;                                     // bit j: row t0 + j is the first of its request's portion
+#pragma unroll
+    for (int j = 0; j < NR; ++j) {
+        const int t = t0 + j;
+        if (t >= A.T) continue;
+        const int slot = A.req_slot[t];
+        const bool first = A.single || t == 0 || A.req_slot[t - 1] != slot;
+        if (first) firsts |= 1u << j;
+        const bool start = first && A.pos[t] == 0;
+        const float* st = A.prev + (size_t)slot * A.prev_stride;
+#pragma unroll
+        for (int k = 0; k < NV; ++k) {
+            const int c = threadIdx.x + k * blockDim.x;
+            if (c < nvec) {
+                float pv[VEC], mu[VEC], o[VEC];
+                P::load(A.shift + (size_t)c * VEC, mu);
+                if (start) {
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) pv[e] = 0.f;
+                } else if (first) P::load(st + (size_t)c * VEC, pv);
+                else {
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) pv[e] = v[j][k][e];
+                }
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) o[e] = fmaf(pv[e] - v[j + 1][k][e], mu[e], v[j + 1][k][e]);
+                P::store(h + (size_t)t * A.W + (size_t)c * VEC, o);
+            }
+        }
+    }
+    // the state: n of the portion's last row, by the block (and the threads) that have just read the slot
+#pragma unroll 1
+    for (int j = 0; j < NR; ++j) {
+        if (!((firsts >> j) & 1u)) continue;
+        const int t = t0 + j;
+        float* st = A.prev + (size_t)A.req_slot[t] * A.prev_stride;
+        int last = t;
+        if (!A.single) {                                     // the request whose rows start at t
+            int lo = 0, hi = A.B - 1;
+            while (lo < hi) { const int mid = (lo + hi) >> 1; if (A.q_start[mid] < t) lo = mid + 1; else hi = mid; }
+            last = A.q_start[lo + 1] - 1;
+        }
+        float n[1][NV][VEC], s1[1];
+        s1[0] = sum_row<TA, VEC, NV>(A, (size_t)last, nvec, n[0]);
+        block_sums<1>(s1, red);
+        const float rstd = 1.0f / sqrtf(s1[0] / (float)A.W + A.eps);
+#pragma unroll
+        for (int k = 0; k < NV; ++k) {
+            const int c = threadIdx.x + k * blockDim.x;
+            if (c < nvec) {
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) n[0][k][e] = n[0][k][e] * rstd * wv[k][e];
+                P::store(st + (size_t)c * VEC, n[0][k]);
+            }
+        }
+    }
+}
+
+template <typename TA, typename TW, int VEC>
+static int launch_sum_norm(const SumNormArgs& A, cudaStream_t stream) {
+    const int nvec = A.W / VEC;
+    const bool shift = A.shift != nullptr;
+    // one thread count for a width whatever the step (the order of additions), rows a block by how many there are
+#define SN(NV, NR, S) launch_after_wait(sum_norm_kernel<TA, TW, VEC, NV, NR, S>, dim3((A.T + NR - 1) / NR), dim3(((nvec + NV - 1) / NV + 31) / 32 * 32), 0, stream, A)
+    if (nvec <= 1024) {
+        if (shift) return (A.T >= 512 && !A.single) ? SN(1, 3, true) : SN(1, 1, true);
+        return SN(1, 1, false);
+    }
+    if (nvec <= 2048) return shift ? SN(2, 1, true) : SN(2, 1, false);
+    if (nvec <= 8192) return shift ? SN(8, 1, true) : SN(8, 1, false);
+#undef SN
+    return 1;
+}
+
+TL_EXPORT int tl_sum_norm(float* x, int W, int T, const void* a0, const float* s0, const void* a1, const float* s1, const void* a2,
+                          const float* s2, int n_add, int act_dtype, const float* base, const float* row, const void* w, int w_dtype,
+                          float eps, void* h, const int* rows, int write_x, const float* shift, float* prev, long long prev_stride,
+                          const int* pos, const int* req_slot, const int* q_start, int B, int single, cudaStream_t stream) {
+    if (T <= 0) return 0;
+    if (n_add < 0 || n_add > SUM_ADDENDS || (shift && (rows || write_x || !h || !prev || !pos || !req_slot || !q_start)) || (rows && write_x)) return 1;
+    const SumNormArgs A{x, W, {a0, a1, a2}, {s0, s1, s2}, n_add, base, row, w, eps, h, rows, T, write_x, shift, prev, prev_stride,
+                        pos, req_slot, q_start, B, single};
+    const uintptr_t all = (uintptr_t)x | (uintptr_t)a0 | (uintptr_t)s0 | (uintptr_t)a1 | (uintptr_t)s1 | (uintptr_t)a2 | (uintptr_t)s2 |
+                          (uintptr_t)base | (uintptr_t)row | (uintptr_t)w | (uintptr_t)h | (uintptr_t)shift | (uintptr_t)prev;
+    const bool vec = (W & 3) == 0 && (prev_stride & 3) == 0 && (all & 15) == 0;
+#define SNT(TA, TW) (vec ? launch_sum_norm<TA, TW, 4>(A, stream) : launch_sum_norm<TA, TW, 1>(A, stream))
+    if (act_dtype == TL_F32) return w_dtype == TL_F32 ? SNT(float, float) : SNT(float, bf16);
+    return w_dtype == TL_F32 ? SNT(bf16, float) : SNT(bf16, bf16);
+#undef SNT
+}

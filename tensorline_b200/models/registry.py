@@ -18,6 +18,7 @@ from ..config.vutesun import VutesunConfig
 from ..config.dekerax import DekeraxConfig
 from ..config.sumuvik import SumuvikConfig
 from ..config.tenalorn import TenalornConfig
+from ..config.zosurax import ZosuraxConfig
 from ..parts import Runtime
 from ..weights import load_weights
 from .qwen2 import describe_qwen2
@@ -25,6 +26,7 @@ from .vutesun import describe_vutesun
 from .dekerax import describe_dekerax
 from .sumuvik import describe_sumuvik
 from .tenalorn import describe_tenalorn
+from .zosurax import describe_zosurax
 from .spec import Model
 
 
@@ -57,6 +59,7 @@ register_architecture("Vutesun", VutesunConfig, describe_vutesun)
 register_architecture("Dekerax", DekeraxConfig, describe_dekerax)
 register_architecture("Sumuvik", SumuvikConfig, describe_sumuvik)
 register_architecture("Tenalorn", TenalornConfig, describe_tenalorn)
+register_architecture("Zosurax", ZosuraxConfig, describe_zosurax)
 
 
 def load_config(folder):
@@ -78,9 +81,9 @@ def load_model(folder, rt: Runtime):
     expected = model.expected_tensors()
     if model.spec.tie_word_embeddings:
         # A tied head is the embedding table: a stored head is neither loaded nor an error.
-        head = f"{model.spec.head_prefix}.weight"
-        expected = {k: v for k, v in expected.items() if k != head}
-        weights = load_weights(folder, expected, device=rt.device, ignore=(head,))
+        head = tuple(model.head.expected_tensors(model.spec.head_prefix))
+        expected = {k: v for k, v in expected.items() if k not in head}
+        weights = load_weights(folder, expected, device=rt.device, ignore=head)
     else:
         weights = load_weights(folder, expected, device=rt.device)
     model.bind(weights)

@@ -15,7 +15,7 @@ from dataclasses import dataclass
 import torch
 
 from ..parts import BLOCKS, EMBEDDINGS, HEADS, NORMS, POSITION_ENCODINGS, KVCacheView, PartSpec, Runtime, TensorSpec
-from ..parts.linear import with_row
+from ..parts.linear import with_base, with_row
 
 
 @dataclass(frozen=True)
@@ -29,6 +29,7 @@ class RunEntry:
     layer: int                          # index into ModelSpec.layers
     reads_cache_of: int | None = None   # index of an earlier run entry whose cache this one reads
     add_row: int | None = None          # row of `ModelSpec.stream_rows` added to the residual stream in front of this entry
+    add_start: bool = False             # the stream as it was in front of the first entry is added to it in front of this one (first)
 
 
 @dataclass(frozen=True)
@@ -154,7 +155,10 @@ class Model:
         if self.embedding_norm is not None:
             x = self.embedding_norm.norm_stream(x)
         pending = None
+        start = x.clone() if any(e.add_start for e in self.spec.run) else None      # x itself is added to in place
         for i, e in enumerate(self.spec.run):
+            if e.add_start:
+                pending = with_base(x, pending, start)
             if e.add_row is not None:
                 pending = with_row(x, pending, self.stream_rows[e.add_row], self.spec.stream_rows_eps)
             if e.reads_cache_of is None:

@@ -14,7 +14,7 @@ import torch
 from .csrc.build import CHECK_BUILD, load_library
 
 CORE_SOURCES = ["elementwise.cu", "rope_kv.cu", "attn_tokenwise.cu", "gemm_f32.cu", "sampling.cu", "recurrent.cu", "moe.cu",
-                "delta.cu", "latent.cu", "rglru.cu", "streams.cu"]
+                "delta.cu", "latent.cu", "rglru.cu", "streams.cu", "stream_norm.cu", "attn_mixed_tokenwise.cu"]
 
 _P, _I, _F = ctypes.c_void_p, ctypes.c_int, ctypes.c_float
 
@@ -26,13 +26,13 @@ _SIGNATURES = {
     "tl_head_gate": [_P, _I, _P, _I, _I, _I, _P],
     "tl_post_norm_add_norm": [_P, _P, _P, _P, _P, _I, _P, _I, _P, _I, _I, _F, _I, _P],
     "tl_rope_kv_write": [_P, _I, _P, _I, _P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _P, _P, _I, _I, _P, _I, ctypes.c_longlong,
-                         _I, _P, _P, _F, _I, _I, _I, _P, _P],
+                         _I, _P, _P, _F, _I, _I, _I, _I, _P, _P],
     "tl_attn_tokenwise": [_P, _I, _P, _I, _P, _P, _P, _I, _I, _P, _P, _I, _I, _I, _I, _I, _F, _P, _I, _P, _I, _P, _I, _I, _P, _P],
     "tl_gemm_f32": [_P, _I, _P, _I, _I, _P, _P, _I, _I, _I, _I, _P],
     "tl_argmax": [_P, _I, _I, _I, _P, _P, _P],
     "tl_sample": [_P, _I, _I, _I, _P, _P, _P, _P, _P],
     "tl_linear_scan": [_P, _I, _I, _I, _I, _I, _P, _F, _P, _P, _I, _I, _P, _F, _F, _P, ctypes.c_longlong, _P, _P, _P, _I, _I,
-                       _I, _I, _F, _I, _P],
+                       _I, _I, _F, _I, _P, _P, _P],
     "tl_scan_state_floats": [_I, _I],
     "tl_scan_columns": [],
     "tl_head_norm_gate": [_P, _P, _I, _I, _P, _I, _P, _I, _I, _I, _I, _F, _I, _P],
@@ -59,6 +59,9 @@ _SIGNATURES = {
     "tl_embed_streams": [_P, _P, _I, _P, _I, _I, _F, _I, _P, _I, _I, _I, _P, _P, _P, _P],
     "tl_remember_last": [_P, _P, _P, _I, _P, _P],
     "tl_stream_step": [_P, _I, _I, _P, _F, _P, _F, _I, _P, _P, _P, _P, _I, _F, _P, _P, _P, _I, _I, _P],
+    "tl_sum_norm": [_P, _I, _I, _P, _P, _P, _P, _P, _P, _I, _I, _P, _P, _P, _I, _F, _P, _P, _I, _P, _P, ctypes.c_longlong, _P, _P, _P, _I,
+                    _I, _P],
+    "tl_attn_mixed_tokenwise": [_P, _I, _P, _I, _P, _P, _P, _I, _I, _P, _P, _I, _I, _I, _I, _F, _P, _I, _I, _P, _P],
     "tl_softcap": [_P, ctypes.c_longlong, _F, _P],
     "tl_sigmoid_gate": [_P, _P, _I, _P, _I, _I, _I, _P],
     "tl_head_matmul": [_P, _I, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _P],
@@ -331,6 +334,54 @@ def stream_step(x: torch.Tensor, S: int, a: torch.Tensor | None = None, alpha: f
                                  _ptr(rows), R, int(rows is None), _stream()), "stream_step")
 
 
+SUM_ADDENDS = 3                     # addends one launch of `sum_norm` takes
+
+
+def sum_norm(x: torch.Tensor, addends=(), base: torch.Tensor | None = None, row: torch.Tensor | None = None,
+             w: torch.Tensor | None = None, eps: float = 0.0, h: torch.Tensor | None = None, rows: torch.Tensor | None = None,
+             shift: torch.Tensor | None = None, prev: torch.Tensor | None = None, ctx=None) -> None:
+    """v = x (+ base) (+ row) + sum of scale_i * a_i in float32 (`addends`: up to SUM_ADDENDS pairs (a [T, W] of the activation
+    type, scale float32 [W] or None); base float32 [T, W], row float32 [W]).  Without `rows` and `shift` x becomes v.  With `h`
+    its RMS norm times `w` goes to `h` (activation type).  `rows` (int32) picks rows; x is then left alone.  `shift` (float32
+    [W], with `prev` float32 [slots, W] and the step's `ctx`): h = n + (n' - n) * shift, n' the normed row of the request's
+    token in front (from `prev` for the first row of a portion, zeros at position 0; `prev` then takes the portion's last
+    normed row); x is left alone."""
+    T, W = x.shape
+    addends = tuple(addends)
+    act = h.dtype if h is not None else (addends[0][0].dtype if addends else torch.float32)
+    if x.dtype != torch.float32 or not x.is_contiguous() or len(addends) > SUM_ADDENDS:
+        raise KernelError(f"sum_norm: x must be float32 [T, W] and there are at most {SUM_ADDENDS} addends")
+    for a, sc in addends:
+        if a.shape != (T, W) or a.dtype != act or not a.is_contiguous():
+            raise KernelError("sum_norm: addends must be [T, W] of the activation type, contiguous")
+        if sc is not None and (sc.dtype != torch.float32 or sc.numel() != W or not sc.is_contiguous()):
+            raise KernelError("sum_norm: an addend's scale must be float32 [W]")
+    if base is not None and (base.shape != (T, W) or base.dtype != torch.float32 or not base.is_contiguous()):
+        raise KernelError("sum_norm: base must be float32 [T, W]")
+    for name, t in (("row", row), ("shift", shift)):
+        if t is not None and (t.dtype != torch.float32 or t.numel() != W or not t.is_contiguous()):
+            raise KernelError(f"sum_norm: {name} must be float32 [W]")
+    R = T if rows is None else rows.numel()
+    if h is not None and (h.shape != (R, W) or w is None or w.numel() != W or not w.is_contiguous() or not h.is_contiguous()):
+        raise KernelError("sum_norm: h [rows, W] comes with a weight [W]")
+    if rows is not None:
+        _ints(rows, "rows")
+        if h is None:
+            raise KernelError("sum_norm: picked rows are normalised")
+    stride = 0
+    if shift is not None:
+        if prev is None or prev.dtype != torch.float32 or prev.shape[1] != W or not prev.is_contiguous() or ctx is None or h is None or rows is not None:
+            raise KernelError("sum_norm: a shift needs h, the step's context and a state float32 [slots, W]")
+        stride = prev.shape[1]
+    a = [(_ptr(t), _ptr(sc)) for t, sc in addends] + [(None, None)] * (SUM_ADDENDS - len(addends))
+    _check(core().tl_sum_norm(_ptr(x), W, R, *a[0], *a[1], *a[2], len(addends), dtype_code(act), _ptr(base), _ptr(row), _ptr(w),
+                              dtype_code(w.dtype) if w is not None else 0, float(eps), _ptr(h), _ptr(rows),
+                              int(rows is None and shift is None), _ptr(shift), _ptr(prev), stride,
+                              _ptr(ctx.pos) if shift is not None else None, _ptr(ctx.req_slot) if shift is not None else None,
+                              _ptr(ctx.q_start) if shift is not None else None, ctx.B if shift is not None else 0,
+                              int(ctx.decode_only) if shift is not None else 0, _stream()), "sum_norm" if shift is None else "sum_norm_shift")
+
+
 def softcap(z: torch.Tensor, cap: float) -> None:
     """z <- cap * tanh(z / cap) in place, z float32."""
     if z.dtype != torch.float32 or not z.is_contiguous():
@@ -489,12 +540,13 @@ def rope_kv_write(qkv: torch.Tensor, bias: torch.Tensor | None, pos: torch.Tenso
                   table: torch.Tensor, page_size: int, inv_freq: torch.Tensor, rot: int, nq: int, nkv: int,
                   d: int, k_pages: torch.Tensor | None, v_pages: torch.Tensor | None, write_kv: bool = True,
                   pieces: torch.Tensor | None = None, pairing: str = "half", q_norm: torch.Tensor | None = None,
-                  k_norm: torch.Tensor | None = None, norm_eps: float = 0.0, norm_dim: int = 0) -> None:
+                  k_norm: torch.Tensor | None = None, norm_eps: float = 0.0, norm_dim: int = 0, norm_cast: bool = True) -> None:
     """Bias, rotary encoding of q and k in place, and the write of k, v into their pages.
     `pairing`: "half" rotates dimensions (i, i + rot/2), "interleaved" (2i, 2i + 1).  `q_norm`, `k_norm`
     (float32 [d], both or neither): every q and k head is RMS-normalised over its d dimensions (after the
     bias, before the rotation; statistics in float32) and multiplied by the weight.  `norm_dim` (0: d): the mean of squares
-    is taken over this many dimensions (a head that is padded with zeros to d).
+    is taken over this many dimensions (a head that is padded with zeros to d).  `norm_cast` False: the normalised values are
+    not rounded to the activation type before the weight.
     `pieces` [S, T, width] float32: the projection as a split-K product left it; the kernel sums them
     (bfloat16, full rotary, d % 16 == 0 only) and qkv is output only (its q columns are written)."""
     T = qkv.shape[0]
@@ -529,7 +581,7 @@ def rope_kv_write(qkv: torch.Tensor, bias: torch.Tensor | None, pos: torch.Tenso
         _ptr(pos), _ptr(req_slot), _ptr(table), table.shape[1], page_size, _ptr(inv_freq), rot, nq, nkv, d,
         _ptr(k_pages) if write_kv else None, _ptr(v_pages) if write_kv else None, int(write_kv), T,
         _ptr(pieces), splits, plane, int(pairing == "interleaved"), _ptr(q_norm), _ptr(k_norm), float(norm_eps),
-        int(norm_dim), table.shape[0], k_pages.shape[0] if write_kv else 0, fault_words(qkv.device), _stream()), "rope_kv_write")
+        int(norm_dim), int(norm_cast), table.shape[0], k_pages.shape[0] if write_kv else 0, fault_words(qkv.device), _stream()), "rope_kv_write")
 
 
 def attn_tokenwise(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
@@ -562,6 +614,29 @@ def attn_tokenwise(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_pages: t
                                     int(window or 0), float(scale), _ptr(sink), int(keep_first), _ptr(gate), int(chunk or 0),
                                     _ptr(slopes), table.shape[0], k_pages.shape[0], fault_words(out.device), _stream()),
            "attn_tokenwise")
+
+
+def attn_mixed_tokenwise(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
+                         table: torch.Tensor, page_size: int, pos: torch.Tensor, req_slot: torch.Tensor, nq: int, nkv: int, d: int,
+                         scale: float, mix: torch.Tensor) -> None:
+    """Exact-order paged causal attention whose heads' softmax weights are mixed before they meet the values: head h applies
+    sum_g mix[h, g] P_g to the values of its own KV head (`mix` float32 [nq, nq])."""
+    T = out.shape[0]
+    if out.shape[1] != nq * d or out.dtype != q.dtype or k_pages.dtype != q.dtype:
+        raise KernelError("attn_mixed_tokenwise: out must be [T, nq*d] and all tensors of one type")
+    if d > 512 or 4 * nq * (d + 35) > 227 * 1024:
+        raise KernelError(f"attn_mixed_tokenwise: {nq} heads of {d} are not supported")
+    _contig(out, "out"); _contig(k_pages, "k_pages"); _contig(v_pages, "v_pages")
+    _ints(pos, "pos"); _ints(req_slot, "req_slot"); _ints(table, "table")
+    _mix(mix, nq)
+    _check(core().tl_attn_mixed_tokenwise(_ptr(q), q_stride, _ptr(out), dtype_code(q.dtype), _ptr(k_pages), _ptr(v_pages), _ptr(table),
+                                          table.shape[1], page_size, _ptr(pos), _ptr(req_slot), T, nq, nkv, d, float(scale), _ptr(mix),
+                                          table.shape[0], k_pages.shape[0], fault_words(out.device), _stream()), "attn_mixed_tokenwise")
+
+
+def _mix(mix, nq: int) -> None:
+    if mix.dtype != torch.float32 or mix.shape != (nq, nq) or not mix.is_contiguous():
+        raise KernelError("the heads' mix must be float32 [query heads, query heads]")
 
 
 def _sink(sink, nq: int, who: str) -> None:
@@ -633,18 +708,24 @@ def linear_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, H: int, 
                 q_start: torch.Tensor, slots: torch.Tensor, pos: torch.Tensor, out: torch.Tensor, *, B: int,
                 decay: torch.Tensor | None = None, gates: torch.Tensor | None = None, cap: float = 1.0,
                 inv_freq: torch.Tensor | None = None, rot: int = 0, pairing: str = "half", q_scale: float = 1.0,
-                k_scale: float = 1.0, den_eps: float = 0.0, single_tokens: bool = False) -> None:
+                k_scale: float = 1.0, den_eps: float = 0.0, single_tokens: bool = False,
+                lower: torch.Tensor | None = None, bias: torch.Tensor | None = None) -> None:
     """S_t = a_t S_(t-1) + b_t k_t v_t^T and o_t = S_t^T q_t per (request, head), tokens of a request in order, the state
     read from and left in `state[slot]` (float32, one row a slot, in the kernel's own layout: `scan_state_floats`).
     q, k [H, d] and v [H, dv] of token t are at `proj[t, q_off:]`, `proj[t, k_off:]`, `proj[t, v_off:]`.
     `decay` (float32 [H]): a_t = decay[h], b_t = 1.  `gates` (float32 [T, 2H], input then forget pre-activations): the
     capped log gates with a running maximum, a normaliser, and o_t divided by max(|n_t . q_t|, exp(-m_t)) + den_eps.
+    `lower` and `bias` (float32 [H * d] each, instead of both): a_t is a vector over the rows of S, f = lower + (1 - lower)
+    sigmoid(x + bias) with x [H, d] at `proj[t, k_off:]`; b_t k_t is 1 - f, q is passed through silu, nothing is rotated.
     q and k are rotated by `pos` over their first `rot` dimensions (`inv_freq` float32 [rot/2]) and scaled; a request's
     tokens of the step stand at consecutive positions (the kernel reads the first one's).  out float32 [T, H * dv].
     `single_tokens`: every request brings exactly one token (T == B): the step kernel, which gives the scan kernel's bits."""
     T = proj.shape[0]
-    if (decay is None) == (gates is None):
-        raise KernelError("linear_scan: either a fixed decay per head or gate pre-activations")
+    if (decay is not None) + (gates is not None) + (lower is not None) != 1 or (lower is None) != (bias is None):
+        raise KernelError("linear_scan: a fixed decay per head, gate pre-activations, or channel gates with their lower bound and bias")
+    for name, t in (("lower", lower), ("bias", bias)):
+        if t is not None and (t.dtype != torch.float32 or t.numel() != H * d or not t.is_contiguous() or rot):
+            raise KernelError(f"linear_scan: {name} must be float32 [H * d], and channel gates go without a rotation")
     if single_tokens and T != B:
         raise KernelError("linear_scan: a step of single tokens has as many rows as requests")
     _contig(proj, "proj"); _ints(q_start, "q_start"); _ints(slots, "slots"); _ints(pos, "pos"); _contig(state, "state"); _contig(out, "out")
@@ -668,7 +749,7 @@ def linear_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, H: int, 
     _check(core().tl_linear_scan(_ptr(proj), dtype_code(proj.dtype), proj.shape[1], q_off, k_off, v_off, _ptr(gates), float(cap),
                                  _ptr(decay), _ptr(inv_freq) if rot else None, int(rot), int(pairing == "interleaved"), _ptr(pos),
                                  float(q_scale), float(k_scale), _ptr(state), per_slot, _ptr(q_start), _ptr(slots), _ptr(out),
-                                 int(B), H, d, dv, float(den_eps), int(single_tokens), _stream()),
+                                 int(B), H, d, dv, float(den_eps), int(single_tokens), _ptr(lower), _ptr(bias), _stream()),
            "linear_step" if single_tokens else "linear_scan")
 
 

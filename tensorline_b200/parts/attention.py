@@ -30,7 +30,12 @@ output projection.
 reads the keys of its own chunk only; the pages of chunks that lie behind are given back.  `distance_slopes` (one number a
 query head): the score of key j seen from position p loses slope * (p - j), in float32 beside the scaled product.
 `qk_norm_weight` False: the q/k norm has no weights (every head is divided by its root mean square and nothing else); the
-norm then also works over a head that is padded, taking its mean over the head's own size.
+norm then also works over a head that is padded, taking its mean over the head's own size.  (Without weights the norm and the
+rotation commute: a rotation leaves the mean of squares alone.)  `qk_norm_cast` False: the weighted norm is float32 up to the
+result, instead of a rounding to the activation type before the weight.
+
+`head_mix` (tensor `head_mix`, [query heads, query heads]): the heads' softmax weights are mixed before they meet the values
+(Shazeer et al., "Talking-Heads Attention"): head h applies sum_g mix[h, g] P_g to the values of its own KV head.
 """
 from __future__ import annotations
 
@@ -43,7 +48,7 @@ from .linear import SplitSum, matmul, resolve
 
 _NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
           "q_bias": "q_proj.bias", "k_bias": "k_proj.bias", "v_bias": "v_proj.bias",
-          "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "sink": "sink", "head_gate": "gate"}
+          "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "sink": "sink", "head_gate": "gate", "head_mix": "head_mix"}
 
 
 def _pad_heads(t: torch.Tensor, heads: int, size: int, to: int) -> torch.Tensor:
@@ -65,7 +70,8 @@ class PagedAttention(Part):
                  qkv_bias: bool, position: PartSpec, window: int | None = None, scale: float | None = None,
                  qk_norm_eps: float | None = None, v_head_dim: int | None = None, sink: bool = False,
                  names: dict | None = None, keep_first: int = 0, sink_value: float | None = None, head_gate: bool = False,
-                 chunk: int | None = None, distance_slopes=None, qk_norm_weight: bool = True):
+                 chunk: int | None = None, distance_slopes=None, qk_norm_weight: bool = True, qk_norm_cast: bool = True,
+                 head_mix: bool = False):
         super().__init__(rt)
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} query heads are not a multiple of {num_kv_heads} KV heads")
@@ -76,8 +82,9 @@ class PagedAttention(Part):
             d = -(-d // 16) * 16                          # the bfloat16 attention kernels take multiples of 16
         else:
             d += d & 1                                    # the kernel that writes the pages works on pairs of dimensions
-        if d != self.dk and qk_norm_eps is not None and qk_norm_weight:
-            raise ValueError("a weighted q/k norm over a padded head is not supported")
+        if head_mix and (window is not None or chunk is not None or sink or sink_value is not None or head_gate or distance_slopes is not None):
+            raise ValueError("heads whose weights are mixed see every earlier key, without a sink, a gate or distance slopes")
+        self.has_mix, self.qk_norm_cast = bool(head_mix), bool(qk_norm_cast)
         if chunk is not None and (window is not None or chunk < 1):
             raise ValueError("chunks are positive and stand instead of a window")
         if distance_slopes is not None and len(distance_slopes) != num_heads:
@@ -96,7 +103,7 @@ class PagedAttention(Part):
         self.qk_norm_eps = qk_norm_eps
         self.has_sink = bool(sink)
         self.names = {**_NAMES, **(names or {})}
-        self.w_qkv = self.b_qkv = self.w_o = self.q_norm = self.k_norm = self.sink = self.w_gate = None
+        self.w_qkv = self.b_qkv = self.w_o = self.q_norm = self.k_norm = self.sink = self.w_gate = self.mix = None
 
     def cache_need(self):
         return PagedKV(self.nkv, self.d, self.window, keep_first=self.keep_first, chunk=self.chunk)
@@ -115,6 +122,8 @@ class PagedAttention(Part):
             out[n["sink"]] = TensorSpec((nq,))
         if self.head_gate:
             out[n["head_gate"]] = TensorSpec((nq, H))
+        if self.has_mix:
+            out[n["head_mix"]] = TensorSpec((nq, nq))
         return out
 
     def bind(self, weights, prefix):
@@ -131,8 +140,9 @@ class PagedAttention(Part):
             w_o = _pad_heads(w_o.t().contiguous(), nq, dv, d).t()
         self.w_o = self._compute_copy(w_o)
         if self.qk_norm_eps is not None and self.qk_norm_weight:
-            self.q_norm = weights[n["q_norm"]].float().contiguous()
-            self.k_norm = weights[n["k_norm"]].float().contiguous()
+            pad = torch.ones(d - dk, dtype=torch.float32, device=self.w_o.device)        # behind the head's own size: zeros stay zeros
+            self.q_norm = torch.cat([weights[n["q_norm"]].float(), pad]).contiguous()
+            self.k_norm = torch.cat([weights[n["k_norm"]].float(), pad]).contiguous()
         elif self.qk_norm_eps is not None:
             self.q_norm = self.k_norm = torch.ones(d, dtype=torch.float32, device=self.w_o.device)
         if self.has_sink:
@@ -141,6 +151,9 @@ class PagedAttention(Part):
             self.sink = torch.full((nq,), float(self.sink_value), dtype=torch.float32, device=self.w_o.device)
         if self.head_gate:
             self.w_gate = weights[n["head_gate"]].contiguous()      # stored type; the gate's product accumulates in float32
+
+        if self.has_mix:
+            self.mix = weights[n["head_mix"]].float().contiguous()
 
     def forward(self, h, ctx, cache):
         nq, nkv, d = self.nq, self.nkv, self.d
@@ -165,13 +178,14 @@ class PagedAttention(Part):
         def rotary_kernel():
             ops.rope_kv_write(qkv, self.b_qkv, ctx.pos, ctx.req_slot, table, ctx.page_size, inv_freq, rot,
                               nq, nkv, d, cache.k, cache.v, write_kv=cache.owner, pieces=pieces, pairing=rotary.pairing,
-                              q_norm=self.q_norm, k_norm=self.k_norm, norm_eps=self.qk_norm_eps or 0.0, norm_dim=self.dk)
+                              q_norm=self.q_norm, k_norm=self.k_norm, norm_eps=self.qk_norm_eps or 0.0, norm_dim=self.dk,
+                              norm_cast=self.qk_norm_cast)
 
         # A step of single tokens whose attention kernel can do bias, rotation and the page write of its own tokens
         # (the TMA decode kernel) needs no rotary kernel in front of it.
         fold = None
         if (ctx.decode_only and not ctx.force_exact_attention and qkv.dtype == torch.bfloat16 and pieces is None and plain
-                and rot == d and self.sink is None and self._folds_rope(ctx)):
+                and rot == d and self.sink is None and self.mix is None and self._folds_rope(ctx)):
             fold = {"inv_freq": inv_freq, "bias": self.b_qkv, "write_kv": cache.owner, "unfold": rotary_kernel}
         else:
             rotary_kernel()

@@ -20,6 +20,10 @@ def attend(mixer, qkv, o, ctx, cache, table, rope=None, gate=None) -> None:
     keep_first = getattr(mixer, "keep_first", 0) if mixer.window else 0
     chunk, slopes = getattr(mixer, "chunk", None), getattr(mixer, "slopes", None)
     from .. import ops_attention
+    if getattr(mixer, "mix", None) is not None:              # the heads' weights are mixed: kernels of their own
+        ops.attn_mixed_tokenwise(qkv, qkv.shape[1], o, cache.k, cache.v, table, ctx.page_size, ctx.pos, ctx.req_slot, nq, nkv, d,
+                                 mixer.scale, mixer.mix)
+        return
     if qkv.dtype == torch.float32 or ctx.force_exact_attention or d > 256 or \
             (keep_first and not ops_attention.TAKES_KEEP_FIRST) or \
             ((chunk or slopes is not None) and not ops_attention.TAKES_CHUNKS):   # heads wider than the tensor-core kernels take

@@ -9,7 +9,7 @@ first norm (or the model's last) as `pending`.
 from __future__ import annotations
 
 from .base import FEED_FORWARDS, MIXERS, NORMS, Part, PartSpec, Runtime, register_block
-from .linear import PairSum, PostNormed, Scaled, StreamUpdate, resolve
+from .linear import PairSum, PostNormed, Scaled, StreamSum, StreamUpdate, resolve
 
 
 @register_block("pre_norm")
@@ -190,3 +190,69 @@ class HyperConnectionBlock(PreNormBlock):
             return update
         h = self.norm2.read_streams(x, update, self.hc[2]["in"])
         return StreamUpdate(self.ff.forward(h, ctx), self.hc[2]["mix"], self.hc[2]["out"])
+
+
+@register_block("shifted_pre_norm")
+class ShiftedPreNormBlock(PreNormBlock):
+    """A pre-norm block with two options, each with or without the other:
+
+        token_shift   the mixer reads h + (h' - h) * shift, h = norm1(x) and h' the previous token's h (zeros for a request's
+                      first token); tensor `shift` [hidden].  The last token's h is a state of the request.
+        layer_scale   x += ls1 * mixer(...), x += ls2 * feed_forward(...), element by element; tensors `ls1`, `ls2` [hidden]
+
+    (the token shift of RWKV: Peng et al., "RWKV: Reinventing RNNs for the Transformer Era"; layer scale: Touvron et al.,
+    "Going deeper with Image Transformers").  Sub-blocks' outputs travel as a `StreamSum`.  The norm behind a feed-forward
+    reads a row and the row in front of it, so it leaves the stream as it is; the next norm, which owns its rows, writes both
+    waiting addends at once: the stream is read twice and written once a layer."""
+
+    def __init__(self, rt: Runtime, mixer: PartSpec, feed_forward: PartSpec | None, norm1: PartSpec, norm2: PartSpec | None,
+                 token_shift: bool = True, layer_scale: bool = True, names: dict | None = None):
+        super().__init__(rt, mixer, feed_forward, norm1, norm2, {"shift": "shift", "ls1": "ls1", "ls2": "ls2", **(names or {})})
+        self.token_shift, self.layer_scale = bool(token_shift), bool(layer_scale)
+        self.shift = self.ls1 = self.ls2 = None
+
+    def _vectors(self):
+        return (["shift"] if self.token_shift else []) + (["ls1"] + (["ls2"] if self.ff is not None else []) if self.layer_scale else [])
+
+    def expected_tensors(self, prefix):
+        import dataclasses
+        from .base import TensorSpec
+        out = super().expected_tensors(prefix)
+        for v in self._vectors():
+            out[f"{prefix}.{self.names[v]}"] = TensorSpec((self.norm1.dim,), init="ones" if v != "shift" else "normal")
+        if self.layer_scale and self.ff is None:         # as the second norm: a stored one is accepted and left alone
+            out[f"{prefix}.{self.names['ls2']}"] = dataclasses.replace(out[f"{prefix}.{self.names['ls1']}"], optional=True)
+        return out
+
+    def bind(self, weights, prefix):
+        super().bind(weights, prefix)
+        for v in self._vectors():                        # they enter float32 sums
+            setattr(self, v, weights[f"{prefix}.{self.names[v]}"].float().contiguous())
+
+    def cache_need(self):
+        need = self.mixer.cache_need()
+        if not self.token_shift:
+            return need
+        from ..cache import SlotState
+        out = {"shift": SlotState((self.norm1.dim,), "float32")}
+        if isinstance(need, dict):
+            out.update({f"mixer.{k}": v for k, v in need.items()})
+        elif need is not None:
+            out["mixer"] = need
+        return out
+
+    def forward(self, x, pending, ctx, cache):
+        pending = StreamSum.of(pending)
+        if pending.full:                                 # the mixer's output is one more
+            pending = pending.write_into(x)
+        if self.token_shift:
+            h = self.norm1.sum_norm(x, pending, shift=self.shift, prev=cache["shift"].state, ctx=ctx)
+            cache = cache["mixer"] if "mixer" in cache else {k[6:]: v for k, v in cache.items() if k.startswith("mixer.")} or None
+        else:
+            h = self.norm1.sum_norm(x, pending)
+            pending = StreamSum()
+        pending = pending.plus(self.mixer.forward(h, ctx, cache), self.ls1)
+        if self.ff is None:
+            return pending
+        h = self.norm2.sum_norm(x, pending)
+        return StreamSum().plus(self.ff.forward(h, ctx), self.ls2)

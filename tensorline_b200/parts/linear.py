@@ -168,8 +168,57 @@ class StreamUpdate:
         self.mix, self.out = mix, out
 
 
+class StreamSum:
+    """Addends of the residual stream x that have not been written into it yet: x (+ base) (+ row) + sum of scale_i * value_i.
+    `items`: pairs (value [T, W] of the activation type, scale float32 [W] or None: ones); `base` float32 [T, W]; `row` float32
+    [W].  A norm that reads neighbouring rows (`RMSNorm.sum_norm` with a shift) only reads them, the next one that owns its
+    rows also writes the sum into x (`RMSNorm.sum_norm` without); whoever cannot wait calls `write_into`."""
+
+    def __init__(self, items=(), base=None, row=None):
+        self.items, self.base, self.row = tuple(items), base, row
+
+    @classmethod
+    def of(cls, pending) -> "StreamSum":
+        """Any pending addend as a sum."""
+        if pending is None:
+            return cls()
+        if isinstance(pending, cls):
+            return pending
+        if isinstance(pending, PostNormed) and pending.value is None:
+            return cls(row=pending.extra)
+        return cls(((resolve(pending), None),))
+
+    def plus(self, value, scale=None) -> "StreamSum":
+        return StreamSum(self.items + ((resolve(value), scale),), self.base, self.row)
+
+    @property
+    def full(self) -> bool:
+        return len(self.items) >= ops.SUM_ADDENDS
+
+    @property
+    def empty(self) -> bool:
+        return not self.items and self.base is None and self.row is None
+
+    def write_into(self, x: torch.Tensor) -> "StreamSum":
+        """x becomes the sum; returns the empty one."""
+        if not self.empty:
+            ops.sum_norm(x, self.items, base=self.base, row=self.row)
+        return StreamSum()
+
+
+def with_base(x: torch.Tensor, pending, base: torch.Tensor) -> StreamSum:
+    """`pending` with one more addend: the float32 rows `base` [T, W]."""
+    s = StreamSum.of(pending)
+    if s.base is not None or s.row is not None:          # the kernel takes one of each, in this order in front of the addends
+        s = s.write_into(x)
+    return StreamSum(s.items, base, None)
+
+
 def with_row(x: torch.Tensor, pending, row: torch.Tensor, eps: float):
     """`pending` with one more addend: the float32 vector `row`, added once to every row of the stream x."""
+    if isinstance(pending, StreamSum):
+        s = pending.write_into(x) if pending.row is not None else pending
+        return StreamSum(s.items, s.base, row)
     if pending is None:
         return PostNormed(None, None, eps, extra=row)
     if isinstance(pending, PostNormed) and pending.extra is None:
@@ -192,6 +241,8 @@ def resolve(t):
         return (t.a.float() + t.b.float()).to(t.dtype)
     if isinstance(t, WeightedPair):
         return (t.a.float() * t.alpha + t.b.float() * t.beta).to(t.dtype)
+    if isinstance(t, StreamSum):
+        raise TypeError("a sum over the residual stream has no value of its own: the next norm writes it")
     if isinstance(t, StreamUpdate):
         raise TypeError("an update of several stream copies has no value of its own: the next norm applies it")
     if isinstance(t, PendingProduct):                    # whoever asks for the tensor itself has no use for split-K pieces:

@@ -1,4 +1,6 @@
-"""Dense gated feed-forward: y = (act(h Wg^T) * (h Wu^T)) Wd^T, act = silu or the tanh form of gelu, no biases.
+"""Dense feed-forwards: gated (`gated_mlp`) and with one matrix in front of the activation (`plain_mlp`, at the end).
+
+Dense gated feed-forward: y = (act(h Wg^T) * (h Wu^T)) Wd^T, act = silu or the tanh form of gelu, no biases.
 A third activation, `swish_clamped`, works on the pair: with g' = min(g, limit) and u' = clamp(u, -limit, limit) the unit
 is g' sigmoid(alpha g') (u' + 1); `act_limit` and `act_alpha` are its constants.
 
@@ -13,7 +15,7 @@ import torch
 
 from .. import ops
 from .base import Part, Runtime, TensorSpec, register_feed_forward
-from .linear import NormedInput, matmul, use_pair_product, use_tc
+from .linear import NormedInput, matmul, resolve, use_pair_product, use_tc
 
 GATE_BLOCK = 64
 
@@ -73,4 +75,32 @@ class GatedMLP(Part):
         gu = matmul(h, self.w_gate_up)
         m = torch.empty((h.shape[0], I), dtype=h.dtype, device=h.device)
         ops.silu_mul(gu, m, block=self.block, act=self.gate)
+        return matmul(m, self.w_down, may_defer=True, to_residual=True)          # the next norm adds it up
+
+
+@register_feed_forward("plain_mlp")
+class PlainMLP(Part):
+    """y = act(h Wu^T) Wd^T, no gate and no biases; act = the square of relu (`relu_squared`)."""
+    graph_capturable = True
+
+    def __init__(self, rt: Runtime, hidden: int, intermediate: int, activation: str = "relu_squared", names: dict | None = None):
+        """`names`: the two tensors' names under the part's prefix (keys up, down)."""
+        super().__init__(rt)
+        if activation != "relu_squared":
+            raise ValueError(f"plain_mlp runs 'relu_squared', not {activation!r}")
+        self.hidden, self.intermediate, self.activation = hidden, intermediate, activation
+        self.names = {"up": "up_proj.weight", "down": "down_proj.weight", **(names or {})}
+        self.w_up = self.w_down = None
+
+    def expected_tensors(self, prefix):
+        H, I, n = self.hidden, self.intermediate, self.names
+        return {f"{prefix}.{n['up']}": TensorSpec((I, H)), f"{prefix}.{n['down']}": TensorSpec((H, I))}
+
+    def bind(self, weights, prefix):
+        self.w_up = self._compute_copy(weights[f"{prefix}.{self.names['up']}"])
+        self.w_down = self._compute_copy(weights[f"{prefix}.{self.names['down']}"])
+
+    def forward(self, h, ctx):
+        m = resolve(matmul(h, self.w_up))
+        ops.relu_square(m)
         return matmul(m, self.w_down, may_defer=True, to_residual=True)          # the next norm adds it up

@@ -5,7 +5,7 @@ import torch
 
 from .. import ops
 from .base import Part, Runtime, TensorSpec, register_norm, tensor_name
-from .linear import FUSE_NORMS, NormedInput, PairSum, PendingProduct, PostNormed, Scaled, SplitSum, StreamUpdate, WeightedPair, resolve
+from .linear import FUSE_NORMS, NormedInput, PairSum, PendingProduct, PostNormed, Scaled, SplitSum, StreamSum, StreamUpdate, WeightedPair, resolve
 
 
 @register_norm("rms_norm")
@@ -74,11 +74,28 @@ class RMSNorm(Part):
         ops.stream_step(x, S, read=read, w=self.weight, eps=self.eps, h=h, rows=rows, **kw)
         return h
 
+    def sum_norm(self, x, pending: StreamSum, rows=None, shift=None, prev=None, ctx=None):
+        """The norm of x with every addend of `pending`, float32 up to the rounding of the result.  Without `rows` and `shift`
+        the sum is written into x.  `shift` (float32 [dim]): the result is n + (n' - n) * shift with n' the normed row of the
+        request's token in front, kept across steps in `prev` (float32 [slots, dim]); x is then only read."""
+        if self.cast_first or self.one_plus:
+            raise NotImplementedError("a stream with waiting addends is read by plain float32 norms")
+        n = x.shape[0] if rows is None else rows.numel()
+        h = torch.empty((n, self.dim), dtype=self.rt.act_dtype, device=x.device)
+        ops.sum_norm(x, pending.items, base=pending.base, row=pending.row, w=self.weight, eps=self.eps, h=h, rows=rows, shift=shift,
+                     prev=prev, ctx=ctx)
+        return h
+
     def add_norm(self, x, pending, rows=None, defer=False):
         """`defer`: the caller's next step is a product that takes a `NormedInput`."""
         n = x.shape[0] if rows is None else rows.numel()
         if isinstance(pending, StreamUpdate) or x.shape[1] != self.dim:       # several copies: their sum is what this norm reads
             return self.read_streams(x, pending, None, rows=rows)
+        if isinstance(pending, StreamSum):
+            if not (self.cast_first or self.one_plus):
+                return self.sum_norm(x, pending, rows=rows)
+            pending.write_into(x)
+            pending = None
         if isinstance(pending, WeightedPair):
             pending = resolve(pending)
         if isinstance(pending, PairSum):

@@ -2,7 +2,7 @@
 
     S_t = a_t S_(t-1) + b_t k_t v_t^T,    o_t = S_t^T q_t          S: [d, dv] per head, float32
 
-Two kinds, one pipeline (one stacked projection, one scan kernel, one kernel for the per-head norm and the
+Three kinds, one pipeline (one stacked projection, one scan kernel, one kernel for the per-head norm and the
 gate, the output projection):
 
 * `retention`: a_t is a fixed decay per head, b_t = 1; q and k are rotated by position and k is scaled by
@@ -14,6 +14,11 @@ gate, the output projection):
   a_t = exp(f_t + m_(t-1) - m_t), b_t = exp(i_t - m_t); a normaliser n_t follows the same recurrence with k
   alone, and o_t = S_t^T q_t / (max(|n_t . q_t|, exp(-m_t)) + 1e-6) with q scaled by d^-1/2.  Every head's o
   is divided by its root mean square, multiplied by a weight over all heads, by sigmoid(g), and projected.
+
+* `hgrn2` (Qin et al., "HGRN2: Gated Linear RNNs with State Expansion"): the forget gate decides what is written and there is
+  no key: f = l + (1 - l) sigmoid(W_f x + b_f) per head and channel with a stored lower bound l, q = silu(W_q x),
+  S_t = diag(f_t) S_(t-1) + (1 - f_t) v_t^T; every head's o is divided by its root mean square, multiplied by a weight that
+  the heads share, and projected.
 
 The state lives in the request's state slot (`SlotState`), in float32, zero for a new request (which is also
 m_0 = 0), in the scan kernel's own layout; the gates' pre-activations, the rotation, the exponentials and the
@@ -158,3 +163,41 @@ class MLSTM(_MatrixState):
         ops.small_proj(h, self.w_gates, self.b_gates, gates)
         ops.linear_scan(proj, 0, H * d, 2 * H * d, H, d, dv, state, ctx.q_start, ctx.slots, ctx.pos, o, B=ctx.B,
                         gates=gates, cap=self.cap, q_scale=d ** -0.5, den_eps=self.den_eps, single_tokens=ctx.decode_only)
+
+
+@register_mixer("hgrn2")
+class HGRN2(_MatrixState):
+    def __init__(self, rt: Runtime, hidden: int, num_heads: int, head_dim: int, v_head_dim: int, norm_eps: float,
+                 names: dict | None = None):
+        super().__init__(rt, hidden, num_heads, head_dim, v_head_dim, norm_eps, None,
+                         {"f": "f", "f_bias": "f.b", "lower": "lower", "norm": "norm", **(names or {})})
+        self.f_bias = self.lower = self.head_weight = None
+
+    def _projections(self):
+        H, d, dv = self.H, self.d, self.dv
+        return (("q", H * d), ("f", H * d), ("v", H * dv))
+
+    def expected_tensors(self, prefix):
+        n, H = self.names, self.H
+        out = super().expected_tensors(prefix)
+        out.update({f"{prefix}.{n['f_bias']}": TensorSpec((H * self.d,)), f"{prefix}.{n['lower']}": TensorSpec((H * self.d,)),
+                    f"{prefix}.{n['norm']}": TensorSpec((self.dv,), init="ones")})
+        return out
+
+    def bind(self, weights, prefix):
+        super().bind(weights, prefix)
+        n = self.names
+        self.f_bias = weights[f"{prefix}.{n['f_bias']}"].float().contiguous()        # they enter float32 gates
+        self.lower = weights[f"{prefix}.{n['lower']}"].float().contiguous()
+        self.head_weight = weights[f"{prefix}.{n['norm']}"].repeat(self.H).contiguous()
+
+    def forward(self, h, ctx, cache):
+        H, d, dv = self.H, self.d, self.dv
+        T = h.shape[0]
+        proj = resolve(matmul(h, self.w_in, out_dtype=torch.float32))            # q | f | v, as the product accumulated them
+        o = torch.empty((T, H * dv), dtype=torch.float32, device=h.device)
+        ops.linear_scan(proj, 0, H * d, 2 * H * d, H, d, dv, cache.state, ctx.q_start, ctx.slots, ctx.pos, o, B=ctx.B,
+                        lower=self.lower, bias=self.f_bias, single_tokens=ctx.decode_only)
+        y = torch.empty((T, H * dv), dtype=h.dtype, device=h.device)
+        ops.head_norm_gate(o, y, H, dv, self.eps, weight=self.head_weight)
+        return matmul(y, self.w_o)
