@@ -80,6 +80,8 @@ class PagedAttention(Part):
         d = max(self.dk, self.dv)
         if not rt.exact:
             d = -(-d // 16) * 16                          # the bfloat16 attention kernels take multiples of 16
+            if head_mix and d <= 256:
+                d = -(-d // 64) * 64                      # those of mixed heads multiples of 64
         else:
             d += d & 1                                    # the kernel that writes the pages works on pairs of dimensions
         if head_mix and (window is not None or chunk is not None or sink or sink_value is not None or head_gate or distance_slopes is not None):
@@ -103,7 +105,7 @@ class PagedAttention(Part):
         self.qk_norm_eps = qk_norm_eps
         self.has_sink = bool(sink)
         self.names = {**_NAMES, **(names or {})}
-        self.w_qkv = self.b_qkv = self.w_o = self.q_norm = self.k_norm = self.sink = self.w_gate = self.mix = None
+        self.w_qkv = self.b_qkv = self.w_o = self.q_norm = self.k_norm = self.sink = self.w_gate = self.mix = self.mix_pad = None
 
     def cache_need(self):
         return PagedKV(self.nkv, self.d, self.window, keep_first=self.keep_first, chunk=self.chunk)
@@ -153,7 +155,11 @@ class PagedAttention(Part):
             self.w_gate = weights[n["head_gate"]].contiguous()      # stored type; the gate's product accumulates in float32
 
         if self.has_mix:
-            self.mix = weights[n["head_mix"]].float().contiguous()
+            mix = weights[n["head_mix"]]
+            self.mix = mix.float().contiguous()
+            if not self.rt.exact and mix.dtype == torch.bfloat16:        # exact in bfloat16: what the tensor-core kernels take
+                from .. import ops_attention_mix
+                self.mix_pad = ops_attention_mix.pad_mix(mix)
 
     def forward(self, h, ctx, cache):
         nq, nkv, d = self.nq, self.nkv, self.d

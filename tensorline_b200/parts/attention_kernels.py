@@ -19,8 +19,12 @@ def attend(mixer, qkv, o, ctx, cache, table, rope=None, gate=None) -> None:
     sink = getattr(mixer, "sink", None)
     keep_first = getattr(mixer, "keep_first", 0) if mixer.window else 0
     chunk, slopes = getattr(mixer, "chunk", None), getattr(mixer, "slopes", None)
-    from .. import ops_attention
+    from .. import ops_attention, ops_attention_mix
     if getattr(mixer, "mix", None) is not None:              # the heads' weights are mixed: kernels of their own
+        if mixer.mix_pad is not None and qkv.dtype == torch.bfloat16 and not ctx.force_exact_attention and \
+                ops_attention_mix.takes(nq, d, ctx.page_size, mixer.mix_pad.dtype):
+            ops_attention_mix.attend(qkv, o, ctx, cache.k, cache.v, table, nq, nkv, d, mixer.scale, mixer.mix_pad)
+            return
         ops.attn_mixed_tokenwise(qkv, qkv.shape[1], o, cache.k, cache.v, table, ctx.page_size, ctx.pos, ctx.req_slot, nq, nkv, d,
                                  mixer.scale, mixer.mix)
         return
