@@ -624,6 +624,22 @@ def _tenalorn_sizes(z):
             "layers": [order[i % 4] for i in range(z["layers"])]}
 
 
+def _zosurax_sizes(z):
+    """Four layer runs: HGRN2 twice (one set of weights, a loop of two passes with the embedding added again), attention with
+    weighted q/k norms, attention with mixed softmax weights; token shift and layer scales in every layer, a plain feed-forward
+    with as many active weights a token as the routed one of the other arm."""
+    mlp = {"kind": "dense", "ff": z["top"] * z["ff"]}
+    rec = {"type": "hgrn2", "mlp": mlp, "mixer": {"heads": z["rec_heads"], "dim": z["rec_dim"], "vdim": z["rec_vdim"]}}
+
+    def attention(kind, dims):
+        return {"type": kind, "mlp": mlp, "mixer": {
+            "heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["head"], "vdim": z["head"], "scale": z["head"] ** -0.5,
+            "rot": {"base": 500000.0, "dims": dims}}}
+    return {"architecture": "Zosurax", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5},
+            "loop": {"start": 0, "stop": 1, "times": max(1, z["layers"] - 2)},
+            "layers": [rec, attention("attention", z["head"] // 2), attention("attention_2", z["head"])]}
+
+
 def run_design(a):
     import torch
     from tensorline_b200 import Engine, Qwen2Config
@@ -631,6 +647,7 @@ def run_design(a):
     from tensorline_b200.config.sumuvik import SumuvikConfig
     from tensorline_b200.config.tenalorn import TenalornConfig
     from tensorline_b200.config.vutesun import VutesunConfig
+    from tensorline_b200.config.zosurax import ZosuraxConfig
     if not torch.cuda.is_available():
         print(json.dumps({"impl": "ours", "error": "no CUDA device: this engine runs on the GPU only"}))
         return 1
@@ -651,6 +668,8 @@ def run_design(a):
             arms = {"sumuvik": SumuvikConfig.from_dict(_sumuvik_sizes(z)), "dekerax": DekeraxConfig.from_dict(_dekerax_sizes(z))}
         if a.design == "tenalorn":                                       # its closest: a pair of mixers, the matrix memory, routed experts
             arms = {"tenalorn": TenalornConfig.from_dict(_tenalorn_sizes(z)), "vutesun": arms["vutesun"]}
+        if a.design == "zosurax":                                        # its closest: a matrix memory in the scan kernel, rotated attention
+            arms = {"zosurax": ZosuraxConfig.from_dict(_zosurax_sizes(z)), "vutesun": arms["vutesun"]}
         out[tag] = {"sizes": dict(z, dense_intermediate=dense)}
         for name, cfg in arms.items():
             weights = random_weights(cfg, device)
@@ -674,7 +693,7 @@ def run_design(a):
             import gc
             gc.collect(); torch.cuda.empty_cache()
     first = out[sorted(out)[0]]
-    beside = {"vutesun": "Qwen2", "dekerax": "Vutesun", "sumuvik": "Dekerax", "tenalorn": "Vutesun"}[a.design]
+    beside = {"vutesun": "Qwen2", "dekerax": "Vutesun", "sumuvik": "Dekerax", "tenalorn": "Vutesun", "zosurax": "Vutesun"}[a.design]
     print(json.dumps({"metric": f"decode tok/s of the {a.design.capitalize()} decoder beside {beside} at equal layer sizes (bf16, batch {batch}, context {context})",
                       "value": first[a.design][f"decode_b{batch}_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": K, "warmup": W,
                       "ms_per_step": first[a.design][f"decode_b{batch}_ms"], "higher_is_better": True, "scaling": "weak",
@@ -713,9 +732,9 @@ def main(argv=None):
     ap.add_argument("--timeline", action="store_true",
                     help="print the time line of one captured decode step from the kernels' own stamps (needs TENSORLINE_B200_TRACE=1)")
     ap.add_argument("--no-warm-mix", dest="warm_mix", action="store_false", help="mix: time the first pass (graph capture included)")
-    ap.add_argument("--design", choices=["vutesun", "dekerax", "sumuvik", "tenalorn"], default=None,
+    ap.add_argument("--design", choices=["vutesun", "dekerax", "sumuvik", "tenalorn", "zosurax"], default=None,
                     help="instead of the default workload: this design beside the closest other one at equal layer sizes "
-                         "(vutesun beside Qwen2, dekerax beside vutesun, sumuvik beside dekerax, tenalorn beside vutesun; "
+                         "(vutesun beside Qwen2, dekerax beside vutesun, sumuvik beside dekerax, tenalorn beside vutesun, zosurax beside vutesun; "
                          "prefill, decode, --profile)")
     ap.add_argument("--design-size", default="", help="--design: which of the sizes (2k, 4k; commas between them; default all)")
     a = ap.parse_args(argv)

@@ -222,7 +222,7 @@ def test_attention_with_mixed_weights(case, kernel):
     num_pages = max(300, B * max_pages)
     kps = torch.full((num_pages + 1, nkv, ps, d), 37.0, dtype=adt)
     vps = torch.full_like(kps, -53.0)
-    mix = (torch.eye(nq) + rnd(nq, nq, seed=9, scale=0.4)).to(torch.bfloat16)
+    mix = (torch.eye(nq) + rnd(nq, nq, seed=9, scale=1.2 * nq ** -0.5)).to(torch.bfloat16)
     rows, qs, want, pos_all, slot_all = [], [], [], [], []
     for b in range(B):
         n = ctx_lens[b] + step_lens[b]
