@@ -45,22 +45,46 @@ struct MixArgs {
     int nq, nkv;
     float scale_log2;
     const int4* tiles; int n_tiles;      // row tiles: (request, tile of 128 rows, first unit in the scratch, key tiles)
+    const int2* parts; int n_parts;      // runs of a row tile's key tiles, a block of the scores each: (row tile, number of the run)
     const int* unit_tile; int n_units;   // unit (row tile x key tile) -> its row tile
     float* scores;                       // [units][nq][128][64]
-    float* lse;                          // [T][nq]  log2 of the denominator, in the scores' scaled units
+    float2* part_ml;                     // [T][nq][MAX_PARTS]  maximum and sum of each run, in the scores' scaled base-2 units
+    float* lse;                          // [T][nq]  log2 of the denominator
     bf16* mixed;                         // [units][nq][128][64]
     const bf16* mix; int hp;             // [hp][hp], nq padded with zeros to a multiple of 16
     int* status;
     TlLimits lim;
 };
 
-// Copy of keys [key0, key0 + 64) of one KV head into a swizzled [64][D] tile; the calling threads are number `part` of
-// `parts` lanes; keys past last_key are zeros.
+// A row tile's key tiles are dealt out to several blocks of the scores kernel, in runs of eight or of a sixteenth of them.
+constexpr int MAX_PARTS = 16;
+__host__ __device__ __forceinline__ int part_tiles(int n_kt) { return n_kt > 8 * MAX_PARTS ? (n_kt + MAX_PARTS - 1) / MAX_PARTS : 8; }
+
+// Keys [key0, key0 + 64) of one KV head as TMA boxes (a page, 64 elements wide), by one thread: pages of 8 tokens or more.
+__device__ __forceinline__ void pages_of(int (&page)[8], const int* tab, int max_pages, int ps_shift, int key0, const TlLimits& L) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+        if (i < (BN >> ps_shift)) page[i] = tl_checked(tab[min((key0 >> ps_shift) + i, max_pages - 1)], L.total_pages, L, TL_K_TC_PREFILL);
+}
+__device__ __forceinline__ void fetch_keys(uint32_t dst, const CUtensorMap* map, uint64_t* bar, const int (&page)[8], int ps_shift, int nkv, int kh) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+        if (i >= (BN >> ps_shift)) break;
+#pragma unroll
+        for (int db = 0; db < D / 64; ++db)
+            tma_box(dst + db * (BN * 128) + ((i << ps_shift) * 128), map, bar, db * 64, (page[i] * nkv + kh) << ps_shift);
+    }
+}
+
+// Copy of keys [key0, key0 + 64) of one KV head into a swizzled [64][D] tile; the calling thread is number `part` of PARTS;
+// keys past last_key are zeros.
+template <int PARTS>
 __device__ __forceinline__ void copy_keys(uint32_t dst, const bf16* pages, const int* tab, int ps_shift, size_t page_stride, int key0,
-                                          int last_key, int part, int parts, const TlLimits& L) {
+                                          int last_key, int part, const TlLimits& L) {
     const int ps_mask = (1 << ps_shift) - 1;
-    for (int idx = part; idx < BN * CH; idx += parts) {
-        const int key = idx / CH, c = idx - key * CH;
+#pragma unroll 8
+    for (int i = 0; i < BN * CH / PARTS; ++i) {
+        const int idx = part + i * PARTS, key = idx / CH, c = idx - key * CH;
         const bool valid = key0 + key <= last_key;
         const int page = valid ? tl_checked(tab[(key0 + key) >> ps_shift], L.total_pages, L, TL_K_TC_PREFILL) : 0;
         const bf16* src = pages + (size_t)page * page_stride + (size_t)((key & ps_mask) * D + c * 8);
@@ -68,10 +92,6 @@ __device__ __forceinline__ void copy_keys(uint32_t dst, const bf16* pages, const
     }
 }
 __device__ __forceinline__ int shift_of(int page_size) { int s = 0; while ((1 << s) < page_size) ++s; return s; }
-__device__ __forceinline__ void named_sync(int id, int threads) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
-__device__ __forceinline__ void expect_tx(uint64_t* bar, uint32_t bytes) {
-    asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(smem_addr(bar)), "r"(bytes) : "memory");
-}
 __device__ __forceinline__ void bulk_load(uint32_t dst, const void* src, uint32_t bytes, uint64_t* bar) {
     asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
                  ::"r"(dst), "l"(src), "r"(bytes), "r"(smem_addr(bar)) : "memory");
@@ -83,13 +103,15 @@ __device__ __forceinline__ void bulk_store(void* dst, uint32_t src, uint32_t byt
 
 // ------------------------------------------------------------------------------------------------ prompts: scores
 // Warps 0..3: one row a thread (scores out of tensor memory, mask, running maximum and sum, the tile to scratch through
-// shared memory); warp 4: MMA issue; warps 5, 6: copies of K, every other tile each.
+// shared memory); warp 4: MMA issue; warps 5, 6: K, by TMA (warp 5) or by asynchronous copies, every other tile each.
 constexpr int S_THREADS = 224;
-constexpr int SS_TILES = Q_BYTES + 2 * K_BYTES + 2 * S_BYTES;
+constexpr int SS_TILES = Q_BYTES + 2 * K_BYTES + S_BYTES;          // two blocks an SM up to head size 128
 constexpr int SS_SMEM = SS_TILES + 1024 + 128;
 constexpr uint32_t SS_COLS = 128;        // two score slots of 64 columns
 
-__global__ void __launch_bounds__(S_THREADS, 1) mix_scores_kernel(const MixArgs A) {
+template <bool TMA>
+__global__ void __launch_bounds__(S_THREADS, D <= 128 ? 2 : 1)
+mix_scores_kernel(const __grid_constant__ CUtensorMap map_k, const MixArgs A) {
     extern __shared__ unsigned char smem_raw[];
     unsigned char* base = reinterpret_cast<unsigned char*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
     const uint32_t sQ = smem_addr(base), sK = sQ + Q_BYTES, sS = sK + 2 * K_BYTES;
@@ -102,8 +124,9 @@ __global__ void __launch_bounds__(S_THREADS, 1) mix_scores_kernel(const MixArgs 
     volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int h = blockIdx.x % A.nq, kh = h / (A.nq / A.nkv);
-    const int4 tl = A.tiles[blockIdx.x / A.nq];
-    const int b = tl.x, row0 = tl.y * BM, n_kt = tl.w;
+    const int2 pt = A.parts[blockIdx.x / A.nq];
+    const int4 tl = A.tiles[pt.x];
+    const int b = tl.x, row0 = tl.y * BM, kt0 = pt.y * part_tiles(tl.w), n_kt = min(part_tiles(tl.w), tl.w - kt0);
     const int qs = A.q_start[b], qlen = A.q_start[b + 1] - qs, sp = A.start_pos[b];
     const int row_end = min(row0 + BM, qlen), pos_hi = sp + row_end - 1;
     const int* tab = A.table + (size_t)tl_checked(A.slots[b], A.lim.table_rows, A.lim, TL_K_TC_PREFILL) * A.max_pages;
@@ -111,7 +134,7 @@ __global__ void __launch_bounds__(S_THREADS, 1) mix_scores_kernel(const MixArgs 
 
     if (tid == 0) {
         mbar_init(bar_q, BM);
-        for (int i = 0; i < 2; ++i) { mbar_init(bar_k + i, 32); mbar_init(bar_s + i, 1); mbar_init(bar_f + i, BM); }
+        for (int i = 0; i < 2; ++i) { mbar_init(bar_k + i, TMA ? 1 : 32); mbar_init(bar_s + i, 1); mbar_init(bar_f + i, BM); }
         *abort_flag = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
@@ -139,7 +162,6 @@ __global__ void __launch_bounds__(S_THREADS, 1) mix_scores_kernel(const MixArgs 
         bool ok = true;
         for (int i = 0; i < n_kt; ++i) {
             const int sl = i & 1;
-            // every thread of the four warps passes the same number of named barriers, whatever a wait did
             if (ok) ok = mbar_wait(bar_s + sl, (i >> 1) & 1, abort_flag, A.status, 41);
             float s[BN];
             if (__all_sync(0xffffffffu, ok)) {
@@ -156,9 +178,10 @@ __global__ void __launch_bounds__(S_THREADS, 1) mix_scores_kernel(const MixArgs 
             }
 #pragma unroll
             for (int c = 0; c < BN; ++c) s[c] *= A.scale_log2;
-            if (i * BN + BN - 1 > pos_r) {
+            const int key0 = (kt0 + i) * BN;
+            if (key0 + BN - 1 > pos_r) {
 #pragma unroll
-                for (int c = 0; c < BN; ++c) if (i * BN + c > pos_r) s[c] = -INFINITY;
+                for (int c = 0; c < BN; ++c) if (key0 + c > pos_r) s[c] = -INFINITY;
             }
             const float mx = row_max(s);
             const float m_new = fmaxf(m, mx), m_use = m_new == -INFINITY ? 0.f : m_new;
@@ -167,18 +190,19 @@ __global__ void __launch_bounds__(S_THREADS, 1) mix_scores_kernel(const MixArgs 
             for (int c = 0; c < BN; ++c) l4[c & 3] += fast_exp2(s[c] - m_use);
             l = l * fast_exp2(m - m_use) + ((l4[0] + l4[1]) + (l4[2] + l4[3]));
             m = m_new;
-            if (tid == 0) asm volatile("cp.async.bulk.wait_group.read 1;" ::: "memory");      // the slot's store before last has read it
-            named_sync(1, BM);
+            // a warp's 32 rows are 8 KB in a row of the tile's image: it stages and stores them by itself
+            if (lane == 0) asm volatile("cp.async.bulk.wait_group.read 0;" ::: "memory");     // its last store has read the place
+            __syncwarp();
 #pragma unroll
             for (int c = 0; c < BN / 4; ++c)
-                asm volatile("st.shared.v4.f32 [%0], {%1, %2, %3, %4};" ::"r"(sS + sl * S_BYTES + tid * 256 + ((c ^ (tid & 7)) << 4)),
+                asm volatile("st.shared.v4.f32 [%0], {%1, %2, %3, %4};" ::"r"(sS + tid * 256 + ((c ^ (tid & 7)) << 4)),
                              "f"(s[4 * c]), "f"(s[4 * c + 1]), "f"(s[4 * c + 2]), "f"(s[4 * c + 3]) : "memory");
             fence_async_proxy();
-            named_sync(1, BM);
-            if (tid == 0) bulk_store(A.scores + ((size_t)(tl.z + i) * A.nq + h) * (BM * BN), sS + sl * S_BYTES, S_BYTES);
+            __syncwarp();
+            if (lane == 0) bulk_store(A.scores + ((size_t)(tl.z + kt0 + i) * A.nq + h) * (BM * BN) + warp * (32 * BN), sS + warp * (32 * BN * 4), 32 * BN * 4);
         }
-        if (R < qlen) A.lse[(size_t)(qs + R) * A.nq + h] = m + log2f(l);
-        if (tid == 0) asm volatile("cp.async.bulk.wait_group 0;" ::: "memory");
+        if (R < qlen) A.part_ml[((size_t)(qs + R) * A.nq + h) * MAX_PARTS + pt.y] = make_float2(m, l);
+        if (lane == 0) asm volatile("cp.async.bulk.wait_group 0;" ::: "memory");
     } else if (warp == 4) {
         if (lane == 0) {
             constexpr uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(BN >> 3) << 17) | ((uint32_t)(BM >> 4) << 24);
@@ -202,11 +226,29 @@ __global__ void __launch_bounds__(S_THREADS, 1) mix_scores_kernel(const MixArgs 
         const size_t page_stride = (size_t)A.nkv * A.page_size * D;
         const bf16* pages = A.k_pages + (size_t)kh * A.page_size * D;
         bool ok = true;
-        for (int j = warp - 5; j < n_kt && ok; j += 2) {
+        if (TMA) {
+            if (warp == 5 && lane == 0) {
+                asm volatile("prefetch.tensormap [%0];" ::"l"(&map_k) : "memory");
+                int j = 0;
+                for (; j < n_kt && ok; ++j) {
+                    const int sl = j & 1;
+                    int page[8];
+                    pages_of(page, tab, A.max_pages, ps_shift, (kt0 + j) * BN, A.lim);       // asked for before the wait
+                    if (j >= 2) ok = mbar_wait(bar_s + sl, ((j - 2) >> 1) & 1, abort_flag, A.status, 45, true);
+                    if (!ok) break;
+                    mbar_expect_tx(bar_k + sl, K_BYTES);
+                    fetch_keys(sK + sl * K_BYTES, &map_k, bar_k + sl, page, ps_shift, A.nkv, kh);
+                }
+                for (int i = max(0, j - 2); !ok && i < j; ++i) {         // a block that gives up waits (bounded) for its own copies
+                    const long long t0 = clock64();
+                    while (!mbar_try_wait(bar_k + (i & 1), (i >> 1) & 1) && clock64() - t0 < 2000000LL) { }
+                }
+            }
+        } else for (int j = warp - 5; j < n_kt && ok; j += 2) {
             const int sl = j & 1;
             if (j >= 2) ok = mbar_wait(bar_s + sl, ((j - 2) >> 1) & 1, abort_flag, A.status, 45, true);
             if (!ok) break;
-            copy_keys(sK + sl * K_BYTES, pages, tab, ps_shift, page_stride, j * BN, pos_hi, lane, 32, A.lim);
+            copy_keys<32>(sK + sl * K_BYTES, pages, tab, ps_shift, page_stride, (kt0 + j) * BN, pos_hi, lane, A.lim);
             cp_async_wait_all();
             fence_async_proxy();
             mbar_arrive(bar_k + sl);
@@ -241,11 +283,14 @@ __device__ __forceinline__ void split3(float x, float y, uint32_t (&o)[3]) {
 }
 
 // One row's P' over 32 keys by one warp.  Lane (n = lane / 4, c = lane % 4) reads, for the heads 2c, 2c + 1, 2c + 8, 2c + 9 of
-// a group of 16, the scores of keys 4n .. 4n + 3 (`load(g)` -> float4) and makes their weights exp2(s - L_g); product e of four
-// takes key 4n + e as its column n, so the lane's results are keys 8c .. 8c + 7 of the heads lane / 4 and lane / 4 + 8 of every
-// 16: acc[m][e][0..1] (keys 8c + e, 8c + 4 + e) and acc[m][e][2..3].  `live` = number of the 32 keys that are visible.
-template <int MT, typename Load, typename Lse>
-__device__ __forceinline__ void mix_row(float (&acc)[MT][4][4], const bf16* mix, int hp, int nq, int lane, int live, Load load, Lse lse) {
+// every 16, the scores of keys 4n .. 4n + 3 (`load(g)` -> float4) and makes their weights exp2(s - L_g), L[t][..] of group t;
+// product e of four takes key 4n + e as its column n, so the lane's results are keys 8c .. 8c + 7 of the heads lane / 4 and
+// lane / 4 + 8 of every 16: acc[m][e][0..1] (keys 8c + e, 8c + 4 + e) and acc[m][e][2..3].  `live` = number of the 32 keys that
+// are visible.
+__device__ __forceinline__ int mix_head(int t, int k, int c) { return t * 16 + 2 * c + (k & 1) + (k >> 1) * 8; }
+
+template <int MT, typename Load>
+__device__ __forceinline__ void mix_row(float (&acc)[MT][4][4], const bf16* mix, int hp, int nq, int lane, int live, const float (&L)[MT][4], Load load) {
     const int n = lane >> 2, c = lane & 3;
 #pragma unroll
     for (int m = 0; m < MT; ++m)
@@ -253,16 +298,22 @@ __device__ __forceinline__ void mix_row(float (&acc)[MT][4][4], const bf16* mix,
         for (int e = 0; e < 4; ++e)
 #pragma unroll
             for (int k = 0; k < 4; ++k) acc[m][e][k] = 0.f;
-    for (int g0 = 0; g0 < nq; g0 += 16) {
+#pragma unroll
+    for (int t = 0; t < MT; ++t) {
         float p[4][4];                                       // [head of the lane][key e]
 #pragma unroll
         for (int k = 0; k < 4; ++k) {
-            const int g = g0 + 2 * c + (k & 1) + (k >> 1) * 8;
+            const int g = mix_head(t, k, c);
             float4 s = make_float4(-INFINITY, -INFINITY, -INFINITY, -INFINITY);
-            float L = 0.f;
-            if (g < nq) { s = load(g); L = lse(g); }
-            p[k][0] = 4 * n < live ? fast_exp2(s.x - L) : 0.f;     p[k][1] = 4 * n + 1 < live ? fast_exp2(s.y - L) : 0.f;
-            p[k][2] = 4 * n + 2 < live ? fast_exp2(s.z - L) : 0.f; p[k][3] = 4 * n + 3 < live ? fast_exp2(s.w - L) : 0.f;
+            if (g < nq) s = load(g);
+            p[k][0] = fast_exp2(s.x - L[t][k]); p[k][1] = fast_exp2(s.y - L[t][k]);
+            p[k][2] = fast_exp2(s.z - L[t][k]); p[k][3] = fast_exp2(s.w - L[t][k]);
+        }
+        if (live < 32) {
+#pragma unroll
+            for (int k = 0; k < 4; ++k)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) if (4 * n + e >= live) p[k][e] = 0.f;
         }
         uint32_t b0[4][3], b1[4][3];
 #pragma unroll
@@ -270,7 +321,7 @@ __device__ __forceinline__ void mix_row(float (&acc)[MT][4][4], const bf16* mix,
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
             uint32_t a[4];
-            const bf16* w = mix + (size_t)(m * 16 + n) * hp + g0 + 2 * c;
+            const bf16* w = mix + (size_t)(m * 16 + n) * hp + t * 16 + 2 * c;
             a[0] = *reinterpret_cast<const uint32_t*>(w);     a[1] = *reinterpret_cast<const uint32_t*>(w + 8 * hp);
             a[2] = *reinterpret_cast<const uint32_t*>(w + 8); a[3] = *reinterpret_cast<const uint32_t*>(w + 8 * hp + 8);
 #pragma unroll
@@ -281,69 +332,130 @@ __device__ __forceinline__ void mix_row(float (&acc)[MT][4][4], const bf16* mix,
     }
 }
 
-constexpr int MIX_ROWS = 4;              // rows a warp
+// L of every (row, head) of the row tiles from its runs, in their order.
+__global__ void __launch_bounds__(256) mix_lse_kernel(const MixArgs A) {
+    const int4 tl = A.tiles[blockIdx.x];
+    const int qs = A.q_start[tl.x], qlen = A.q_start[tl.x + 1] - qs, np = (tl.w + part_tiles(tl.w) - 1) / part_tiles(tl.w);
+    for (int i = blockIdx.y * 256 + threadIdx.x; i < BM * A.nq; i += gridDim.y * 256) {
+        const int R = tl.y * BM + i / A.nq;
+        if (R >= qlen) return;
+        const size_t at = (size_t)(qs + R) * A.nq + i % A.nq;
+        float m = -INFINITY, l = 0.f;
+        for (int p = 0; p < np; ++p) {                       // a run behind the row's position holds (-inf, 0)
+            const float2 v = A.part_ml[at * MAX_PARTS + p];
+            const float mn = fmaxf(m, v.x), u = mn == -INFINITY ? 0.f : mn;
+            l = l * fast_exp2(m - u) + v.y * fast_exp2(v.x - u);
+            m = mn;
+        }
+        A.lse[at] = m + log2f(l);
+    }
+}
+
+// A block takes MIX_GROUPS groups of four rows of a unit; the group's scores of all heads come as one 1 KB bulk copy a head, three
+// groups ahead; a warp mixes half a row.  A head's place is 16 bytes longer than its data, so that the four heads a quarter of a
+// warp reads together lie in different banks.
+constexpr int MIX_ROWS = 4, MIX_GROUPS = 8, MIX_STAGES = 3, MIX_PLANE = MIX_ROWS * BN * 4 + 16;
 template <int MT>
-__global__ void __launch_bounds__(256) mix_weights_kernel(const MixArgs A) {
-    const int unit = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+__global__ void __launch_bounds__(256, MT == 1 ? 3 : MT == 2 ? 2 : 1) mix_weights_kernel(const MixArgs A) {
+    extern __shared__ __align__(16) unsigned char msm[];
+    __shared__ uint64_t bar[MIX_STAGES];
+    __shared__ int abort_shared;
+    volatile int* abort_flag = &abort_shared;
+    const int unit = A.n_units - 1 - blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int4 tl = A.tiles[A.unit_tile[unit]];
-    const int b = tl.x, key0 = (unit - tl.z) * BN;
+    const int b = tl.x, key0 = (unit - tl.z) * BN, r0 = blockIdx.y * (MIX_ROWS * MIX_GROUPS);
     const int qs = A.q_start[b], qlen = A.q_start[b + 1] - qs, sp = A.start_pos[b];
-    const int n = lane >> 2, c = lane & 3;
+    const int n = lane >> 2, c = lane & 3, row_in = warp >> 1, half = warp & 1;
+    const int rows = min(MIX_ROWS * MIX_GROUPS, qlen - tl.y * BM - r0), groups = rows > 0 ? (rows + MIX_ROWS - 1) / MIX_ROWS : 0;
+    const uint32_t stage_bytes = (uint32_t)A.nq * MIX_PLANE;
+    const float* src = A.scores + (size_t)unit * A.nq * (BM * BN) + r0 * BN;
+    auto fetch = [&](int gq) {                               // by warp 0: group gq's rows of every head
+        uint64_t* br = bar + gq % MIX_STAGES;
+        if (lane == 0) mbar_expect_tx(br, (uint32_t)A.nq * (MIX_ROWS * BN * 4));
+        __syncwarp();
+        for (int h = lane; h < A.nq; h += 32)
+            bulk_load(smem_addr(msm) + (gq % MIX_STAGES) * stage_bytes + h * MIX_PLANE, src + (size_t)h * (BM * BN) + gq * (MIX_ROWS * BN), MIX_ROWS * BN * 4, br);
+    };
+    if (threadIdx.x == 0) {
+        for (int i = 0; i < MIX_STAGES; ++i) mbar_init(bar + i, 1);
+        abort_shared = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    __syncthreads();
+    if (warp == 0)
+        for (int gq = 0; gq < MIX_STAGES && gq < groups; ++gq) fetch(gq);
+    bool ok = true;
 #pragma unroll 1
-    for (int k = 0; k < MIX_ROWS; ++k) {
-        const int r = blockIdx.y * (8 * MIX_ROWS) + k * 8 + warp, R = tl.y * BM + r;
-        const float* L = A.lse + (size_t)(qs + R) * A.nq;
-        bf16* dst = A.mixed + (size_t)unit * A.nq * (BM * BN) + r * BN;
-#pragma unroll 1
-        for (int half = 0; half < 2; ++half) {
-            const int live = R < qlen ? sp + R - (key0 + half * 32) + 1 : 0;         // keys of this half that the row sees
-            float acc[MT][4][4];
-            if (live > 0) {
-                const float* src = A.scores + (size_t)unit * A.nq * (BM * BN) + r * BN + (((half * 8 + n) ^ (r & 7)) << 2);
-                mix_row<MT>(acc, A.mix, A.hp, A.nq, lane, live,
-                            [&](int g) { return *reinterpret_cast<const float4*>(src + (size_t)g * (BM * BN)); }, [&](int g) { return L[g]; });
-            } else {
+    for (int gq = 0; gq < MIX_GROUPS; ++gq) {
+        const int r = r0 + gq * MIX_ROWS + row_in, R = tl.y * BM + r;
+        const int live = R < qlen ? sp + R - (key0 + half * 32) + 1 : 0;             // keys of this half that the row sees
+        float acc[MT][4][4], L[MT][4];
+        if (live > 0) {
 #pragma unroll
-                for (int m = 0; m < MT; ++m)
+            for (int t = 0; t < MT; ++t)
 #pragma unroll
-                    for (int e = 0; e < 4; ++e)
-#pragma unroll
-                        for (int q = 0; q < 4; ++q) acc[m][e][q] = 0.f;
-            }
-            const int piece = ((half * 4 + c) ^ (r & 7)) << 3;
+                for (int k = 0; k < 4; ++k) {
+                    const int g = mix_head(t, k, c);
+                    L[t][k] = g < A.nq ? A.lse[(size_t)(qs + R) * A.nq + g] : 0.f;
+                }
+        }
+        if (gq < groups && ok) ok = __all_sync(0xffffffffu, mbar_wait(bar + gq % MIX_STAGES, (gq / MIX_STAGES) & 1, abort_flag, A.status, 51));
+        if (live > 0 && ok) {
+            const unsigned char* st = msm + (size_t)(gq % MIX_STAGES) * stage_bytes + row_in * (BN * 4) + (((half * 8 + n) ^ (r & 7)) << 4);
+            mix_row<MT>(acc, A.mix, A.hp, A.nq, lane, live, L, [&](int g) { return *reinterpret_cast<const float4*>(st + (size_t)g * MIX_PLANE); });
+        } else {
 #pragma unroll
             for (int m = 0; m < MT; ++m)
 #pragma unroll
-                for (int u = 0; u < 2; ++u) {
-                    const int h = m * 16 + u * 8 + n;
-                    if (h < A.nq) {
-                        uint4 v;
-                        v.x = pack_bf16(acc[m][0][2 * u], acc[m][1][2 * u]);         v.y = pack_bf16(acc[m][2][2 * u], acc[m][3][2 * u]);
-                        v.z = pack_bf16(acc[m][0][2 * u + 1], acc[m][1][2 * u + 1]); v.w = pack_bf16(acc[m][2][2 * u + 1], acc[m][3][2 * u + 1]);
-                        *reinterpret_cast<uint4*>(dst + (size_t)h * (BM * BN) + piece) = v;
-                    }
-                }
+                for (int e = 0; e < 4; ++e)
+#pragma unroll
+                    for (int q = 0; q < 4; ++q) acc[m][e][q] = 0.f;
         }
+        bf16* dst = A.mixed + (size_t)unit * A.nq * (BM * BN) + r * BN + (((half * 4 + c) ^ (r & 7)) << 3);
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+                const int h = m * 16 + u * 8 + n;
+                if (h < A.nq) {
+                    uint4 v;
+                    v.x = pack_bf16(acc[m][0][2 * u], acc[m][1][2 * u]);         v.y = pack_bf16(acc[m][2][2 * u], acc[m][3][2 * u]);
+                    v.z = pack_bf16(acc[m][0][2 * u + 1], acc[m][1][2 * u + 1]); v.w = pack_bf16(acc[m][2][2 * u + 1], acc[m][3][2 * u + 1]);
+                    *reinterpret_cast<uint4*>(dst + (size_t)h * (BM * BN)) = v;
+                }
+            }
+        if (gq + MIX_STAGES < groups) {                      // uniform over the block: the stage has been read by every warp
+            __syncthreads();
+            if (warp == 0) fetch(gq + MIX_STAGES);
+        }
+    }
+    // a block that gave up on a wait leaves only when its own copies have had their (bounded) time
+    if (!ok) {
+        const long long t0 = clock64();
+        while (clock64() - t0 < 2000000LL) { }
     }
 }
 
 // ------------------------------------------------------------------------------------------------ prompts: values
-// Warps 0..3: copies of V, then the epilogue (one row a thread); warp 4: MMA issue; warp 5: P' tiles by bulk copies.
-constexpr int V_STAGES = D <= 128 ? 3 : 2;
+// Warps 0..3: V by asynchronous copies (pages under 8 tokens), then the epilogue (one row a thread); warp 4: MMA issue; warp 5: P'
+// tiles by bulk copies and V by TMA.
+constexpr int V_STAGES = D == 64 ? 8 : D == 128 ? 6 : 4;      // one block an SM: a tile's latency is hidden by depth
 constexpr int V_THREADS = 192;
 constexpr int SV_TILES = V_STAGES * (P_BYTES + K_BYTES);
-constexpr int SV_SMEM = SV_TILES + 1024 + 128;
+constexpr int SV_SMEM = SV_TILES + 1024 + 256;
+static_assert(SV_SMEM <= 227 * 1024 && V_STAGES <= 8, "shared memory");
 
-__global__ void __launch_bounds__(V_THREADS, 1) mix_values_kernel(const MixArgs A) {
+template <bool TMA>
+__global__ void __launch_bounds__(V_THREADS, 1) mix_values_kernel(const __grid_constant__ CUtensorMap map_v, const MixArgs A) {
     extern __shared__ unsigned char smem_raw[];
     unsigned char* base = reinterpret_cast<unsigned char*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
     const uint32_t sP = smem_addr(base), sV = sP + V_STAGES * P_BYTES;
     uint64_t* bars = reinterpret_cast<uint64_t*>(base + SV_TILES);
     uint64_t* bar_p = bars;              // [stage] P' has landed (bytes)
-    uint64_t* bar_v = bars + 3;          // [stage] V has landed
-    uint64_t* bar_free = bars + 6;       // [stage] the product that read the stage is complete (commit)
-    uint64_t* bar_o = bars + 9;          // O is complete
-    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 10);
+    uint64_t* bar_v = bars + 8;          // [stage] V has landed
+    uint64_t* bar_free = bars + 16;      // [stage] the product that read the stage is complete (commit)
+    uint64_t* bar_o = bars + 24;         // O is complete
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 25);
     volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int h = blockIdx.x % A.nq, kh = h / (A.nq / A.nkv);
@@ -374,11 +486,11 @@ __global__ void __launch_bounds__(V_THREADS, 1) mix_values_kernel(const MixArgs 
         const size_t page_stride = (size_t)A.nkv * A.page_size * D;
         const bf16* pages = A.v_pages + (size_t)kh * A.page_size * D;
         bool ok = true;
-        for (int j = 0; j < n_kt && ok; ++j) {               // tile j is on its way while tile j - 1 is waited for
+        for (int j = 0; !TMA && j < n_kt && ok; ++j) {       // tile j is on its way while tile j - 1 is waited for
             const int st = j % V_STAGES;
             if (j >= V_STAGES) ok = mbar_wait(bar_free + st, (j / V_STAGES - 1) & 1, abort_flag, A.status, 46, true);
             if (!ok) break;
-            copy_keys(sV + st * K_BYTES, pages, tab, ps_shift, page_stride, j * BN, pos_hi, tid, BM, A.lim);
+            copy_keys<BM>(sV + st * K_BYTES, pages, tab, ps_shift, page_stride, j * BN, pos_hi, tid, A.lim);
             asm volatile("cp.async.commit_group;" ::: "memory");
             if (j >= 1) {
                 asm volatile("cp.async.wait_group 1;" ::: "memory");
@@ -386,9 +498,11 @@ __global__ void __launch_bounds__(V_THREADS, 1) mix_values_kernel(const MixArgs 
                 mbar_arrive(bar_v + (j - 1) % V_STAGES);
             }
         }
-        cp_async_wait_all();
-        fence_async_proxy();
-        if (ok) mbar_arrive(bar_v + (n_kt - 1) % V_STAGES);
+        if (!TMA) {
+            cp_async_wait_all();
+            fence_async_proxy();
+            if (ok) mbar_arrive(bar_v + (n_kt - 1) % V_STAGES);
+        }
         if (ok) ok = mbar_wait(bar_o, 0, abort_flag, A.status, 47, true);
         if (__all_sync(0xffffffffu, ok)) {
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
@@ -417,7 +531,7 @@ __global__ void __launch_bounds__(V_THREADS, 1) mix_values_kernel(const MixArgs 
             bool ok = true;
             for (int j = 0; j < n_kt && ok; ++j) {
                 const int st = j % V_STAGES, ph = (j / V_STAGES) & 1;
-                ok = mbar_wait(bar_p + st, ph, abort_flag, A.status, 48, true) && mbar_wait(bar_v + st, ph, abort_flag, A.status, 49, true);
+                ok = mbar_wait(bar_p + st, ph, abort_flag, A.status, 48, true) && (TMA || mbar_wait(bar_v + st, ph, abort_flag, A.status, 49, true));
                 if (!ok) break;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
 #pragma unroll
@@ -432,11 +546,16 @@ __global__ void __launch_bounds__(V_THREADS, 1) mix_values_kernel(const MixArgs 
         if (lane == 0) {
             bool ok = true;
             int issued = 0;
+            const int ps_shift = shift_of(A.page_size);
+            if (TMA) asm volatile("prefetch.tensormap [%0];" ::"l"(&map_v) : "memory");
             for (int j = 0; j < n_kt && ok; ++j) {
                 const int st = j % V_STAGES;
+                int page[8];
+                if (TMA) pages_of(page, tab, A.max_pages, ps_shift, j * BN, A.lim);
                 if (j >= V_STAGES) ok = mbar_wait(bar_free + st, (j / V_STAGES - 1) & 1, abort_flag, A.status, 50, true);
                 if (!ok) break;
-                expect_tx(bar_p + st, P_BYTES);
+                mbar_expect_tx(bar_p + st, P_BYTES + (TMA ? K_BYTES : 0));
+                if (TMA) fetch_keys(sV + st * K_BYTES, &map_v, bar_p + st, page, ps_shift, A.nkv, kh);
                 bulk_load(sP + st * P_BYTES, A.mixed + ((size_t)(tl.z + j) * A.nq + h) * (BM * BN), P_BYTES, bar_p + st);
                 issued = j + 1;
             }
@@ -585,11 +704,14 @@ __global__ void __launch_bounds__(256) mix_decode_values_kernel(const MixDecodeA
     __syncthreads();
     const size_t span = (size_t)A.splits * A.range;
     for (int k0 = warp * 32; k0 < keys; k0 += 256) {
-        float acc[MT][4][4];
-        const float* src = A.scores + (size_t)n * A.nq * span + k_lo + k0 + 4 * (lane >> 2);
-        mix_row<MT>(acc, A.mix, A.hp, A.nq, lane, keys - k0, [&](int gg) { return *reinterpret_cast<const float4*>(src + (size_t)gg * span); },
-                    [&](int gg) { return lse[gg]; });
         const int nr = lane >> 2, c = lane & 3;
+        float acc[MT][4][4], L[MT][4];
+#pragma unroll
+        for (int t = 0; t < MT; ++t)
+#pragma unroll
+            for (int k = 0; k < 4; ++k) { const int gg = mix_head(t, k, c); L[t][k] = gg < A.nq ? lse[gg] : 0.f; }
+        const float* src = A.scores + (size_t)n * A.nq * span + k_lo + k0 + 4 * nr;
+        mix_row<MT>(acc, A.mix, A.hp, A.nq, lane, keys - k0, L, [&](int gg) { return *reinterpret_cast<const float4*>(src + (size_t)gg * span); });
 #pragma unroll
         for (int m = 0; m < MT; ++m)
 #pragma unroll
@@ -700,32 +822,58 @@ int raise_smem(K kernel, int bytes, bool (&done)[TL_MAX_DEVICES]) {
 
 }  // namespace
 
-// Prompt portions: three launches over `n_tiles` row tiles.  The caller sizes the scratch: scores n_units * nq * 32 KB, mixed
-// half of it, lse [T, nq].  Pages of 2 to 64 tokens, a power of two; up to 64 query heads.
+template <int MT>
+static int launch_mix(const MixArgs& A, cudaStream_t stream) {
+    const int most = MIX_STAGES * 16 * MT * MIX_PLANE, smem = MIX_STAGES * A.nq * MIX_PLANE;
+    static bool done[TL_MAX_DEVICES] = {};
+    const int e = raise_smem(mix_weights_kernel<MT>, most, done);
+    if (e) return e;
+    mix_weights_kernel<MT><<<dim3(A.n_units, BM / (MIX_ROWS * MIX_GROUPS)), 256, smem, stream>>>(A);
+    return tl_launch_status();
+}
+
+// Runs a row tile of n_kt key tiles is cut into.
+TL_EXPORT int tl_mix_parts(int n_kt) { return (n_kt + part_tiles(n_kt) - 1) / part_tiles(n_kt); }
+TL_EXPORT int tl_mix_max_parts() { return MAX_PARTS; }
+
+// Prompt portions: four launches over `n_tiles` row tiles.  The caller sizes the scratch: scores n_units * nq * 32 KB, mixed
+// half of it, part_ml [T, nq, MAX_PARTS, 2], lse [T, nq].  Pages of 2 to 64 tokens, a power of two; up to 64 query heads.
 TL_EXPORT int tl_mix_prefill(const void* q, int q_stride, void* out, const void* k_pages, const void* v_pages, const int* table, int max_pages,
                              int page_size, const int* q_start, const int* start_pos, const int* slots, int nq, int nkv, float scale,
-                             const int* tiles, int n_tiles, const int* unit_tile, int n_units, float* scores, float* lse, void* mixed,
-                             const void* mix, int hp, int* status, int table_rows, int total_pages, int* fault, cudaStream_t stream) {
+                             const int* tiles, int n_tiles, const int* parts, int n_parts, const int* unit_tile, int n_units, float* scores,
+                             float* part_ml, float* lse, void* mixed, const void* mix, int hp, int* status, int table_rows, int total_pages,
+                             int* fault, cudaStream_t stream) {
     if (n_tiles <= 0) return 0;
     if (nq < 1 || nq > 64 || nq % nkv || hp < nq || hp % 16 || page_size < 2 || page_size > 64 || (page_size & (page_size - 1)) || (q_stride & 7)) return 1;
     const MixArgs A{(const bf16*)q, q_stride, (bf16*)out, (const bf16*)k_pages, (const bf16*)v_pages, table, max_pages, page_size, q_start,
-                    start_pos, slots, nq, nkv, scale * 1.4426950408889634f, (const int4*)tiles, n_tiles, unit_tile, n_units, scores, lse,
+                    start_pos, slots, nq, nkv, scale * 1.4426950408889634f, (const int4*)tiles, n_tiles, (const int2*)parts, n_parts, unit_tile, n_units, scores, (float2*)part_ml, lse,
                     (bf16*)mixed, (const bf16*)mix, hp, status, TlLimits{table_rows, total_pages, fault}};
-    static bool done_s[TL_MAX_DEVICES] = {}, done_v[TL_MAX_DEVICES] = {};
-    int e = raise_smem(mix_scores_kernel, SS_SMEM, done_s);
-    if (!e) e = raise_smem(mix_values_kernel, SV_SMEM, done_v);
+    static bool done_s[TL_MAX_DEVICES] = {}, done_v[TL_MAX_DEVICES] = {}, done_st[TL_MAX_DEVICES] = {}, done_vt[TL_MAX_DEVICES] = {};
+    int e = raise_smem(mix_scores_kernel<false>, SS_SMEM, done_s);
+    if (!e) e = raise_smem(mix_scores_kernel<true>, SS_SMEM, done_st);
+    if (!e) e = raise_smem(mix_values_kernel<false>, SV_SMEM, done_v);
+    if (!e) e = raise_smem(mix_values_kernel<true>, SV_SMEM, done_vt);
     if (e) return e;
-    mix_scores_kernel<<<n_tiles * nq, S_THREADS, SS_SMEM, stream>>>(A);
-    if ((e = tl_launch_status())) return e;
-    const dim3 grid(n_units, BM / (8 * MIX_ROWS));
-    switch ((nq + 15) / 16) {
-        case 1: mix_weights_kernel<1><<<grid, 256, 0, stream>>>(A); break;
-        case 2: mix_weights_kernel<2><<<grid, 256, 0, stream>>>(A); break;
-        case 3: mix_weights_kernel<3><<<grid, 256, 0, stream>>>(A); break;
-        default: mix_weights_kernel<4><<<grid, 256, 0, stream>>>(A);
+    const bool tma = page_size >= 8 && (((uintptr_t)k_pages | (uintptr_t)v_pages) & 127) == 0 && total_pages > 0;
+    CUtensorMap mk{}, mv{};
+    if (tma) {
+        const long long rows = (long long)total_pages * nkv * page_size;
+        if ((e = load_encode()) || (e = make_pages_map(&mk, k_pages, rows, D, page_size)) || (e = make_pages_map(&mv, v_pages, rows, D, page_size))) return e;
     }
+    if (tma) mix_scores_kernel<true><<<n_parts * nq, S_THREADS, SS_SMEM, stream>>>(mk, A);
+    else mix_scores_kernel<false><<<n_parts * nq, S_THREADS, SS_SMEM, stream>>>(mk, A);
     if ((e = tl_launch_status())) return e;
-    mix_values_kernel<<<n_tiles * nq, V_THREADS, SV_SMEM, stream>>>(A);
+    mix_lse_kernel<<<dim3(n_tiles, (BM * nq + 255) / 256), 256, 0, stream>>>(A);
+    if ((e = tl_launch_status())) return e;
+    switch ((nq + 15) / 16) {
+        case 1: e = launch_mix<1>(A, stream); break;
+        case 2: e = launch_mix<2>(A, stream); break;
+        case 3: e = launch_mix<3>(A, stream); break;
+        default: e = launch_mix<4>(A, stream);
+    }
+    if (e) return e;
+    if (tma) mix_values_kernel<true><<<n_tiles * nq, V_THREADS, SV_SMEM, stream>>>(mv, A);
+    else mix_values_kernel<false><<<n_tiles * nq, V_THREADS, SV_SMEM, stream>>>(mv, A);
     return tl_launch_status();
 }
 

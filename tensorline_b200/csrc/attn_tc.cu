@@ -414,14 +414,6 @@ constexpr uint32_t S2_COL = 0, O2_COL = QT * 2 * BN;
 static_assert(O2_COL + QT * D <= 512, "S and O of both tiles must fit the tensor memory");
 static_assert(SMEM2_BYTES <= 227 * 1024, "shared memory");
 
-__device__ __forceinline__ void mbar_expect_tx(uint64_t* bar, uint32_t bytes) {
-    asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(smem_addr(bar)), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ void tma_box(uint32_t dst, const CUtensorMap* map, uint64_t* bar, int x, int y) {
-    asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];"
-                 ::"r"(dst), "l"(map), "r"(smem_addr(bar)), "r"(x), "r"(y) : "memory");
-}
-
 // D[tmem] (+)= A[tmem] * B[smem]: the A operand (P: one row a lane, two bfloat16 a column) comes from tensor memory.
 __device__ __forceinline__ void umma_a_tmem(uint32_t tmem_d, uint32_t tmem_a, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
     asm volatile("{\n\t.reg .pred p;\n\t"
@@ -1093,24 +1085,9 @@ attn_tc3_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     }
 }
 
-typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*,
-                                  const cuuint64_t*, const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave,
-                                  CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-EncodeTiledFn g_encode = nullptr;
 bool g_attr2_done[TL_MAX_DEVICES] = {};
 bool g_attr3_done[TL_MAX_DEVICES] = {};
 
-// The cache tensor [pages, nkv, page, D] as rows of D elements; a box is one page of one KV head, 64 wide.
-int make_pages_map(CUtensorMap* map, const void* base, long long rows, int page_size) {
-    cuuint64_t dims[2] = {(cuuint64_t)D, (cuuint64_t)rows};
-    cuuint64_t strides[1] = {(cuuint64_t)D * 2};
-    cuuint32_t box[2] = {64, (cuuint32_t)page_size};
-    cuuint32_t elem[2] = {1, 1};
-    CUresult r = g_encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, elem,
-                          CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
-                          CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-    return r == CUDA_SUCCESS ? 0 : 101;
-}
 #endif  // HEAD_DIM <= 128
 
 bool g_attr_done[TL_MAX_DEVICES] = {};
@@ -1209,13 +1186,7 @@ static int tc2_prefill_impl(const void* q, int q_stride, void* out, const void* 
     if (page_size < 8 || page_size > 64 || (page_size & (page_size - 1))) return 2;
     if (((uintptr_t)k_pages & 127) || ((uintptr_t)v_pages & 127)) return 2;
     if (nq % nkv || (q_stride & 7) || ((uintptr_t)q & 15)) return 1;
-    if (!g_encode) {
-        void* fn = nullptr;
-        cudaDriverEntryPointQueryResult qres;
-        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &fn, cudaEnableDefault, &qres) != cudaSuccess || !fn ||
-            qres != cudaDriverEntryPointSuccess) return 100;
-        g_encode = (EncodeTiledFn)fn;
-    }
+    if (const int e0 = load_encode()) return e0;
     const int dev = tl_device_index();
     if (dev < 0) return 1;
     if (!g_attr2_done[dev]) {
@@ -1227,8 +1198,8 @@ static int tc2_prefill_impl(const void* q, int q_stride, void* out, const void* 
     CUtensorMap mk, mv;
     const long long rows = total_pages * nkv * page_size;
     int e;
-    if ((e = make_pages_map(&mk, k_pages, rows, page_size))) return e;
-    if ((e = make_pages_map(&mv, v_pages, rows, page_size))) return e;
+    if ((e = make_pages_map(&mk, k_pages, rows, D, page_size))) return e;
+    if ((e = make_pages_map(&mv, v_pages, rows, D, page_size))) return e;
     TcAttnArgs A{};
     A.sink = g_sink;
     A.q = (const bf16*)q; A.q_stride = q_stride; A.out = (bf16*)out;
@@ -1301,13 +1272,7 @@ TL_EXPORT int tl_attn_tc3_prefill(const void* q, int q_stride, void* out, const 
     if (page_size < 8 || page_size > 64 || (page_size & (page_size - 1))) return 2;
     if (((uintptr_t)k_pages & 127) || ((uintptr_t)v_pages & 127)) return 2;
     if (nq % nkv || (q_stride & 7) || ((uintptr_t)q & 15)) return 1;
-    if (!g_encode) {
-        void* fn = nullptr;
-        cudaDriverEntryPointQueryResult qres;
-        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &fn, cudaEnableDefault, &qres) != cudaSuccess || !fn ||
-            qres != cudaDriverEntryPointSuccess) return 100;
-        g_encode = (EncodeTiledFn)fn;
-    }
+    if (const int e0 = load_encode()) return e0;
     const int dev = tl_device_index();
     if (dev < 0) return 1;
     if (!g_attr3_done[dev]) {
@@ -1318,8 +1283,8 @@ TL_EXPORT int tl_attn_tc3_prefill(const void* q, int q_stride, void* out, const 
     CUtensorMap mk, mv;
     const long long rows = total_pages * nkv * page_size;
     int e;
-    if ((e = make_pages_map(&mk, k_pages, rows, page_size))) return e;
-    if ((e = make_pages_map(&mv, v_pages, rows, page_size))) return e;
+    if ((e = make_pages_map(&mk, k_pages, rows, D, page_size))) return e;
+    if ((e = make_pages_map(&mv, v_pages, rows, D, page_size))) return e;
     TcAttnArgs A{};
     A.sink = g_sink;
     A.q = (const bf16*)q; A.q_stride = q_stride; A.out = (bf16*)out;

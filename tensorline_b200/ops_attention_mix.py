@@ -31,13 +31,24 @@ def lib(head_dim: int):
         if head_dim % HEAD_MULTIPLE or not HEAD_MULTIPLE <= head_dim <= 256:
             raise KernelError(f"head_dim {head_dim}: the mixed-head attention kernels take multiples of {HEAD_MULTIPLE} up to 256")
         l = load_library(f"tl_attn_mix_hd{head_dim}", ["attn_mix.cu"], {"HEAD_DIM": head_dim})
-        l.tl_mix_prefill.argtypes = [_P, _I, _P, _P, _P, _P, _I, _I, _P, _P, _P, _I, _I, _F, _P, _I, _P, _I, _P, _P, _P, _P, _I, _P, _I, _I,
-                                     _P, _P]
+        l.tl_mix_prefill.argtypes = [_P, _I, _P, _P, _P, _P, _I, _I, _P, _P, _P, _I, _I, _F, _P, _I, _P, _I, _P, _I, _P, _P, _P, _P, _P, _I,
+                                     _P, _I, _I, _P, _P]
         l.tl_mix_prefill.restype = ctypes.c_int
         l.tl_mix_decode.argtypes = [_P, _I, _P, _P, _P, _P, _I, _I, _P, _P, _P, _I, _I, _I, _F, _I, _I, _P, _P, _P, _P, _I, _I, _I, _P, _P]
         l.tl_mix_decode.restype = ctypes.c_int
+        if l.tl_mix_max_parts() != MAX_PARTS or any(l.tl_mix_parts(n) != parts_of(n) for n in (1, 8, 9, 128, 129, 1000, 5000)):
+            raise KernelError("the mixed-head attention library cuts key tiles into other runs than its launcher")
         _libs[head_dim] = l
     return l
+
+
+MAX_PARTS = 16
+
+
+def parts_of(n_kt: int) -> int:
+    """Runs a row tile of n_kt key tiles is cut into for the scores kernel: of eight key tiles, or sixteen runs of more."""
+    size = -(-n_kt // MAX_PARTS) if n_kt > 8 * MAX_PARTS else 8
+    return -(-n_kt // size)
 
 
 def takes(nq: int, d: int, page_size: int, mix_dtype) -> bool:
@@ -58,7 +69,7 @@ def pad_mix(mix: torch.Tensor) -> torch.Tensor:
 def row_tiles(h_q_start, h_start_pos, requests, max_units: int):
     """Row tiles of 128 tokens of the given requests, the one that reads the most keys first, cut into launches of at most
     `max_units` (row tile x key tile) pairs (a single row tile may exceed it): [(tiles int32 [n, 4] rows (request, tile, first
-    unit, key tiles), unit -> row tile int32)], numpy."""
+    unit, key tiles), parts int32 [m, 2] (row tile, run of its key tiles), unit -> row tile int32)], numpy."""
     tiles = []
     for b in requests:
         n = h_q_start[b + 1] - h_q_start[b]
@@ -71,7 +82,9 @@ def row_tiles(h_q_start, h_start_pos, requests, max_units: int):
     def close():
         nonlocal cur, units
         if cur:
-            out.append((np.array(cur, dtype=np.int32), np.repeat(np.arange(len(cur), dtype=np.int32), [c[3] for c in cur])))
+            parts = [(i, p) for i, c in enumerate(cur) for p in range(parts_of(c[3]))]
+            out.append((np.array(cur, dtype=np.int32), np.array(parts, dtype=np.int32),
+                        np.repeat(np.arange(len(cur), dtype=np.int32), [c[3] for c in cur])))
         cur, units = [], 0
 
     for kt, b, t in tiles:
@@ -84,19 +97,20 @@ def row_tiles(h_q_start, h_start_pos, requests, max_units: int):
 
 
 def prefill(q, out, k_pages, v_pages, table, page_size, q_start, start_pos, slots, launches, nq, nkv, d, scale, mix, lse=None) -> None:
-    """The prompt kernels over `launches` ([(tiles, unit -> tile)] device tensors, see `row_tiles`)."""
+    """The prompt kernels over `launches` ([(tiles, parts, unit -> tile)] device tensors, see `row_tiles`)."""
     from .ops_gemm import status_word
     T = out.shape[0]
-    most = max(u.numel() for _, u in launches)
+    most = max(u.numel() for _, _, u in launches)
     scores = torch.empty(most * nq * ROW_TILE * KEY_TILE, dtype=torch.float32, device=q.device)
     mixed = torch.empty(most * nq * ROW_TILE * KEY_TILE, dtype=torch.bfloat16, device=q.device)
     lse = torch.empty((T, nq), dtype=torch.float32, device=q.device) if lse is None else lse
-    for tiles, unit_tile in launches:
+    part_ml = torch.empty((T, nq, MAX_PARTS, 2), dtype=torch.float32, device=q.device)
+    for tiles, parts, unit_tile in launches:
         _check(lib(d).tl_mix_prefill(_ptr(q), q.shape[1], _ptr(out), _ptr(k_pages), _ptr(v_pages), _ptr(table), table.shape[1], page_size,
                                      _ptr(q_start), _ptr(start_pos), _ptr(slots), nq, nkv, float(scale), _ptr(tiles), tiles.shape[0],
-                                     _ptr(unit_tile), unit_tile.numel(), _ptr(scores), _ptr(lse), _ptr(mixed), _ptr(mix), mix.shape[0],
-                                     _ptr(status_word(q.device)), table.shape[0], k_pages.shape[0], ops.fault_words(q.device), _stream()),
-               "mix_prefill", launches=3)
+                                     _ptr(parts), parts.shape[0], _ptr(unit_tile), unit_tile.numel(), _ptr(scores), _ptr(part_ml), _ptr(lse),
+                                     _ptr(mixed), _ptr(mix), mix.shape[0], _ptr(status_word(q.device)), table.shape[0], k_pages.shape[0],
+                                     ops.fault_words(q.device), _stream()), "mix_prefill", launches=4)
 
 
 def plan_ranges(n: int, nkv: int, group: int, d: int, span: int, sms: int | None = None) -> tuple:
@@ -136,8 +150,8 @@ def attend(qkv, o, ctx, k_pages, v_pages, table, nq, nkv, d, scale, mix) -> None
     if key not in ctx.scratch:                           # one description a step, for every layer
         ones = [b for b in range(ctx.B) if ctx.h_q_start[b + 1] - ctx.h_q_start[b] == 1]
         rest = [b for b in range(ctx.B) if ctx.h_q_start[b + 1] - ctx.h_q_start[b] > 1]
-        launches = [(torch.from_numpy(t).to(qkv.device, non_blocking=True), torch.from_numpy(u).to(qkv.device, non_blocking=True))
-                    for t, u in row_tiles(ctx.h_q_start, ctx.h_start_pos, rest, units)]
+        launches = [tuple(torch.from_numpy(a).to(qkv.device, non_blocking=True) for a in l)
+                    for l in row_tiles(ctx.h_q_start, ctx.h_start_pos, rest, units)]
         singles = None
         if ones:
             packed = torch.tensor([[ctx.h_q_start[b] for b in ones], [ctx.h_start_pos[b] for b in ones], [ctx.h_slots[b] for b in ones]],

@@ -65,7 +65,8 @@ def test_row_tiles_of_prompt_portions():
     q_start, start = [0, 300, 301, 429], [0, 900, 70]
     launches = row_tiles(q_start, start, [0, 2], 7)
     seen = {}
-    for tiles, unit_tile in launches:
+    for tiles, parts, unit_tile in launches:
+        assert parts.tolist() == [[i, p] for i, t in enumerate(tiles) for p in range(-(-int(t[3]) // 8))]
         units = 0
         for i, (b, t, first, kt) in enumerate(tiles.tolist()):
             assert first == units and unit_tile[first:first + kt].tolist() == [i] * kt
@@ -75,7 +76,7 @@ def test_row_tiles_of_prompt_portions():
             seen[(b, t)] = kt
         assert units == len(unit_tile) and (units <= 7 or len(tiles) == 1)
     assert sorted(seen) == [(0, 0), (0, 1), (0, 2), (2, 0)]
-    flat = [int(x[3]) for t, _ in launches for x in t]
+    flat = [int(x[3]) for t, _, _ in launches for x in t]
     assert flat == sorted(flat, reverse=True)
 
 

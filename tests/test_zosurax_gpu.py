@@ -264,7 +264,7 @@ def test_attention_with_mixed_weights(case, kernel):
         ops.attn_mixed_tokenwise(qkv, qkv.shape[1], out, kd, vd, table, ps, i32(pos_all), i32(slot_all), nq, nkv, d, scale, mix.float().cuda())
     elif kernel == "prompt_bf16":                              # everything through the prompt kernels, single tokens too
         for units in (1000, 3):
-            launches = [(torch.from_numpy(t).cuda(), torch.from_numpy(u).cuda()) for t, u in om.row_tiles(q_start, ctx_lens, range(B), units)]
+            launches = [tuple(torch.from_numpy(a).cuda() for a in l) for l in om.row_tiles(q_start, ctx_lens, range(B), units)]
             out.fill_(float("nan"))
             om.prefill(qkv, out, kd, vd, table, ps, *where, launches, nq, nkv, d, scale, pad)
             assert_close(out.view(T, nq, d), W, f"{kernel}, {units} tiles a launch", **BF16)
