@@ -385,20 +385,28 @@ __global__ void __launch_bounds__(256, MT == 1 ? 3 : MT == 2 ? 2 : 1) mix_weight
     if (warp == 0)
         for (int gq = 0; gq < MIX_STAGES && gq < groups; ++gq) fetch(gq);
     bool ok = true;
+    float L[MT][4], L_next[MT][4];                           // the next group's while this one is worked on
+    auto fetch_lse = [&](int gq) {
+        const int R = tl.y * BM + r0 + gq * MIX_ROWS + row_in;
+#pragma unroll
+        for (int t = 0; t < MT; ++t)
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                const int g = mix_head(t, k, c);
+                L_next[t][k] = g < A.nq && R < qlen ? A.lse[(size_t)(qs + R) * A.nq + g] : 0.f;
+            }
+    };
+    fetch_lse(0);
 #pragma unroll 1
     for (int gq = 0; gq < MIX_GROUPS; ++gq) {
         const int r = r0 + gq * MIX_ROWS + row_in, R = tl.y * BM + r;
         const int live = R < qlen ? sp + R - (key0 + half * 32) + 1 : 0;             // keys of this half that the row sees
-        float acc[MT][4][4], L[MT][4];
-        if (live > 0) {
+        float acc[MT][4][4];
 #pragma unroll
-            for (int t = 0; t < MT; ++t)
+        for (int t = 0; t < MT; ++t)
 #pragma unroll
-                for (int k = 0; k < 4; ++k) {
-                    const int g = mix_head(t, k, c);
-                    L[t][k] = g < A.nq ? A.lse[(size_t)(qs + R) * A.nq + g] : 0.f;
-                }
-        }
+            for (int k = 0; k < 4; ++k) L[t][k] = L_next[t][k];
+        if (gq + 1 < groups) fetch_lse(gq + 1);
         if (gq < groups && ok) ok = __all_sync(0xffffffffu, mbar_wait(bar + gq % MIX_STAGES, (gq / MIX_STAGES) & 1, abort_flag, A.status, 51));
         if (live > 0 && ok) {
             const unsigned char* st = msm + (size_t)(gq % MIX_STAGES) * stage_bytes + row_in * (BN * 4) + (((half * 8 + n) ^ (r & 7)) << 4);
@@ -439,14 +447,14 @@ __global__ void __launch_bounds__(256, MT == 1 ? 3 : MT == 2 ? 2 : 1) mix_weight
 // ------------------------------------------------------------------------------------------------ prompts: values
 // Warps 0..3: V by asynchronous copies (pages under 8 tokens), then the epilogue (one row a thread); warp 4: MMA issue; warp 5: P'
 // tiles by bulk copies and V by TMA.
-constexpr int V_STAGES = D == 64 ? 8 : D == 128 ? 6 : 4;      // one block an SM: a tile's latency is hidden by depth
+constexpr int V_STAGES = D <= 128 ? 3 : 2;                    // two blocks an SM (one block of six stages was slower)
 constexpr int V_THREADS = 192;
 constexpr int SV_TILES = V_STAGES * (P_BYTES + K_BYTES);
 constexpr int SV_SMEM = SV_TILES + 1024 + 256;
 static_assert(SV_SMEM <= 227 * 1024 && V_STAGES <= 8, "shared memory");
 
 template <bool TMA>
-__global__ void __launch_bounds__(V_THREADS, 1) mix_values_kernel(const __grid_constant__ CUtensorMap map_v, const MixArgs A) {
+__global__ void __launch_bounds__(V_THREADS, 2) mix_values_kernel(const __grid_constant__ CUtensorMap map_v, const MixArgs A) {
     extern __shared__ unsigned char smem_raw[];
     unsigned char* base = reinterpret_cast<unsigned char*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
     const uint32_t sP = smem_addr(base), sV = sP + V_STAGES * P_BYTES;
