@@ -9,12 +9,14 @@ from __future__ import annotations
 import collections
 import ctypes
 
+import numpy as np
 import torch
 
 from .csrc.build import CHECK_BUILD, load_library
 
 CORE_SOURCES = ["elementwise.cu", "rope_kv.cu", "attn_tokenwise.cu", "gemm_f32.cu", "sampling.cu", "recurrent.cu", "moe.cu",
-                "delta.cu", "latent.cu", "rglru.cu", "streams.cu", "stream_norm.cu", "attn_mixed_tokenwise.cu"]
+                "delta.cu", "latent.cu", "rglru.cu", "streams.cu", "stream_norm.cu", "attn_mixed_tokenwise.cu",
+                "channel_scan.cu"]
 
 _P, _I, _F = ctypes.c_void_p, ctypes.c_int, ctypes.c_float
 
@@ -33,6 +35,8 @@ _SIGNATURES = {
     "tl_sample": [_P, _I, _I, _I, _P, _P, _P, _P, _P],
     "tl_linear_scan": [_P, _I, _I, _I, _I, _I, _P, _F, _P, _P, _I, _I, _P, _F, _F, _P, ctypes.c_longlong, _P, _P, _P, _I, _I,
                        _I, _I, _F, _I, _P, _P, _P],
+    "tl_channel_scan": [_P, _I, _I, _I, _I, _P, _P, _P, ctypes.c_longlong, _P, _P, _P, _I, _P, _I, _P, _P, _P, _I, _I, _I, _P],
+    "tl_channel_chunk": [],
     "tl_scan_state_floats": [_I, _I],
     "tl_scan_columns": [],
     "tl_head_norm_gate": [_P, _P, _I, _I, _P, _I, _P, _I, _I, _I, _I, _F, _I, _P],
@@ -751,6 +755,51 @@ def linear_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, H: int, 
                                  float(q_scale), float(k_scale), _ptr(state), per_slot, _ptr(q_start), _ptr(slots), _ptr(out),
                                  int(B), H, d, dv, float(den_eps), int(single_tokens), _ptr(lower), _ptr(bias), _stream()),
            "linear_step" if single_tokens else "linear_scan")
+
+
+def channel_chunks(h_q_start, chunk: int) -> tuple:
+    """The chunks of a step's requests for `channel_scan`: (int32 [n, 4] rows (request, number, the request's chunks, its first
+    row in this list), int32 rows that begin a request of several chunks), numpy."""
+    rows, carried = [], []
+    for b in range(len(h_q_start) - 1):
+        n = -(-(h_q_start[b + 1] - h_q_start[b]) // chunk)
+        if n > 1:
+            carried.append(len(rows))
+        first = len(rows)
+        rows += [(b, c, n, first) for c in range(n)]
+    return np.array(rows, dtype=np.int32).reshape(-1, 4), np.array(carried, dtype=np.int32)
+
+
+def channel_scan(proj: torch.Tensor, q_off: int, f_off: int, v_off: int, H: int, d: int, dv: int, state: torch.Tensor, ctx,
+                 out: torch.Tensor, lower: torch.Tensor, bias: torch.Tensor) -> None:
+    """`linear_scan` with channel gates for steps of several tokens a request: chunks of a request's tokens side by side (their
+    end states from zero, the carry from chunk to chunk, their outputs).  proj float32; the state as `linear_scan` keeps it, so
+    the two may take turns.  A position's sums depend on where its step began, to rounding."""
+    T = proj.shape[0]
+    _contig(proj, "proj"); _contig(state, "state"); _contig(out, "out")
+    if proj.dtype != torch.float32 or out.dtype != torch.float32 or out.shape != (T, H * dv) or state.dtype != torch.float32:
+        raise KernelError("channel_scan: proj, the state and out [T, H * dv] are float32")
+    floats = -(-dv // scan_columns()) * scan_state_floats(d, False)
+    if state[0].numel() != H * floats:
+        raise KernelError(f"channel_scan: a slot holds {state[0].numel()} floats, these sizes need {H * floats}")
+    for name, off, width in (("q", q_off, H * d), ("f", f_off, H * d), ("v", v_off, H * dv)):
+        if off < 0 or off + width > proj.shape[1]:
+            raise KernelError(f"channel_scan: {name} does not lie inside a projection row")
+    for name, t in (("lower", lower), ("bias", bias)):
+        if t.dtype != torch.float32 or t.numel() != H * d or not t.is_contiguous():
+            raise KernelError(f"channel_scan: {name} must be float32 [H * d]")
+    key = "channel_chunks"
+    if key not in ctx.scratch:                           # one description a step, for every layer
+        rows, carried = channel_chunks(ctx.h_q_start, core().tl_channel_chunk())
+        both = torch.from_numpy(np.concatenate([rows.reshape(-1), carried])).to(proj.device, non_blocking=True)
+        ctx.scratch[key] = (both, len(rows), len(carried))
+    both, n, n_carried = ctx.scratch[key]
+    rows_padded = 32 if d <= 32 else 64 if d <= 64 else 128 if d <= 128 else 256
+    carry = torch.empty((n, H * floats) if n_carried else (1,), dtype=torch.float32, device=proj.device)
+    decay = torch.empty((n, H, rows_padded) if n_carried else (1,), dtype=torch.float32, device=proj.device)
+    _check(core().tl_channel_scan(_ptr(proj), proj.shape[1], q_off, f_off, v_off, _ptr(lower), _ptr(bias), _ptr(state), H * floats,
+                                  _ptr(ctx.q_start), _ptr(ctx.slots), _ptr(both), n, _ptr(both) + 16 * n, n_carried, _ptr(carry),
+                                  _ptr(decay), _ptr(out), H, d, dv, _stream()), "channel_scan", launches=3 if n_carried else 1)
 
 
 _ACTS = {None: 0, "sigmoid": 1, "silu": 2}

@@ -196,8 +196,11 @@ class HGRN2(_MatrixState):
         T = h.shape[0]
         proj = resolve(matmul(h, self.w_in, out_dtype=torch.float32))            # q | f | v, as the product accumulated them
         o = torch.empty((T, H * dv), dtype=torch.float32, device=h.device)
-        ops.linear_scan(proj, 0, H * d, 2 * H * d, H, d, dv, cache.state, ctx.q_start, ctx.slots, ctx.pos, o, B=ctx.B,
-                        lower=self.lower, bias=self.f_bias, single_tokens=ctx.decode_only)
+        if h.dtype == torch.float32 or ctx.decode_only:      # the 32-bit engine walks every step in order: the same floats however cut
+            ops.linear_scan(proj, 0, H * d, 2 * H * d, H, d, dv, cache.state, ctx.q_start, ctx.slots, ctx.pos, o, B=ctx.B,
+                            lower=self.lower, bias=self.f_bias, single_tokens=ctx.decode_only)
+        else:                                                # chunks of a portion side by side
+            ops.channel_scan(proj, 0, H * d, 2 * H * d, H, d, dv, cache.state, ctx, o, self.lower, self.f_bias)
         y = torch.empty((T, H * dv), dtype=h.dtype, device=h.device)
         ops.head_norm_gate(o, y, H, dv, self.eps, weight=self.head_weight)
         return matmul(y, self.w_o)

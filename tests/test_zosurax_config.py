@@ -119,3 +119,10 @@ def test_a_loop_over_no_layers_runs_every_layer_once():
     cfg = ZosuraxConfig.from_dict(raw)
     assert cfg.run_order() == [(i, None) for i in range(4)] == zosurax_plain.order(raw)
     assert tuple(expected_tensors(cfg)["loop.step"].shape) == (3, 48)
+
+
+def test_chunks_of_a_step():
+    from tensorline_b200.ops import channel_chunks
+    rows, carried = channel_chunks([0, 1, 301, 429, 558], 128)
+    assert rows.tolist() == [[0, 0, 1, 0], [1, 0, 3, 1], [1, 1, 3, 1], [1, 2, 3, 1], [2, 0, 1, 4], [3, 0, 2, 5], [3, 1, 2, 5]]
+    assert carried.tolist() == [1, 5]

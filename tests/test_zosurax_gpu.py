@@ -131,11 +131,14 @@ def test_token_shift_across_portions_and_slots(adt, W):
     assert float((wrong - want["a"]).abs().max()) > 0.1, "a shift that is left out must show"
 
 
-@pytest.mark.parametrize("H,d,dv", [(3, 7, 5), (2, 32, 16), (1, 40, 33), (2, 128, 64), (1, 200, 24), (4, 64, 256)])
-def test_memory_with_channel_gates(H, d, dv):
-    """The recurrence of HGRN2 over portions, single tokens and slots that change their owner; the state starts at zero."""
+@pytest.mark.parametrize("chunked", [False, True])
+@pytest.mark.parametrize("H,d,dv", [(3, 7, 5), (2, 32, 16), (1, 40, 33), (2, 128, 64), (1, 200, 24), (4, 64, 256), (2, 256, 70), (3, 128, 200)])
+def test_memory_with_channel_gates(H, d, dv, chunked):
+    """The recurrence of HGRN2 over portions, single tokens and slots that change their owner; the state starts at zero.  In order
+    (single tokens by the step kernel): the bits of one whole pass whatever the cuts.  `chunked`: portions as chunks side by
+    side, in turns with the step kernel for single tokens."""
     from tensorline_b200 import ops
-    lens = {"a": 150, "b": 20, "c": 61}
+    lens = {"a": 150 + 400, "b": 20, "c": 61 + 128}
     slot = {"a": 1, "b": 0, "c": 0}
     g = torch.Generator().manual_seed(5)
     lower, bias = torch.rand(H * d, generator=g) * 0.95, torch.rand(H * d, generator=g) * 4 - 1
@@ -152,7 +155,7 @@ def test_memory_with_channel_gates(H, d, dv):
     state = torch.zeros(3, per, device="cuda")
     at = {k: 0 for k in lens}
     got = {k: [] for k in lens}
-    steps = [[("a", 17), ("b", 2)], [("b", 1), ("a", 1)], [("b", 17)], [("c", 33), ("a", 2)], [("a", 1), ("c", 1)], [("c", 27), ("a", 129)]]
+    steps = [[("a", 17), ("b", 2)], [("b", 1), ("a", 1)], [("b", 17)], [("c", 33), ("a", 2)], [("a", 1), ("c", 1)], [("c", 27), ("a", 129)], [("a", 400), ("c", 128)]]
     for step in steps:
         if step[0][0] == "c" and at["c"] == 0:
             state[slot["c"]].zero_()                          # what the runner does at admission
@@ -160,8 +163,12 @@ def test_memory_with_channel_gates(H, d, dv):
         ctx = step_of(step, at, slot)
         p = torch.cat([proj[k][frm[k]:frm[k] + n] for k, n in step]).cuda()
         o = torch.full((ctx.T, H * dv), float("nan"), device="cuda")
-        ops.linear_scan(p, 0, H * d, 2 * H * d, H, d, dv, state, ctx.q_start, ctx.slots, ctx.pos, o, B=ctx.B, lower=lower.cuda(),
-                        bias=bias.cuda(), single_tokens=ctx.decode_only)
+        if chunked and not ctx.decode_only:
+            ctx.scratch = {}
+            ops.channel_scan(p, 0, H * d, 2 * H * d, H, d, dv, state, ctx, o, lower.cuda(), bias.cuda())
+        else:
+            ops.linear_scan(p, 0, H * d, 2 * H * d, H, d, dv, state, ctx.q_start, ctx.slots, ctx.pos, o, B=ctx.B, lower=lower.cuda(),
+                            bias=bias.cuda(), single_tokens=ctx.decode_only)
         for (k, n), r in zip(step, ctx.h_q_start):
             got[k].append(o[r:r + n])
     assert at == lens
@@ -172,7 +179,7 @@ def test_memory_with_channel_gates(H, d, dv):
         o = torch.empty(lens[k], H * dv, device="cuda")
         ops.linear_scan(proj[k].cuda(), 0, H * d, 2 * H * d, H, d, dv, torch.zeros(3, per, device="cuda"), ctx.q_start, ctx.slots, ctx.pos, o,
                         B=1, lower=lower.cuda(), bias=bias.cuda())
-        assert torch.equal(o, torch.cat(got[k])), f"request {k}: the cuts show"
+        assert chunked or torch.equal(o, torch.cat(got[k])), f"request {k}: the cuts show"
     lost = plain(proj["a"][17:])                              # a state that is lost at a cut shows long after it
     assert float((lost[5] - want["a"][22]).abs().max()) > 1e-3
 
