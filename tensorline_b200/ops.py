@@ -35,7 +35,7 @@ _SIGNATURES = {
     "tl_sample": [_P, _I, _I, _I, _P, _P, _P, _P, _P],
     "tl_linear_scan": [_P, _I, _I, _I, _I, _I, _P, _F, _P, _P, _I, _I, _P, _F, _F, _P, ctypes.c_longlong, _P, _P, _P, _I, _I,
                        _I, _I, _F, _I, _P, _P, _P],
-    "tl_channel_scan": [_P, _I, _I, _I, _I, _P, _P, _P, ctypes.c_longlong, _P, _P, _P, _I, _P, _I, _P, _P, _P, _I, _I, _I, _P],
+    "tl_channel_scan": [_P, _I, _I, _I, _I, _I, _P, _P, _P, ctypes.c_longlong, _P, _P, _P, _I, _P, _I, _P, _P, _P, _I, _I, _I, _P],
     "tl_channel_chunk": [],
     "tl_scan_state_floats": [_I, _I],
     "tl_scan_columns": [],
@@ -774,7 +774,7 @@ def channel_scan(proj: torch.Tensor, q_off: int, f_off: int, v_off: int, H: int,
                  out: torch.Tensor, lower: torch.Tensor, bias: torch.Tensor) -> None:
     """`linear_scan` with channel gates for steps of several tokens a request: chunks of a request's tokens side by side (their
     end states from zero, the carry from chunk to chunk, their outputs).  proj float32; the state as `linear_scan` keeps it, so
-    the two may take turns.  A position's sums depend on where its step began, to rounding."""
+    the two may take turns.  `proj` is worked on in place (the gates take the place of their pre-activations).  A position's sums depend on where its step began, to rounding."""
     T = proj.shape[0]
     _contig(proj, "proj"); _contig(state, "state"); _contig(out, "out")
     if proj.dtype != torch.float32 or out.dtype != torch.float32 or out.shape != (T, H * dv) or state.dtype != torch.float32:
@@ -797,9 +797,9 @@ def channel_scan(proj: torch.Tensor, q_off: int, f_off: int, v_off: int, H: int,
     rows_padded = 32 if d <= 32 else 64 if d <= 64 else 128 if d <= 128 else 256
     carry = torch.empty((n, H * floats) if n_carried else (1,), dtype=torch.float32, device=proj.device)
     decay = torch.empty((n, H, rows_padded) if n_carried else (1,), dtype=torch.float32, device=proj.device)
-    _check(core().tl_channel_scan(_ptr(proj), proj.shape[1], q_off, f_off, v_off, _ptr(lower), _ptr(bias), _ptr(state), H * floats,
+    _check(core().tl_channel_scan(_ptr(proj), T, proj.shape[1], q_off, f_off, v_off, _ptr(lower), _ptr(bias), _ptr(state), H * floats,
                                   _ptr(ctx.q_start), _ptr(ctx.slots), _ptr(both), n, _ptr(both) + 16 * n, n_carried, _ptr(carry),
-                                  _ptr(decay), _ptr(out), H, d, dv, _stream()), "channel_scan", launches=3 if n_carried else 1)
+                                  _ptr(decay), _ptr(out), H, d, dv, _stream()), "channel_scan", launches=4 if n_carried else 2)
 
 
 _ACTS = {None: 0, "sigmoid": 1, "silu": 2}
