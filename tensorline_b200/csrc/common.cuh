@@ -185,6 +185,13 @@ __device__ __forceinline__ float tl_act(float g, int act) {
     return g / (1.0f + expf(-g));
 }
 
+// relu(v)^2 of a product's accumulator, rounded to bfloat16 first (what a stored product would hold): the epilogues of the
+// bfloat16 products without a gate.
+__device__ __forceinline__ float tl_relu_squared_rounded(float v) {
+    const float r = fmaxf(__bfloat162float(__float2bfloat16_rn(v)), 0.f);
+    return r * r;
+}
+
 // The clamped swish works on the pair: g' = min(g, limit), u' = clamp(u, -limit, limit); g' sigmoid(alpha g') (u' + 1).
 #define TL_ACT_SWISH_CLAMPED 3
 __device__ __forceinline__ float tl_swish_clamped(float g, float u, float limit, float alpha) {

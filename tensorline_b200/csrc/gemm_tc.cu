@@ -128,6 +128,7 @@ struct GemmArgs {
     int gated;            // swap, one split: rows 0..63 of every 128-row tile of A are gate features, rows 64..127 the
                           // up features of the same 64 columns; out[b, 64 tile + j] = silu(gate) * up, [RB, RA / 2]
     float gate_limit, gate_alpha;   // gated = 3: the clamped swish's constants
+    int act;              // swap, bfloat16 out, one split or splits summed in a cluster: out = relu(.)^2
     long long wait_cycles;   // how long a wait on a barrier may take before the block gives up
     int drop_last_load;      // tests only: the copy thread leaves out its last stage, so the MMA thread's wait runs out
     // The residual add folded into the product that makes the addend (swap, cluster_reduce): the block that finishes a
@@ -434,7 +435,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                         const int b = b0 + c0 + j;
                         if (b < G.RB) {
                             if (G.out_f32) ((float*)G.out)[(size_t)b * G.ldo + a] = __uint_as_float(r[j]);
-                            else ((bf16*)G.out)[(size_t)b * G.ldo + a] = __float2bfloat16_rn(__uint_as_float(r[j]));
+                            else ((bf16*)G.out)[(size_t)b * G.ldo + a] = __float2bfloat16_rn(G.act ? tl_relu_squared_rounded(__uint_as_float(r[j])) : __uint_as_float(r[j]));
                         }
                     }
                 } else {
@@ -533,6 +534,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                     sq = warp_sum(sq);
                     if (lane == 0) G.ssq_out[(size_t)(b0 + tok) * gridDim.x + blockIdx.x] = sq;
                     continue;
+                }
+                if (G.act) {
+                    acc.x = tl_relu_squared_rounded(acc.x); acc.y = tl_relu_squared_rounded(acc.y);
+                    acc.z = tl_relu_squared_rounded(acc.z); acc.w = tl_relu_squared_rounded(acc.w);
                 }
                 const size_t o = (size_t)(b0 + tok) * G.ldo + a;
                 if (wide && a + 3 < G.RA) {
@@ -694,7 +699,7 @@ TL_EXPORT int tl_gemm_tc_set_gate(float limit, float alpha) { g_gate_limit = lim
 // (splits * T * N floats); with `counters` (n_counters zeroed ints, at least one per tile, left zeroed) the
 // last block of a tile sums the partials inside the same launch, else a second kernel does.  `status` (device int, zero before
 // the call) receives a non-zero code if a wait inside the kernel ran out.  `gated` (swap = 1, one split, N % 128 == 0, bfloat16 out):
-// w holds gate and up rows interleaved in blocks of 64 and y [T, N / 2] receives silu(gate) * up.  `cluster_reduce` (swap = 1,
+// w holds gate and up rows interleaved in blocks of 64 and y [T, N / 2] receives silu(gate) * up; 4: no gate, y [T, N] receives relu(.)^2 (swap = 1, splits only in a cluster).  `cluster_reduce` (swap = 1,
 // 2..8 ranges): the ranges of a tile are a thread-block cluster and sum their tiles through distributed shared memory.
 namespace {
 // The two fusions with the layer's norms (see GemmArgs).  All null / zero: the plain product.
@@ -727,9 +732,14 @@ int gemm_impl(const void* x, const void* w, void* y, int out_f32, int ldo, int T
     const int per = (k_tiles + splits - 1) / splits;
     splits = (k_tiles + per - 1) / per;                                                  // no empty split
     if (y == nullptr && splits < 2) return 1;
+    const int act = gated == 4;                                                          // no gate: the square of relu over every output
+    if (act) {
+        gated = 0;
+        if (!swap || out_f32 || y == nullptr || adds || (splits > 1 && !cluster_reduce)) return 1;
+    }
     if (gated && (!swap || splits != 1 || out_f32 || (N & 127) || y == nullptr)) return 1;   // whole 64 + 64 tiles, one split
     GemmArgs G{};
-    G.gated = gated;
+    G.gated = gated; G.act = act;
     G.gate_limit = g_gate_limit; G.gate_alpha = g_gate_alpha;
     G.cluster_reduce = (cluster_reduce && splits >= 2) ? 1 : 0;
     if (cluster_reduce && (!swap || splits > 8 || (y == nullptr && !adds))) return 1;

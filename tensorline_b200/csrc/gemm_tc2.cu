@@ -14,7 +14,7 @@
 // the w rows of the tiles in flight inside the L2.  The accumulator is double-buffered in tensor memory
 // (2 x 256 of the 512 columns), so the four epilogue warps of each block read, convert and store tile i while
 // the MMA thread already runs tile i + 1.  Two epilogues:
-//   * plain: y[t, n] in bfloat16 or float;
+//   * plain: y[t, n] in bfloat16 or float, or relu(y[t, n])^2 in bfloat16;
 //   * gated: w holds gate and up rows interleaved in blocks of 64 (rows 128 j .. 128 j + 63 the gate features
 //     64 j .., rows 128 j + 64 .. the up features of the same columns); y[t, 64 j + c] = silu(gate) * up, both
 //     rounded to bfloat16 first (what a stored gate|up product would hold), y is [T, N / 2] bfloat16.
@@ -121,6 +121,7 @@ struct Gemm2Args {
     int T, N, K;
     int m_tiles, n_tiles;  // tiles of 256 rows and 256 columns
     int out_f32, gated;
+    int act;               // plain epilogue, bf16 out: y = relu(y)^2
     float gate_limit, gate_alpha;   // gated = 3: the clamped swish's constants
     int* status;
 };
@@ -281,7 +282,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant
                             } else {
                                 float v[16];
 #pragma unroll
-                                for (int j = 0; j < 16; ++j) v[j] = __uint_as_float(r[j]);
+                                for (int j = 0; j < 16; ++j) v[j] = G.act ? tl_relu_squared_rounded(__uint_as_float(r[j])) : __uint_as_float(r[j]);
                                 store16_bf16((bf16*)G.out + (size_t)t * G.ldo + col, v, G.N - col);
                             }
                         }
@@ -350,13 +351,16 @@ int cached_map(CUtensorMap* map, const void* base, int rows, int K) {
 }  // namespace
 
 // y[T, N] = x[T, K] w[N, K]^T (bfloat16 operands; y bfloat16 or float, rows `ldo` elements apart).  `gated`: see the top of
-// the file; y is then [T, N / 2] bfloat16 and N a multiple of 128.  `status`: device int, zero before the call; non-zero
+// the file; y is then [T, N / 2] bfloat16 and N a multiple of 128; 4: the plain
+// epilogue with relu(y)^2.  `status`: device int, zero before the call; non-zero
 // afterwards if a wait inside the kernel ran out.  `max_pairs`: pairs of blocks to launch at most (0: as many as the GPU
 // holds).  Returns 0, a CUDA error code, or 1 for arguments it does not take.
 TL_EXPORT int tl_gemm_tc2(const void* x, const void* w, void* y, int out_f32, int ldo, int T, int N, int K, int gated,
                           int* status, int max_pairs, cudaStream_t stream) {
     if (T <= 0 || N <= 0) return 0;
     if (K <= 0 || (K & 7) || ((uintptr_t)x & 15) || ((uintptr_t)w & 15) || y == nullptr || status == nullptr) return 1;
+    const int act = gated == 4;                            // no gate: the square of relu over every output
+    if (act) { gated = 0; if (out_f32) return 1; }
     if (gated && (out_f32 || (N & 127))) return 1;
     if (!g_encode) {
         void* fn = nullptr;
@@ -380,7 +384,7 @@ TL_EXPORT int tl_gemm_tc2(const void* x, const void* w, void* y, int out_f32, in
     Gemm2Args G{};
     G.out = y; G.ldo = ldo; G.T = T; G.N = N; G.K = K;
     G.m_tiles = (T + 2 * BM - 1) / (2 * BM); G.n_tiles = (N + BN - 1) / BN;
-    G.out_f32 = out_f32; G.gated = gated; G.status = status;
+    G.out_f32 = out_f32; G.gated = gated; G.act = act; G.status = status;
     G.gate_limit = g_gate_limit; G.gate_alpha = g_gate_alpha;
     long long tiles = (long long)G.m_tiles * G.n_tiles;
     int pairs = tl_num_sms() / 2;

@@ -185,6 +185,93 @@ __global__ void rope_kv_vec_kernel(bf16* __restrict__ qkv, const TW* __restrict_
     }
 }
 
+// The bfloat16 path of the other options (a q/k norm, either pairing, a rotation over part of the head; no bias): one block per
+// token, its angles' cosines and sines once in shared memory for all heads; a thread moves 8 consecutive values, the d / 8
+// lanes of a head (a power of two) sum its squares by shuffles, and a rotate-half partner comes from the lane that holds it.
+template <bool INTERLEAVED>
+__global__ void rope_kv_norm_vec_kernel(bf16* __restrict__ qkv, const int* __restrict__ pos, const int* __restrict__ req_slot,
+                                        const int* __restrict__ table, int max_pages, int page_size, const float* __restrict__ inv_freq,
+                                        int rot, int nq, int nkv, int d, bf16* __restrict__ k_pages, bf16* __restrict__ v_pages, int heads,
+                                        const float* __restrict__ q_norm, const float* __restrict__ k_norm, float norm_eps, int norm_dim,
+                                        int norm_cast, const TlLimits L) {
+    extern __shared__ float cs[];                                // cos[rot / 2], sin[rot / 2]
+    const int t = blockIdx.x, p = pos[t], rhalf = rot >> 1, per_head = d >> 3;
+    for (int i = threadIdx.x; i < rhalf; i += blockDim.x) {
+        float s, c;
+        sincosf(__fmul_rn((float)p, inv_freq[i]), &s, &c);
+        cs[i] = c; cs[rhalf + i] = s;
+    }
+    size_t page_base = 0;
+    if (heads > nq) {
+        const int slot = tl_checked(req_slot[t], L.table_rows, L, TL_K_ROPE);
+        const int page = tl_checked(table[(size_t)slot * max_pages + tl_checked(p / page_size, max_pages, L, TL_K_ROPE)],
+                                    L.total_pages, L, TL_K_ROPE);
+        page_base = ((size_t)page * nkv * page_size + (p % page_size)) * d;
+    }
+    grid_dependency_wait();
+    grid_dependency_trigger();
+    __syncthreads();
+    bf16* row = qkv + (size_t)t * (nq + 2 * nkv) * d;
+    const int items = heads * per_head, hop = rhalf >> 3;       // lanes between a rotate-half pair
+    for (int i0 = threadIdx.x & ~31; i0 < items; i0 += blockDim.x) {         // whole warps: the lanes exchange
+        const int item = min(i0 + (threadIdx.x & 31), items - 1), hh = item / per_head, piece = item - hh * per_head, e0 = piece * 8;
+        const bool mine = i0 + (threadIdx.x & 31) < items;
+        float a[8];
+        load8(row + (size_t)hh * d + e0, a);
+        const bool turns = hh < nq + nkv;
+        const float* nw = !turns ? nullptr : (hh < nq ? q_norm : k_norm);
+        float ss = 0.f;
+#pragma unroll
+        for (int k = 0; k < 8; ++k) ss = fmaf(a[k], a[k], ss);
+        for (int o = 1; o < per_head; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        if (nw) {
+            const float rstd = 1.0f / sqrtf(ss / (float)(norm_dim > 0 ? norm_dim : d) + norm_eps);
+            float w[8];
+            load8(nw + e0, w);
+#pragma unroll
+            for (int k = 0; k < 8; ++k) {
+                a[k] *= rstd;
+                if (norm_cast) a[k] = __bfloat162float(__float2bfloat16_rn(a[k]));
+                a[k] *= w[k];
+            }
+        }
+        if (INTERLEAVED) {
+            if (turns && e0 < rot) {
+#pragma unroll
+                for (int k = 0; k < 8; k += 2) {
+                    const float c = cs[(e0 + k) >> 1], s = cs[rhalf + ((e0 + k) >> 1)];
+                    const float ra = __fmul_rn(a[k], c) - __fmul_rn(a[k + 1], s), rb = __fmul_rn(a[k + 1], c) + __fmul_rn(a[k], s);
+                    a[k] = ra; a[k + 1] = rb;
+                }
+            }
+        } else {
+            const bool low = e0 < rhalf;
+            const int lane = threadIdx.x & 31, other = low ? lane + hop : lane - hop;
+#pragma unroll
+            for (int k = 0; k < 8; ++k) {
+                const float b = __shfl_sync(0xffffffffu, a[k], other & 31);
+                if (turns && e0 < rot) {
+                    const int i = (low ? e0 : e0 - rhalf) + k;
+                    const float c = cs[i], s = cs[rhalf + i];
+                    a[k] = low ? __fmul_rn(a[k], c) - __fmul_rn(b, s) : __fmul_rn(a[k], c) + __fmul_rn(b, s);
+                }
+            }
+        }
+        if (mine) {
+            uint4 o;
+            __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+            for (int k = 0; k < 4; ++k) o2[k] = __floats2bfloat162_rn(a[2 * k], a[2 * k + 1]);
+            bf16* dst = row + (size_t)hh * d;
+            if (hh >= nq) {
+                const int kh = hh < nq + nkv ? hh - nq : hh - nq - nkv;
+                dst = (hh < nq + nkv ? k_pages : v_pages) + page_base + (size_t)kh * page_size * d;
+            }
+            *reinterpret_cast<uint4*>(dst + e0) = o;
+        }
+    }
+}
+
 TL_EXPORT int tl_rope_kv_write(void* qkv, int act_dtype, const void* bias, int bias_dtype,
                                const int* pos, const int* req_slot, const int* table, int max_pages,
                                int page_size, const float* inv_freq, int rot, int nq, int nkv, int d,
@@ -209,6 +296,15 @@ TL_EXPORT int tl_rope_kv_write(void* qkv, int act_dtype, const void* bias, int b
         if (bias_dtype == TL_F32) return pieces ? VROPE(float, true) : VROPE(float, false);
         return pieces ? VROPE(bf16, true) : VROPE(bf16, false);
 #undef VROPE
+    }
+    const int per_head = d / 8;
+    if (act_dtype == TL_BF16 && !bias && (d & 7) == 0 && d <= 256 && (per_head & (per_head - 1)) == 0 && (rot & (interleaved ? 7 : 15)) == 0 &&
+        aligned && (((uintptr_t)q_norm | (uintptr_t)k_norm) & 15) == 0) {
+        const int items = (heads * per_head + 31) / 32 * 32, threads = items < 512 ? items : 512;
+#define NROPE(I) launch_after_wait(rope_kv_norm_vec_kernel<I>, dim3(T), dim3(threads), (size_t)rot * sizeof(float), stream, (bf16*)qkv, pos, req_slot, table, \
+            max_pages, page_size, inv_freq, rot, nq, nkv, d, (bf16*)k_pages, (bf16*)v_pages, heads, q_norm, k_norm, norm_eps, norm_dim, norm_cast, L)
+        return interleaved ? NROPE(true) : NROPE(false);
+#undef NROPE
     }
     dim3 grid(T, heads);
     const int half = d / 2;

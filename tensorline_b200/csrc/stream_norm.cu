@@ -49,66 +49,83 @@ template <> struct Pack<1> {
     template <typename T> static __device__ __forceinline__ void store(T* p, const float (&v)[1]) { *p = from_f<T>(v[0]); }
 };
 
-// v of one row in this thread's columns, and the thread's share of the sum of its squares
-template <typename TA, int VEC, int NV>
-__device__ __forceinline__ float sum_row(const SumNormArgs& A, size_t t, int nvec, float (&v)[NV][VEC]) {
+// v of L rows in this thread's columns, and the thread's shares of the sums of their squares.  `at`: the rows' first elements, or
+// -1 for a row that is not there (its v is zero).  Source after source, so that the loads of all rows are in flight together.
+template <typename TA, int VEC, int NV, int L>
+__device__ __forceinline__ void sum_rows(const SumNormArgs& A, const long long (&at)[L], int nvec, float (&v)[L][NV][VEC], float (&ss)[L]) {
     using P = Pack<VEC>;
-    const size_t base = t * (size_t)A.W;
+    auto place = [&](int k) { return (size_t)(threadIdx.x + k * blockDim.x) * VEC; };
+    auto here = [&](int k) { return threadIdx.x + k * blockDim.x < nvec; };
 #pragma unroll
-    for (int k = 0; k < NV; ++k) {
-        const int c = threadIdx.x + k * blockDim.x;
-        if (c < nvec) P::load(A.x + base + (size_t)c * VEC, v[k]);
-    }
-    if (A.base) {
+    for (int j = 0; j < L; ++j)
 #pragma unroll
         for (int k = 0; k < NV; ++k) {
-            const int c = threadIdx.x + k * blockDim.x;
-            if (c < nvec) {
-                float b[VEC]; P::load(A.base + base + (size_t)c * VEC, b);
 #pragma unroll
-                for (int e = 0; e < VEC; ++e) v[k][e] += b[e];
-            }
+            for (int e = 0; e < VEC; ++e) v[j][k][e] = 0.f;
+            if (at[j] >= 0 && here(k)) P::load(A.x + at[j] + place(k), v[j][k]);
         }
+    if (A.base) {
+        float b[L][NV][VEC];
+#pragma unroll
+        for (int j = 0; j < L; ++j)
+#pragma unroll
+            for (int k = 0; k < NV; ++k) {
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) b[j][k][e] = 0.f;
+                if (at[j] >= 0 && here(k)) P::load(A.base + at[j] + place(k), b[j][k]);
+            }
+#pragma unroll
+        for (int j = 0; j < L; ++j)
+#pragma unroll
+            for (int k = 0; k < NV; ++k)
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) v[j][k][e] += b[j][k][e];
     }
     if (A.row) {
 #pragma unroll
         for (int k = 0; k < NV; ++k) {
-            const int c = threadIdx.x + k * blockDim.x;
-            if (c < nvec) {
-                float b[VEC]; P::load(A.row + (size_t)c * VEC, b);
+            if (!here(k)) continue;
+            float b[VEC]; P::load(A.row + place(k), b);
 #pragma unroll
-                for (int e = 0; e < VEC; ++e) v[k][e] += b[e];
-            }
+            for (int j = 0; j < L; ++j)
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) if (at[j] >= 0) v[j][k][e] += b[e];
         }
     }
 #pragma unroll
     for (int i = 0; i < SUM_ADDENDS; ++i) {
         if (i < A.n_add) {
-            const TA* a = (const TA*)A.add[i] + base;
+            const TA* a = (const TA*)A.add[i];
+            float av[L][NV][VEC];
+#pragma unroll
+            for (int j = 0; j < L; ++j)
+#pragma unroll
+                for (int k = 0; k < NV; ++k) {
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) av[j][k][e] = 0.f;
+                    if (at[j] >= 0 && here(k)) P::load(a + at[j] + place(k), av[j][k]);
+                }
 #pragma unroll
             for (int k = 0; k < NV; ++k) {
-                const int c = threadIdx.x + k * blockDim.x;
-                if (c < nvec) {
-                    float av[VEC], sv[VEC];
-                    P::load(a + (size_t)c * VEC, av);
-                    if (A.scale[i]) P::load(A.scale[i] + (size_t)c * VEC, sv);
-                    else {
+                float sv[VEC];
 #pragma unroll
-                        for (int e = 0; e < VEC; ++e) sv[e] = 1.0f;
-                    }
+                for (int e = 0; e < VEC; ++e) sv[e] = 1.0f;
+                if (A.scale[i] && here(k)) P::load(A.scale[i] + place(k), sv);
 #pragma unroll
-                    for (int e = 0; e < VEC; ++e) v[k][e] = fmaf(sv[e], av[e], v[k][e]);
-                }
+                for (int j = 0; j < L; ++j)
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) v[j][k][e] = fmaf(sv[e], av[j][k][e], v[j][k][e]);
             }
         }
     }
-    float ss = 0.f;
 #pragma unroll
-    for (int k = 0; k < NV; ++k)
-        if (threadIdx.x + k * blockDim.x < nvec)
+    for (int j = 0; j < L; ++j) {
+        ss[j] = 0.f;
 #pragma unroll
-            for (int e = 0; e < VEC; ++e) ss = fmaf(v[k][e], v[k][e], ss);
-    return ss;
+        for (int k = 0; k < NV; ++k)
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) ss[j] = fmaf(v[j][k][e], v[j][k][e], ss[j]);
+    }
 }
 
 // L sums over the block at once; the order of additions is that of one sum alone.  red: [L][33] floats.
@@ -134,7 +151,7 @@ __device__ __forceinline__ void block_sums(float (&s)[L], float (*red)[33]) {
 }
 
 template <typename TA, typename TW, int VEC, int NV, int NR, bool SHIFT>
-__global__ void sum_norm_kernel(const SumNormArgs A) {
+__global__ void __launch_bounds__(1024) sum_norm_kernel(const SumNormArgs A) {
     using P = Pack<VEC>;
     constexpr int L = NR + (SHIFT ? 1 : 0);
     __shared__ float red[L][33];
@@ -155,12 +172,13 @@ __global__ void sum_norm_kernel(const SumNormArgs A) {
     grid_dependency_trigger();
     if (!early) load_w();
     float v[L][NV][VEC], ss[L];
+    long long at[L];
 #pragma unroll
     for (int j = 0; j < L; ++j) {
         const int t = t0 + j - (SHIFT ? 1 : 0);
-        ss[j] = 0.f;
-        if (t >= 0 && t < A.T && !(SHIFT && j == 0 && A.single)) ss[j] = sum_row<TA, VEC, NV>(A, A.rows ? (size_t)A.rows[t] : (size_t)t, nvec, v[j]);
+        at[j] = t >= 0 && t < A.T && !(SHIFT && j == 0 && A.single) ? (long long)(A.rows ? A.rows[t] : t) * A.W : -1;
     }
+    sum_rows<TA, VEC, NV, L>(A, at, nvec, v, ss);
     if (!SHIFT && A.write_x) {
 #pragma unroll
         for (int j = 0; j < L; ++j)
@@ -235,8 +253,17 @@ __global__ void sum_norm_kernel(const SumNormArgs A) {
             while (lo < hi) { const int mid = (lo + hi) >> 1; if (A.q_start[mid] < t) lo = mid + 1; else hi = mid; }
             last = A.q_start[lo + 1] - 1;
         }
+        if (NR == 1 && last == t) {                          // a single token: its own row
+#pragma unroll
+            for (int k = 0; k < NV; ++k) {
+                const int c = threadIdx.x + k * blockDim.x;
+                if (c < nvec) P::store(st + (size_t)c * VEC, v[L - 1][k]);
+            }
+            continue;
+        }
         float n[1][NV][VEC], s1[1];
-        s1[0] = sum_row<TA, VEC, NV>(A, (size_t)last, nvec, n[0]);
+        const long long where[1] = {(long long)last * A.W};
+        sum_rows<TA, VEC, NV, 1>(A, where, nvec, n, s1);
         block_sums<1>(s1, red);
         const float rstd = 1.0f / sqrtf(s1[0] / (float)A.W + A.eps);
 #pragma unroll

@@ -80,7 +80,8 @@ class GatedMLP(Part):
 
 @register_feed_forward("plain_mlp")
 class PlainMLP(Part):
-    """y = act(h Wu^T) Wd^T, no gate and no biases; act = the square of relu (`relu_squared`)."""
+    """y = act(h Wu^T) Wd^T, no gate and no biases; act = the square of relu (`relu_squared`), in the epilogue of the tcgen05
+    products (steps of few tokens, long steps), a kernel of its own in between."""
     graph_capturable = True
 
     def __init__(self, rt: Runtime, hidden: int, intermediate: int, activation: str = "relu_squared", names: dict | None = None):
@@ -101,6 +102,17 @@ class PlainMLP(Part):
         self.w_down = self._compute_copy(weights[f"{prefix}.{self.names['down']}"])
 
     def forward(self, h, ctx):
+        m = self._inner(resolve(h))
+        return matmul(m, self.w_down, may_defer=True, to_residual=True)          # the next norm adds it up
+
+    def _inner(self, h):
+        T, I, H = h.shape[0], self.intermediate, self.hidden
+        if h.dtype == torch.bfloat16 and h.is_cuda and h.is_contiguous():
+            from .. import ops_gemm
+            if use_tc(T, I, H) and ops_gemm.can_act(T, I, H):
+                return ops_gemm.gemm_tc(h, self.w_up, gated="relu_squared")
+            if use_pair_product(T, I, H):
+                return ops_gemm.gemm_tc2(h, self.w_up, gated="relu_squared")
         m = resolve(matmul(h, self.w_up))
         ops.relu_square(m)
-        return matmul(m, self.w_down, may_defer=True, to_residual=True)          # the next norm adds it up
+        return m
