@@ -606,6 +606,15 @@ struct MixDecodeArgs {
     TlLimits lim;
 };
 
+constexpr int MIX_MAX_RANGE = 512;
+// The page numbers of keys [k_lo, k_hi) into shared memory, by `parts` threads.
+__device__ __forceinline__ void range_pages(int* page_of, const int* tab, int max_pages, int ps_shift, int k_lo, int k_hi, int part, int parts,
+                                            const TlLimits& L) {
+    const int first = k_lo >> ps_shift, last = (k_hi - 1) >> ps_shift;
+    for (int i = part; i <= last - first; i += parts)
+        page_of[i] = tl_checked(tab[tl_checked(first + i, max_pages, L, TL_K_DECODE)], L.total_pages, L, TL_K_DECODE);
+}
+
 // grid (ranges, KV heads x tiles of 16 heads of the group, requests), 4 warps; a warp takes 16 keys at a time.  The lanes of
 // a quad hold a key's row in 16-byte pieces, and Q in the same order of dimensions, so K goes from memory to the product.
 __global__ void __launch_bounds__(128) mix_decode_scores_kernel(const MixDecodeArgs A) {
@@ -620,6 +629,9 @@ __global__ void __launch_bounds__(128) mix_decode_scores_kernel(const MixDecodeA
     const int* tab = A.table + (size_t)tl_checked(A.slots[n], A.lim.table_rows, A.lim, TL_K_DECODE) * A.max_pages;
     const bf16* pages = A.k_pages + (size_t)kh * A.page_size * D;
     const size_t page_stride = (size_t)A.nkv * A.page_size * D;
+    __shared__ int page_of[MIX_MAX_RANGE];
+    range_pages(page_of, tab, A.max_pages, ps_shift, k_lo, k_hi, threadIdx.x, 128, A.lim);
+    __syncthreads();
     uint4 qa[D / 32], qb[D / 32];
     {
         const bf16* q = A.q + (size_t)A.rows[n] * A.q_stride + (size_t)h0 * D + 8 * c;
@@ -638,20 +650,22 @@ __global__ void __launch_bounds__(128) mix_decode_scores_kernel(const MixDecodeA
         for (int u = 0; u < 2; ++u) {
             const int j = k0 + u * 8 + r;
             const bool live = j <= p;
-            const int page = live ? tl_checked(tab[tl_checked(j >> ps_shift, A.max_pages, A.lim, TL_K_DECODE)], A.lim.total_pages, A.lim, TL_K_DECODE) : 0;
+            const int page = live ? page_of[(j >> ps_shift) - (k_lo >> ps_shift)] : 0;
             const bf16* src = pages + (size_t)page * page_stride + (size_t)(j & ps_mask) * D + 8 * c;
 #pragma unroll
             for (int s = 0; s < D / 32; ++s) kv[u][s] = live ? *reinterpret_cast<const uint4*>(src + 32 * s) : make_uint4(0, 0, 0, 0);
         }
 #pragma unroll
         for (int u = 0; u < 2; ++u) {
-            float d[4] = {0.f, 0.f, 0.f, 0.f};
+            float d[4] = {0.f, 0.f, 0.f, 0.f}, d1[4] = {0.f, 0.f, 0.f, 0.f};          // two chains
 #pragma unroll
             for (int s = 0; s < D / 32; ++s) {
                 const uint32_t a0[4] = {qa[s].x, qb[s].x, qa[s].y, qb[s].y}, a1[4] = {qa[s].z, qb[s].z, qa[s].w, qb[s].w};
                 mma16816(d, a0, kv[u][s].x, kv[u][s].y);
-                mma16816(d, a1, kv[u][s].z, kv[u][s].w);
+                mma16816(d1, a1, kv[u][s].z, kv[u][s].w);
             }
+#pragma unroll
+            for (int e = 0; e < 4; ++e) d[e] += d1[e];
             const int j = k0 + u * 8 + 2 * c;
 #pragma unroll
             for (int e = 0; e < 4; ++e) d[e] = j + (e & 1) <= p ? d[e] * A.scale_log2 : -INFINITY;
@@ -699,15 +713,39 @@ __global__ void __launch_bounds__(256) mix_decode_values_kernel(const MixDecodeA
     const int used = p / A.range + 1;                        // ranges that hold keys
     const int g = A.nq / A.nkv, all_units = A.nkv * CH, chunks = (g + GC - 1) / GC;
     const int u0 = (blockIdx.z / chunks) * A.units, gi0 = (blockIdx.z % chunks) * GC, un = min(A.units, all_units - u0);
-    for (int h = tid; h < A.nq; h += 256) {
+    // this thread's piece of the values and its first keys, on their way while the weights are made
+    const int ks_n = 256 / un, ks = tid / un, unit = u0 + tid - ks * un, kh = unit / CH, piece = unit - kh * CH;
+    const bool live = ks < ks_n;
+    const int ps_shift = shift_of(A.page_size), ps_mask = A.page_size - 1;
+    const int* tab = A.table + (size_t)tl_checked(A.slots[n], A.lim.table_rows, A.lim, TL_K_DECODE) * A.max_pages;
+    const bf16* pages = A.v_pages + (size_t)kh * A.page_size * D + piece * 8;
+    const size_t page_stride = (size_t)A.nkv * A.page_size * D;
+    __shared__ int page_of[MIX_MAX_RANGE];                   // the range's pages
+    range_pages(page_of, tab, A.max_pages, ps_shift, k_lo, k_hi, tid, 256, A.lim);
+    __syncthreads();
+    constexpr int UN = 8;
+    uint4 v[UN];
+    auto fetch = [&](int k0) {
+#pragma unroll
+        for (int u = 0; u < UN; ++u) {
+            const int k = k0 + u * ks_n, j = k_lo + k;
+            v[u] = make_uint4(0, 0, 0, 0);
+            if (live && k < keys)
+                v[u] = *reinterpret_cast<const uint4*>(pages + (size_t)page_of[(j >> ps_shift) - (k_lo >> ps_shift)] * page_stride + (size_t)(j & ps_mask) * D);
+        }
+    };
+    fetch(ks);
+    for (int h = warp; h < A.nq; h += 8) {                   // a warp a head, a lane a range
         float m = -INFINITY, l = 0.f;
-        for (int s = 0; s < used; ++s) {
-            const float2 v = *reinterpret_cast<const float2*>(A.ml + (((size_t)n * A.splits + s) * A.nq + h) * 2);
-            const float mn = fmaxf(m, v.x);
-            l = l * fast_exp2(m - mn) + v.y * fast_exp2(v.x - mn);
+        for (int s = lane; s < used; s += 32) {
+            const float2 x = *reinterpret_cast<const float2*>(A.ml + (((size_t)n * A.splits + s) * A.nq + h) * 2);
+            const float mn = fmaxf(m, x.x);
+            l = l * fast_exp2(m - mn) + x.y * fast_exp2(x.x - mn);
             m = mn;
         }
-        lse[h] = m + log2f(l);
+        const float top = warp_max(m);
+        l = warp_sum(m == -INFINITY ? 0.f : l * fast_exp2(m - top));
+        if (lane == 0) lse[h] = top + log2f(l);
     }
     __syncthreads();
     const size_t span = (size_t)A.splits * A.range;
@@ -733,8 +771,6 @@ __global__ void __launch_bounds__(256) mix_decode_values_kernel(const MixDecodeA
             }
     }
     __syncthreads();
-    const int ks_n = 256 / un, ks = tid / un, unit = u0 + tid - ks * un, kh = unit / CH, piece = unit - kh * CH;
-    const bool live = ks < ks_n;
     const int gn = min(GC, g - gi0);
     float o[GC][8];
 #pragma unroll
@@ -742,23 +778,9 @@ __global__ void __launch_bounds__(256) mix_decode_values_kernel(const MixDecodeA
 #pragma unroll
         for (int e = 0; e < 8; ++e) o[i][e] = 0.f;
     if (live) {
-        const int ps_shift = shift_of(A.page_size), ps_mask = A.page_size - 1;
-        const int* tab = A.table + (size_t)tl_checked(A.slots[n], A.lim.table_rows, A.lim, TL_K_DECODE) * A.max_pages;
-        const bf16* pages = A.v_pages + (size_t)kh * A.page_size * D + piece * 8;
-        const size_t page_stride = (size_t)A.nkv * A.page_size * D;
         const float* pw = pm + (size_t)(kh * g + gi0) * pstride;
-        constexpr int UN = 4;
         for (int k0 = ks; k0 < keys; k0 += UN * ks_n) {
-            uint4 v[UN];
-#pragma unroll
-            for (int u = 0; u < UN; ++u) {
-                const int k = k0 + u * ks_n;
-                if (k < keys) {
-                    const int j = k_lo + k;
-                    const int page = tl_checked(tab[tl_checked(j >> ps_shift, A.max_pages, A.lim, TL_K_DECODE)], A.lim.total_pages, A.lim, TL_K_DECODE);
-                    v[u] = *reinterpret_cast<const uint4*>(pages + (size_t)page * page_stride + (size_t)(j & ps_mask) * D);
-                }
-            }
+            if (k0 != ks) fetch(k0);
 #pragma unroll
             for (int u = 0; u < UN; ++u) {
                 const int k = k0 + u * ks_n;
@@ -779,20 +801,20 @@ __global__ void __launch_bounds__(256) mix_decode_values_kernel(const MixDecodeA
             }
         }
     }
-    // the key slots' shares, summed in their order; [ks][unit][GC][8] takes the place of the weights
+    // the key slots' shares, summed in their order; [GC * 8][thread] takes the place of the weights
     __syncthreads();
     if (live) {
 #pragma unroll
         for (int i = 0; i < GC; ++i)
 #pragma unroll
-            for (int e = 0; e < 8; ++e) pm[(((size_t)ks * un + tid - ks * un) * GC + i) * 8 + e] = o[i][e];
+            for (int e = 0; e < 8; ++e) pm[(i * 8 + e) * 256 + tid] = o[i][e];
     }
     __syncthreads();
     for (int idx = tid; idx < un * GC * 8; idx += 256) {
-        const int uu = idx / (GC * 8), i = (idx / 8) % GC, e = idx & 7;
+        const int uu = idx % un, ie = idx / un, i = ie >> 3, e = ie & 7;
         if (i >= gn) continue;
         float v = 0.f;
-        for (int s = 0; s < ks_n; ++s) v += pm[(((size_t)s * un + uu) * GC + i) * 8 + e];
+        for (int s = 0; s < ks_n; ++s) v += pm[ie * 256 + s * un + uu];
         const int k2 = (u0 + uu) / CH, pc = (u0 + uu) - k2 * CH, h = k2 * g + gi0 + i;
         if (A.splits == 1) A.out[((size_t)A.rows[n] * A.nq + h) * D + pc * 8 + e] = __float2bfloat16_rn(v);
         else A.part[(((size_t)n * A.splits + blockIdx.x) * A.nq + h) * D + pc * 8 + e] = v;
@@ -807,6 +829,7 @@ __global__ void __launch_bounds__(128) mix_decode_sum_kernel(const MixDecodeArgs
     if (i >= width) return;
     const int used = A.start_pos[n] / A.range + 1;
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
     for (int s = 0; s < used; ++s) {
         const float4 x = *reinterpret_cast<const float4*>(A.part + ((size_t)n * A.splits + s) * width + i);
         v.x += x.x; v.y += x.y; v.z += x.z; v.w += x.w;
@@ -904,7 +927,7 @@ TL_EXPORT int tl_mix_decode(const void* q, int q_stride, void* out, const void* 
                             int total_pages, int* fault, cudaStream_t stream) {
     if (n <= 0) return 0;
     if (nq < 1 || nq > 64 || nq % nkv || hp < nq || hp % 16 || page_size < 1 || page_size > 64 || (page_size & (page_size - 1)) ||
-        (q_stride & 7) || range < 64 || range % 64 || splits < 1 || (splits > 1 && !part) || n > 65535) return 1;
+        (q_stride & 7) || range < 64 || range % 64 || range > MIX_MAX_RANGE || splits < 1 || (splits > 1 && !part) || n > 65535) return 1;
     const int g = nq / nkv, gc = g == 1 ? 1 : g == 2 ? 2 : g <= 4 ? 4 : 8;
     const int units = nkv * CH < 64 ? nkv * CH : 64;
     const MixDecodeArgs A{(const bf16*)q, q_stride, (bf16*)out, (const bf16*)k_pages, (const bf16*)v_pages, table, max_pages, page_size, rows,

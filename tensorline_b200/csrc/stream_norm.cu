@@ -157,21 +157,45 @@ __global__ void __launch_bounds__(1024) sum_norm_kernel(const SumNormArgs A) {
     __shared__ float red[L][33];
     const int nvec = A.W / VEC;
     const int t0 = blockIdx.x * NR;
-    float wv[NV][VEC];
+    float wv[NV][VEC], mu[NV][VEC];
     const bool early = gridDim.x <= 128;                     // few rows: the weights, nobody's output, come before the wait
     auto load_w = [&]() {
         if (A.h == nullptr) return;
 #pragma unroll
         for (int k = 0; k < NV; ++k) {
             const int c = threadIdx.x + k * blockDim.x;
-            if (c < nvec) P::load((const TW*)A.w + (size_t)c * VEC, wv[k]);
+            if (c < nvec) {
+                P::load((const TW*)A.w + (size_t)c * VEC, wv[k]);
+                if (SHIFT) P::load(A.shift + (size_t)c * VEC, mu[k]);
+            }
         }
     };
     if (early) load_w();
     grid_dependency_wait();
     grid_dependency_trigger();
     if (!early) load_w();
+    int slot_of[NR];                                         // which rows are the first of their request's portion, and where its state lies
+    unsigned firsts = 0, starts = 0;
+    if (SHIFT) {
+#pragma unroll
+        for (int j = 0; j < NR; ++j) {
+            const int t = t0 + j;
+            slot_of[j] = 0;
+            if (t >= A.T) continue;
+            slot_of[j] = A.req_slot[t];
+            const int before = t > 0 ? A.req_slot[t - 1] : -1, p = A.pos[t];
+            if (A.single || before != slot_of[j]) { firsts |= 1u << j; if (p == 0) starts |= 1u << j; }
+        }
+    }
     float v[L][NV][VEC], ss[L];
+    float pv_early[NV][VEC];                                 // one row a block: the state's row comes with the others
+    if (SHIFT && NR == 1 && firsts && !starts) {
+#pragma unroll
+        for (int k = 0; k < NV; ++k) {
+            const int c = threadIdx.x + k * blockDim.x;
+            if (c < nvec) P::load(A.prev + (size_t)slot_of[0] * A.prev_stride + (size_t)c * VEC, pv_early[k]);
+        }
+    }
     long long at[L];
 #pragma unroll
     for (int j = 0; j < L; ++j) {
@@ -211,32 +235,30 @@ __global__ void __launch_bounds__(1024) sum_norm_kernel(const SumNormArgs A) {
                 }
         return;
     }
-    unsigned firsts = 0;                                     // bit j: row t0 + j is the first of its request's portion
 #pragma unroll
     for (int j = 0; j < NR; ++j) {
         const int t = t0 + j;
         if (t >= A.T) continue;
-        const int slot = A.req_slot[t];
-        const bool first = A.single || t == 0 || A.req_slot[t - 1] != slot;
-        if (first) firsts |= 1u << j;
-        const bool start = first && A.pos[t] == 0;
-        const float* st = A.prev + (size_t)slot * A.prev_stride;
+        const bool first = (firsts >> j) & 1u, start = (starts >> j) & 1u;
+        const float* st = A.prev + (size_t)slot_of[j] * A.prev_stride;
 #pragma unroll
         for (int k = 0; k < NV; ++k) {
             const int c = threadIdx.x + k * blockDim.x;
             if (c < nvec) {
-                float pv[VEC], mu[VEC], o[VEC];
-                P::load(A.shift + (size_t)c * VEC, mu);
+                float pv[VEC], o[VEC];
                 if (start) {
 #pragma unroll
                     for (int e = 0; e < VEC; ++e) pv[e] = 0.f;
+                } else if (first && NR == 1) {
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) pv[e] = pv_early[k][e];
                 } else if (first) P::load(st + (size_t)c * VEC, pv);
                 else {
 #pragma unroll
                     for (int e = 0; e < VEC; ++e) pv[e] = v[j][k][e];
                 }
 #pragma unroll
-                for (int e = 0; e < VEC; ++e) o[e] = fmaf(pv[e] - v[j + 1][k][e], mu[e], v[j + 1][k][e]);
+                for (int e = 0; e < VEC; ++e) o[e] = fmaf(pv[e] - v[j + 1][k][e], mu[k][e], v[j + 1][k][e]);
                 P::store(h + (size_t)t * A.W + (size_t)c * VEC, o);
             }
         }
@@ -285,7 +307,7 @@ static int launch_sum_norm(const SumNormArgs& A, cudaStream_t stream) {
     // one thread count for a width whatever the step (the order of additions), rows a block by how many there are
 #define SN(NV, NR, S) launch_after_wait(sum_norm_kernel<TA, TW, VEC, NV, NR, S>, dim3((A.T + NR - 1) / NR), dim3(((nvec + NV - 1) / NV + 31) / 32 * 32), 0, stream, A)
     if (nvec <= 1024) {
-        if (shift) return (A.T >= 512 && !A.single) ? SN(1, 3, true) : SN(1, 1, true);
+        if (shift) return A.single || A.T < 256 ? SN(1, 1, true) : A.T < 1024 ? SN(1, 3, true) : SN(1, 7, true);
         return SN(1, 1, false);
     }
     if (nvec <= 2048) return shift ? SN(2, 1, true) : SN(2, 1, false);

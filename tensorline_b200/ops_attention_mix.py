@@ -115,11 +115,11 @@ def prefill(q, out, k_pages, v_pages, table, page_size, q_start, start_pos, slot
 
 def plan_ranges(n: int, nkv: int, group: int, d: int, span: int, sms: int | None = None) -> tuple:
     """(keys a range, ranges) of a decode step of n requests that read at most `span` keys: enough ranges that the blocks of
-    the second kernel fill the GPU twice over, none under 64 keys."""
+    the second kernel fill the GPU once, none under 64 keys."""
     sms = sms or ops.num_sms()
     blocks = n * -(-nkv * d // 8 // 64) * -(-group // 8)
     tiles = max(1, -(-span // 64))
-    splits = min(tiles, max(1, 2 * sms // max(1, blocks)))
+    splits = min(tiles, max(1, sms // max(1, blocks)))
     rng = min(DECODE_MAX_RANGE, -(-tiles // splits) * 64)
     return rng, -(-tiles * 64 // rng)
 
