@@ -14,6 +14,7 @@
 //   decoding   scores   a block a (request, KV head, range of keys): scores and the range's (m, l)
 //              mix and values   a block a (request, range of keys, group of KV heads): P' of the range, then its share of O
 //              sum      the ranges' shares added up (they need no rescaling: the weights are normalised already)
+//              or, where a request's keys fit the shared memory of a cluster of blocks, all of it in one launch
 // Scratch is laid out in the order its reader wants it: scores in 128 x 64 tiles, a row's 16-byte pieces exclusive-ored with the
 // row number (the writer's shared-memory image, stored by one bulk copy); P' as the swizzled A-operand tile, loaded by one.
 // Every wait is bounded; a block whose wait runs out records a code in `status` and leaves.
@@ -839,6 +840,212 @@ __global__ void __launch_bounds__(128) mix_decode_sum_kernel(const MixDecodeArgs
     *reinterpret_cast<uint2*>(A.out + (size_t)A.rows[n] * width + i) = o;
 }
 
+// ------------------------------------------------------------------------------------------------ decoding in a cluster
+// One launch for the three above: the blocks of a request form a thread-block cluster, each with an equal run of its keys and all
+// heads.  A block scores its run into shared memory; the runs' (m, l) meet through distributed shared memory; the block mixes
+// its run in place, applies it to the values and leaves its share of O in shared memory, where the cluster adds the shares up,
+// a slice of the columns a block.  grid (cluster size, requests).
+constexpr int MC_THREADS = D <= 128 ? 512 : 256;
+constexpr int MC_WARPS = MC_THREADS / 32;
+
+struct MixClusterShape { int pstride, pages; };              // floats a head's row of weights, page numbers of a run
+
+__device__ __forceinline__ void mc_barrier() {
+    asm volatile("barrier.cluster.arrive.release;\n\tbarrier.cluster.wait.acquire;" ::: "memory");
+}
+__device__ __forceinline__ uint32_t mc_peer(const void* p, int rank) {
+    uint32_t out;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(out) : "r"(smem_addr(p)), "r"(rank));
+    return out;
+}
+__device__ __forceinline__ float2 mc_load2(uint32_t at) {
+    float2 v;
+    asm volatile("ld.shared::cluster.v2.f32 {%0, %1}, [%2];" : "=f"(v.x), "=f"(v.y) : "r"(at) : "memory");
+    return v;
+}
+__device__ __forceinline__ float4 mc_load4(uint32_t at) {
+    float4 v;
+    asm volatile("ld.shared::cluster.v4.f32 {%0, %1, %2, %3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(at) : "memory");
+    return v;
+}
+// floats of shared memory in front of the weights: (m, l) and L of every head; and behind them: O of every slice of the keys
+__host__ __device__ __forceinline__ int mc_heads_floats(int nq) { return (3 * nq + 3) & ~3; }
+__host__ __device__ __forceinline__ int mc_slices(int nq, int tiles) {
+    const int every = tiles < MC_WARPS ? MC_WARPS / tiles : 1, most = nq < 64 ? 64 / nq : 1;
+    return every < most ? every : most;
+}
+__host__ __device__ __forceinline__ int mc_bytes(int nq, int tiles, MixClusterShape S) {
+    return 4 * (mc_heads_floats(nq) + nq * S.pstride + mc_slices(nq, tiles) * nq * D + ((S.pages + 3) & ~3));
+}
+
+template <int MT>
+__global__ void __launch_bounds__(MC_THREADS, 1) mix_decode_cluster_kernel(const MixDecodeArgs A, const MixClusterShape Sh) {
+    extern __shared__ __align__(16) float dsm[];
+    const int C = gridDim.x, rank = blockIdx.x, n = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    float* ml = dsm;                                         // [nq][2]
+    float* lse = dsm + 2 * A.nq;                             // [nq]
+    float* pm = dsm + mc_heads_floats(A.nq);                 // [nq][pstride]  scores, then weights
+    float* os = pm + (size_t)A.nq * Sh.pstride;              // [slices][nq][D]
+    const int g = A.nq / A.nkv, gt = (g + 15) / 16, nt = A.nkv * gt, slices = mc_slices(A.nq, nt);
+    int* page_of = reinterpret_cast<int*>(os + (size_t)slices * A.nq * D);
+    grid_dependency_wait();
+    grid_dependency_trigger();
+    const int p = A.start_pos[n], rng = ((p + C) / C + 31) & ~31, k_lo = rank * rng, k_hi = min(k_lo + rng, p + 1), keys = max(0, k_hi - k_lo);
+    const int ps_shift = shift_of(A.page_size), ps_mask = A.page_size - 1;
+    const size_t page_stride = (size_t)A.nkv * A.page_size * D, row = A.rows[n];
+    if (keys > 0) {
+        const int* tab = A.table + (size_t)tl_checked(A.slots[n], A.lim.table_rows, A.lim, TL_K_DECODE) * A.max_pages;
+        range_pages(page_of, tab, A.max_pages, ps_shift, k_lo, k_hi, tid, MC_THREADS, A.lim);
+    }
+    __syncthreads();
+    {   // scores: a warp keeps the queries of one tile of heads and takes 16 keys at a time
+        const int groups = min(nt, MC_WARPS), every = MC_WARPS / groups, r = lane >> 2, c = lane & 3;
+        for (int t = warp % groups; t < nt && warp < groups * every; t += groups) {
+            const int kh = t / gt, h0 = kh * g + (t % gt) * 16, hn = min(16, (kh + 1) * g - h0);
+            const bf16* pages = A.k_pages + (size_t)kh * A.page_size * D + 8 * c;
+            const bf16* q = A.q + row * A.q_stride + (size_t)h0 * D + 8 * c;
+            uint4 qa[D / 32], qb[D / 32], kv[2][D / 32];
+#pragma unroll
+            for (int s = 0; s < D / 32; ++s) {
+                qa[s] = r < hn ? *reinterpret_cast<const uint4*>(q + (size_t)r * D + 32 * s) : make_uint4(0, 0, 0, 0);
+                qb[s] = r + 8 < hn ? *reinterpret_cast<const uint4*>(q + (size_t)(r + 8) * D + 32 * s) : make_uint4(0, 0, 0, 0);
+            }
+            for (int k0 = warp / groups * 16; k0 < keys; k0 += every * 16) {
+#pragma unroll
+                for (int u = 0; u < 2; ++u) {
+                    const int k = k0 + u * 8 + r, j = k_lo + k;
+                    const bf16* src = pages + (size_t)(k < keys ? page_of[(j >> ps_shift) - (k_lo >> ps_shift)] : 0) * page_stride + (size_t)(j & ps_mask) * D;
+#pragma unroll
+                    for (int s = 0; s < D / 32; ++s) kv[u][s] = k < keys ? *reinterpret_cast<const uint4*>(src + 32 * s) : make_uint4(0, 0, 0, 0);
+                }
+#pragma unroll
+                for (int u = 0; u < 2; ++u) {
+                    float d[4] = {0.f, 0.f, 0.f, 0.f}, d1[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+                    for (int s = 0; s < D / 32; ++s) {
+                        const uint32_t a0[4] = {qa[s].x, qb[s].x, qa[s].y, qb[s].y}, a1[4] = {qa[s].z, qb[s].z, qa[s].w, qb[s].w};
+                        mma16816(d, a0, kv[u][s].x, kv[u][s].y);
+                        mma16816(d1, a1, kv[u][s].z, kv[u][s].w);
+                    }
+                    const int k = k0 + u * 8 + 2 * c;
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) d[e] = k + (e & 1) < keys ? (d[e] + d1[e]) * A.scale_log2 : -INFINITY;
+                    if (r < hn) *reinterpret_cast<float2*>(pm + (size_t)(h0 + r) * Sh.pstride + k) = make_float2(d[0], d[1]);
+                    if (r + 8 < hn) *reinterpret_cast<float2*>(pm + (size_t)(h0 + r + 8) * Sh.pstride + k) = make_float2(d[2], d[3]);
+                }
+            }
+        }
+    }
+    __syncthreads();
+    for (int h = warp; h < A.nq; h += MC_WARPS) {            // the run's maximum and sum, a warp a head
+        float m = -INFINITY, l = 0.f;
+        for (int k = lane; k < keys; k += 32) m = fmaxf(m, pm[(size_t)h * Sh.pstride + k]);
+        m = warp_max(m);
+        for (int k = lane; k < keys; k += 32) l += fast_exp2(pm[(size_t)h * Sh.pstride + k] - m);
+        l = warp_sum(l);
+        if (lane == 0) { ml[2 * h] = m; ml[2 * h + 1] = l; }
+    }
+    mc_barrier();
+    for (int h = warp; h < A.nq; h += MC_WARPS) {            // over all runs, a lane a run
+        float2 x = make_float2(-INFINITY, 0.f);
+        if (lane < C) x = mc_load2(mc_peer(ml + 2 * h, lane));
+        const float top = warp_max(x.x);
+        const float l = warp_sum(x.x == -INFINITY ? 0.f : x.y * fast_exp2(x.x - top));
+        if (lane == 0) lse[h] = top + log2f(l);
+    }
+    __syncthreads();
+    for (int k0 = warp * 32; k0 < keys; k0 += MC_THREADS) {  // the mix, 32 keys a warp, in place: nobody else touches these keys
+        const int nr = lane >> 2, c = lane & 3;
+        float acc[MT][4][4], L[MT][4];
+#pragma unroll
+        for (int t = 0; t < MT; ++t)
+#pragma unroll
+            for (int k = 0; k < 4; ++k) { const int gg = mix_head(t, k, c); L[t][k] = gg < A.nq ? lse[gg] : 0.f; }
+        mix_row<MT>(acc, A.mix, A.hp, A.nq, lane, keys - k0, L,
+                    [&](int gg) { return *reinterpret_cast<const float4*>(pm + (size_t)gg * Sh.pstride + k0 + 4 * nr); });
+        __syncwarp();
+        // P' rounded for the product with the values: a row's 32 keys as packed pairs in the first half of their 32 floats
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+                const int h = m * 16 + u * 8 + nr;
+                if (h < A.nq) {
+                    uint4 v;
+                    v.x = pack_bf16(acc[m][0][2 * u], acc[m][1][2 * u]);         v.y = pack_bf16(acc[m][2][2 * u], acc[m][3][2 * u]);
+                    v.z = pack_bf16(acc[m][0][2 * u + 1], acc[m][1][2 * u + 1]); v.w = pack_bf16(acc[m][2][2 * u + 1], acc[m][3][2 * u + 1]);
+                    *reinterpret_cast<uint4*>(pm + (size_t)h * Sh.pstride + k0 + 4 * c) = v;
+                }
+            }
+    }
+    __syncthreads();
+    {   // values: a warp takes one tile of heads and every slices-th 16 keys.  Lane (r, c) fetches 16-byte pieces of the rows of keys
+        // 2c, 2c + 1, 2c + 8, 2c + 9, dimensions 64 s + 8 r ..; product i of a piece takes dimension 64 s + 8 n + i as its column n
+        const int groups = min(nt, MC_WARPS / slices), r = lane >> 2, c = lane & 3, slice = warp / groups;
+        for (int t = warp % groups; t < nt && slice < slices; t += groups) {
+            const int kh = t / gt, h0 = kh * g + (t % gt) * 16, hn = min(16, (kh + 1) * g - h0);
+            const bf16* pages = A.v_pages + (size_t)kh * A.page_size * D + 8 * r;
+            float o[D / 8][4];
+#pragma unroll
+            for (int i = 0; i < D / 8; ++i)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) o[i][e] = 0.f;
+            for (int k0 = slice * 16; k0 < keys; k0 += slices * 16) {
+                uint4 v[4][D / 64];
+#pragma unroll
+                for (int q = 0; q < 4; ++q) {
+                    const int k = k0 + 2 * c + (q & 1) + (q >> 1) * 8, j = k_lo + k;
+                    const bf16* src = pages + (size_t)(k < keys ? page_of[(j >> ps_shift) - (k_lo >> ps_shift)] : 0) * page_stride + (size_t)(j & ps_mask) * D;
+#pragma unroll
+                    for (int s = 0; s < D / 64; ++s) v[q][s] = k < keys ? *reinterpret_cast<const uint4*>(src + 64 * s) : make_uint4(0, 0, 0, 0);
+                }
+                uint32_t a[4];
+                const float* w = pm + (size_t)(h0 + r) * Sh.pstride + (k0 & ~31) + ((k0 & 31) >> 1) + c;
+                a[0] = r < hn ? __float_as_uint(w[0]) : 0u;     a[1] = r + 8 < hn ? __float_as_uint(w[8 * (size_t)Sh.pstride]) : 0u;
+                a[2] = r < hn ? __float_as_uint(w[4]) : 0u;     a[3] = r + 8 < hn ? __float_as_uint(w[8 * (size_t)Sh.pstride + 4]) : 0u;
+#pragma unroll
+                for (int s = 0; s < D / 64; ++s) {
+                    const uint32_t x[4][4] = {{v[0][s].x, v[0][s].y, v[0][s].z, v[0][s].w}, {v[1][s].x, v[1][s].y, v[1][s].z, v[1][s].w},
+                                              {v[2][s].x, v[2][s].y, v[2][s].z, v[2][s].w}, {v[3][s].x, v[3][s].y, v[3][s].z, v[3][s].w}};
+#pragma unroll
+                    for (int i = 0; i < 8; ++i)
+                        mma16816(o[s * 8 + i], a, __byte_perm(x[0][i >> 1], x[1][i >> 1], i & 1 ? 0x7632 : 0x5410),
+                                 __byte_perm(x[2][i >> 1], x[3][i >> 1], i & 1 ? 0x7632 : 0x5410));
+                }
+            }
+#pragma unroll
+            for (int s = 0; s < D / 64; ++s)
+#pragma unroll
+                for (int i = 0; i < 8; ++i)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const int hr = r + (e >> 1) * 8;
+                        if (hr < hn) os[((size_t)slice * A.nq + h0 + hr) * D + 64 * s + 8 * (2 * c + (e & 1)) + i] = o[s * 8 + i][e];
+                    }
+        }
+    }
+    __syncthreads();
+    for (int i = tid; slices > 1 && i < A.nq * D; i += MC_THREADS) {
+        float x = os[i];
+        for (int s = 1; s < slices; ++s) x += os[(size_t)s * A.nq * D + i];
+        os[i] = x;
+    }
+    mc_barrier();
+    const int width = A.nq * D, slice = ((width + C - 1) / C + 3) & ~3;
+    for (int i = rank * slice + 4 * tid; i < min(width, (rank + 1) * slice); i += 4 * MC_THREADS) {
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        float4 x[16];                                        // every block's share on its way before the first addition
+#pragma unroll
+        for (int s = 0; s < 16; ++s) if (s < C) x[s] = mc_load4(mc_peer(os + i, s));
+#pragma unroll
+        for (int s = 0; s < 16; ++s) if (s < C) { v.x += x[s].x; v.y += x[s].y; v.z += x[s].z; v.w += x[s].w; }
+        uint2 o;
+        o.x = pack_bf16(v.x, v.y); o.y = pack_bf16(v.z, v.w);
+        *reinterpret_cast<uint2*>(A.out + row * width + i) = o;
+    }
+    mc_barrier();                                            // nobody leaves while its shared memory is still read
+}
+
 template <typename K>
 int raise_smem(K kernel, int bytes, bool (&done)[TL_MAX_DEVICES]) {
     const int dev = tl_device_index();
@@ -946,4 +1153,52 @@ TL_EXPORT int tl_mix_decode(const void* q, int q_stride, void* out, const void* 
 #undef MDV
     if (e || splits == 1) return e;
     return launch_after_wait(mix_decode_sum_kernel, dim3((nq * D / 4 + 127) / 128, n), dim3(128), 0, stream, A);
+}
+
+template <int MT>
+static int launch_decode_cluster(const MixDecodeArgs& A, const MixClusterShape& Sh, int n, int clusters, cudaStream_t stream) {
+    constexpr int most = 220 * 1024;
+    const int g = A.nq / A.nkv, smem = mc_bytes(A.nq, A.nkv * ((g + 15) / 16), Sh);
+    if (smem > most) return 2;
+    static bool done[TL_MAX_DEVICES] = {}, wide[TL_MAX_DEVICES] = {};
+    int e = raise_smem(mix_decode_cluster_kernel<MT>, most, done);
+    if (e) return e;
+    const int dev = tl_device_index();
+    if (clusters > 8 && !wide[dev]) {                        // clusters of 9 to 16 blocks
+        const cudaError_t ce = cudaFuncSetAttribute(mix_decode_cluster_kernel<MT>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+        if (ce != cudaSuccess) return (int)ce;
+        wide[dev] = true;
+    }
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(clusters, n); cfg.blockDim = dim3(MC_THREADS); cfg.dynamicSmemBytes = smem; cfg.stream = stream;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = (unsigned)clusters; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = 1;
+    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = tl_dependent_launch_enabled() ? 2 : 1;
+    const cudaError_t ce = cudaLaunchKernelEx(&cfg, mix_decode_cluster_kernel<MT>, A, Sh);
+    return ce != cudaSuccess ? (int)ce : (int)cudaGetLastError();
+}
+
+// The same in one launch: `clusters` (1 to 16) blocks a request form a cluster, none reads more than `most_keys` keys (a multiple of
+// 32, clusters * most_keys >= the longest context).  Returns 2 if the weights of that many keys do not fit the shared memory.
+TL_EXPORT int tl_mix_decode_cluster(const void* q, int q_stride, void* out, const void* k_pages, const void* v_pages, const int* table,
+                                    int max_pages, int page_size, const int* rows, const int* start_pos, const int* slots, int n, int nq,
+                                    int nkv, float scale, int clusters, int most_keys, const void* mix, int hp, int table_rows,
+                                    int total_pages, int* fault, cudaStream_t stream) {
+    if (n <= 0) return 0;
+    if (nq < 1 || nq > 64 || nq % nkv || hp < nq || hp % 16 || page_size < 1 || page_size > 64 || (page_size & (page_size - 1)) ||
+        (q_stride & 7) || clusters < 1 || clusters > 16 || most_keys < 32 || most_keys % 32 || n > 65535) return 1;
+    const MixDecodeArgs A{(const bf16*)q, q_stride, (bf16*)out, (const bf16*)k_pages, (const bf16*)v_pages, table, max_pages, page_size, rows,
+                          start_pos, slots, nq, nkv, scale * 1.4426950408889634f, 0, 0, nullptr, nullptr, nullptr, (const bf16*)mix, hp,
+                          0, 0, TlLimits{table_rows, total_pages, fault}};
+    const MixClusterShape Sh{most_keys + 4, most_keys / page_size + 2};
+    switch ((nq + 15) / 16) {
+        case 1: return launch_decode_cluster<1>(A, Sh, n, clusters, stream);
+        case 2: return launch_decode_cluster<2>(A, Sh, n, clusters, stream);
+        case 3: return launch_decode_cluster<3>(A, Sh, n, clusters, stream);
+        default: return launch_decode_cluster<4>(A, Sh, n, clusters, stream);
+    }
 }

@@ -81,7 +81,8 @@ def load_model(folder, rt: Runtime):
     expected = model.expected_tensors()
     if model.spec.tie_word_embeddings:
         # A tied head is the embedding table: a stored head is neither loaded nor an error.
-        head = tuple(model.head.expected_tensors(model.spec.head_prefix))
+        own = model.head.expected_tensors(model.spec.head_prefix)
+        head = (f"{model.spec.head_prefix}.weight",) + tuple(n for n, spec in own.items() if spec.optional)
         expected = {k: v for k, v in expected.items() if k not in head}
         weights = load_weights(folder, expected, device=rt.device, ignore=head)
     else:

@@ -22,7 +22,7 @@ HEAD_MULTIPLE = 64                  # head sizes the kernels are compiled for: m
 MAX_HEADS = 64
 ROW_TILE, KEY_TILE = 128, 64
 SCRATCH_BYTES = int(os.environ.get("TENSORLINE_B200_MIX_SCRATCH_MB", 512)) << 20      # score and weight tiles of one launch, at most
-DECODE_MAX_RANGE = 512              # keys a decode block, at most (its weights of all heads lie in shared memory)
+DECODE_MAX_RANGE = 256              # keys a block of the kernels over ranges, at most (they take up to 512; longer was slower)
 
 
 def lib(head_dim: int):
@@ -36,6 +36,8 @@ def lib(head_dim: int):
         l.tl_mix_prefill.restype = ctypes.c_int
         l.tl_mix_decode.argtypes = [_P, _I, _P, _P, _P, _P, _I, _I, _P, _P, _P, _I, _I, _I, _F, _I, _I, _P, _P, _P, _P, _I, _I, _I, _P, _P]
         l.tl_mix_decode.restype = ctypes.c_int
+        l.tl_mix_decode_cluster.argtypes = [_P, _I, _P, _P, _P, _P, _I, _I, _P, _P, _P, _I, _I, _I, _F, _I, _I, _P, _I, _I, _I, _P, _P]
+        l.tl_mix_decode_cluster.restype = ctypes.c_int
         if l.tl_mix_max_parts() != MAX_PARTS or any(l.tl_mix_parts(n) != parts_of(n) for n in (1, 8, 9, 128, 129, 1000, 5000)):
             raise KernelError("the mixed-head attention library cuts key tiles into other runs than its launcher")
         _libs[head_dim] = l
@@ -136,14 +138,51 @@ def decode(q, out, k_pages, v_pages, table, page_size, rows, start_pos, slots, n
            "mix_decode", launches=3 if splits > 1 else 2)
 
 
+def plan_cluster(n: int, nq: int, nkv: int, d: int, span: int, sms: int | None = None) -> int:
+    """Blocks a request of the one-launch decode kernel, or 0 where the kernels over ranges serve better: long contexts and many KV
+    heads, which want every SM.  The two estimates (microseconds) are fits of measurements at 148 SMs: the cluster kernel 12 and
+    0.04 a key a block of 512 values (a third more where every head has keys of its own), the others 24 and the cache's bytes at
+    4.5 TB/s; n = 8, 4 KV heads of 128, 2,304 keys: 23 against 30; 64 requests: 61 against 107; 8 requests of 16 KV heads of 64 at
+    4,096 keys: 62 against 43."""
+    sms = sms or ops.num_sms()
+    # as many blocks as run at once, one an SM: six clusters of sixteen fit this GPU, twelve of eight (measured, 148 SMs)
+    clusters = next((c for c, most in ((16, sms // 24), (8, sms // 12), (4, sms // 4), (2, sms // 2)) if n <= most), 1)
+    keys = -(-span // clusters)
+    one = 12.0 + 0.04 * keys * nkv * d / 512 * (1.3 if nkv == nq else 1.0)
+    three = 24.0 + 4.0 * n * span * nkv * d / 4.5e6
+    return clusters if keys * nq <= 36 * 1024 and one <= 1.2 * three else 0
+
+
+def decode_cluster(q, out, k_pages, v_pages, table, page_size, rows, start_pos, slots, n, nq, nkv, d, scale, mix, clusters, span) -> bool:
+    """`decode` in one launch, `clusters` blocks a request; `span`: the most keys a request reads.  False: nothing launched (the
+    keys' weights do not fit the shared memory)."""
+    most = -(-(-(-span // clusters)) // 32) * 32
+    rc = lib(d).tl_mix_decode_cluster(_ptr(q), q.shape[1], _ptr(out), _ptr(k_pages), _ptr(v_pages), _ptr(table), table.shape[1], page_size,
+                                      _ptr(rows), _ptr(start_pos), _ptr(slots), n, nq, nkv, float(scale), clusters, most, _ptr(mix),
+                                      mix.shape[0], table.shape[0], k_pages.shape[0], ops.fault_words(q.device), _stream())
+    if rc == 2:
+        return False
+    _check(rc, "mix_decode+cluster")
+    return True
+
+
+def _decode(q, out, k_pages, v_pages, table, page_size, rows, start_pos, slots, n, nq, nkv, d, scale, mix, span) -> None:
+    args = (q, out, k_pages, v_pages, table, page_size, rows, start_pos, slots, n, nq, nkv, d, scale, mix)
+    clusters = plan_cluster(n, nq, nkv, d, span)
+    if not (CLUSTER and clusters and decode_cluster(*args, clusters, span)):
+        decode(*args, *plan_ranges(n, nkv, nq // nkv, d, span))
+
+
+CLUSTER = os.environ.get("TENSORLINE_B200_MIX_CLUSTER", "1") != "0"      # 0: the kernels over ranges only (A/B timing)
+
+
 def attend(qkv, o, ctx, k_pages, v_pages, table, nq, nkv, d, scale, mix) -> None:
     """A step's attention: single tokens through the decode kernels, portions through the prompt kernels."""
     if qkv.dtype != torch.bfloat16 or k_pages.dtype != torch.bfloat16 or mix.dtype != torch.bfloat16:
         raise KernelError("mixed-head attention: bfloat16 tensors only")
     args = (k_pages, v_pages, table, ctx.page_size)
     if ctx.decode_only:
-        rng, splits = plan_ranges(ctx.B, nkv, nq // nkv, d, ctx.graph_max_ctx or ctx.max_ctx)
-        decode(qkv, o, *args, ctx.q_start, ctx.start_pos, ctx.slots, ctx.B, nq, nkv, d, scale, mix, rng, splits)
+        _decode(qkv, o, *args, ctx.q_start, ctx.start_pos, ctx.slots, ctx.B, nq, nkv, d, scale, mix, ctx.graph_max_ctx or ctx.max_ctx)
         return
     units = max(1, SCRATCH_BYTES // (nq * ROW_TILE * KEY_TILE * 6))
     key = ("mix_tiles", units)
@@ -161,7 +200,6 @@ def attend(qkv, o, ctx, k_pages, v_pages, table, nq, nkv, d, scale, mix) -> None
     launches, singles = ctx.scratch[key]
     if singles:
         packed, n, span = singles
-        rng, splits = plan_ranges(n, nkv, nq // nkv, d, span)
-        decode(qkv, o, *args, packed[0], packed[1], packed[2], n, nq, nkv, d, scale, mix, rng, splits)
+        _decode(qkv, o, *args, packed[0], packed[1], packed[2], n, nq, nkv, d, scale, mix, span)
     if launches:
         prefill(qkv, o, *args, ctx.q_start, ctx.start_pos, ctx.slots, launches, nq, nkv, d, scale, mix)

@@ -83,7 +83,14 @@ def test_row_tiles_of_prompt_portions():
 @pytest.mark.parametrize("n,nkv,group,d,span", [(1, 4, 4, 128, 2304), (8, 4, 4, 128, 2304), (64, 16, 1, 64, 9000), (1, 1, 1, 64, 1), (2, 2, 3, 256, 131072)])
 def test_ranges_of_a_decode_step_cover_the_keys(n, nkv, group, d, span):
     rng, splits = plan_ranges(n, nkv, group, d, span, sms=148)
-    assert rng % 64 == 0 and 64 <= rng <= 512 and rng * splits >= span > rng * (splits - 1)
+    assert rng % 64 == 0 and 64 <= rng <= 256 and rng * splits >= span > rng * (splits - 1)
+
+
+def test_blocks_of_a_request_in_the_one_launch_decode():
+    from tensorline_b200.ops_attention_mix import plan_cluster
+    assert [plan_cluster(n, 16, 4, 128, 2304, sms=148) for n in (1, 6, 7, 12, 13, 37, 38, 74)] == [16, 16, 8, 8, 4, 4, 2, 2]
+    assert plan_cluster(8, 16, 16, 64, 4096, sms=148) == 0     # every head its own keys, four thousand of them: every SM is wanted
+    assert plan_cluster(1, 64, 8, 128, 65536, sms=148) == 0    # the weights would not fit
 
 
 @pytest.mark.parametrize("path,value,word", [

@@ -281,6 +281,12 @@ def test_attention_with_mixed_weights(case, kernel):
             out.fill_(float("nan"))
             om.decode(qkv, out, kd, vd, table, ps, *where, B, nq, nkv, d, scale, pad, rng, -(-span // rng))
             assert_close(out.view(T, nq, d), W, f"{kernel}, ranges of {rng}", **BF16)
+        for clusters in (1, 3, 8, 16):                         # one launch; contexts shorter than a block's run leave blocks without keys
+            out.fill_(float("nan"))
+            if om.decode_cluster(qkv, out, kd, vd, table, ps, *where, B, nq, nkv, d, scale, pad, clusters, span + 70):
+                assert_close(out.view(T, nq, d), W, f"{kernel}, clusters of {clusters}", **BF16)
+            else:
+                assert nq * span > 8192 * clusters
     else:                                                      # the step's own choice of kernels
         ctx = SimpleNamespace(B=B, T=T, decode_only=all(n == 1 for n in step_lens), page_size=ps, q_start=where[0], start_pos=where[1],
                               slots=where[2], h_q_start=q_start, h_start_pos=list(ctx_lens), h_slots=list(range(B)), graph_max_ctx=0,
