@@ -25,7 +25,7 @@ them point at the sink); groups may have pools of different sizes.
 """
 from __future__ import annotations
 
-from dataclasses import dataclass, field
+from dataclasses import dataclass, field, replace
 
 import numpy as np
 
@@ -52,6 +52,17 @@ class PagedKV:
         if self.chunk is not None:
             return ("paged_kv", None, 0, self.chunk)
         return ("paged_kv", self.window, self.keep_first if self.window is not None else 0)
+
+    def widened(self, other: "PagedKV") -> "PagedKV":
+        """This need with the keys that `other`'s queries, which read the same cache, can see: the wider window, everything
+        where one of the two sees everything or the two cut the sequence in different ways."""
+        if (self.num_kv_heads, self.head_dim, self.shared_values) != (other.num_kv_heads, other.head_dim, other.shared_values):
+            raise ValueError(f"a cache of {self} cannot be read as {other}")
+        if self.group_key == other.group_key:
+            return self
+        if self.window is None or other.window is None:
+            return replace(self, window=None, chunk=None, keep_first=0)
+        return replace(self, window=max(self.window, other.window), keep_first=max(self.keep_first, other.keep_first))
 
 
 @dataclass(frozen=True)

@@ -93,6 +93,7 @@ struct AttnArgs {
     int seg;                           // > 0 (instead of a window): a query reads the keys of its own segment of `seg` positions
                                        // only, segments counted from position 0
     const float* slopes;               // [nq] or null: the score of key j seen from position p loses slopes[h] * (p - j)
+    float cap_in, cap_out;             // kernels with CAP: scores become cap_out tanh(dot * cap_in), in units of log2 e (see tl_cap_scores)
 };
 
 // First key a query at position `pos` reads: the start of its segment, of its window, or 0.
@@ -250,10 +251,16 @@ __device__ __forceinline__ float fast_exp2(float x) {          // 2^x, hardware 
 // running max m[2] (kept in scaled units), the per-thread partial sums l[2] and rescales O.
 // key0: position of S column 0.  MASKED = false: the caller knows every key of the tile is visible
 // to every row of the warp, and the comparisons are skipped.
-template <int NB, bool MASKED>
+// CAP: the scores pass cap * tanh(. / cap) first (slopes, if any, come off the capped score).
+template <int NB, bool MASKED, bool CAP = false>
 __device__ __forceinline__ void softmax_step(float (&s)[NB][4], float (&o)[D / 8][4], float (&m)[2], float (&l)[2],
                                              const int (&pos_r)[2], const int (&lo_r)[2], int key0, float scale_log2,
-                                             int lane, int keep = 0, const float* slope_r = nullptr) {
+                                             int lane, int keep = 0, const float* slope_r = nullptr,
+                                             float cap_in = 0.f, float cap_out = 0.f) {
+    if constexpr (CAP) {
+        tl_cap_scores(reinterpret_cast<float(&)[NB * 4]>(s), cap_in, cap_out);
+        scale_log2 = 1.0f;
+    }
     // slope_r (two numbers, in units of log2 e; null: none): row r's score of key j loses slope_r[r] * (pos_r[r] - j).  The
     // scores are then scaled here, before the maximum is taken, and the exponentials below take them as they are.
     float mx[2] = {-INFINITY, -INFINITY};
@@ -303,7 +310,7 @@ __device__ __forceinline__ void softmax_step(float (&s)[NB][4], float (&o)[D / 8
 // ------------------------------------------------------------------------------------ prefill
 // PBN: keys per tile.  32 leaves room for three blocks per SM (more warps to hide the latencies of the
 // MMA / ldmatrix chains); 64 serves pages of 64 tokens.
-template <int PBN>
+template <int PBN, bool CAP>
 __global__ void __launch_bounds__(128) attn_prefill_kernel(const AttnArgs A) {
     constexpr int BN = PBN;                                // shadows the decode tile size inside this kernel
     extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -401,8 +408,8 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const AttnArgs A) {
         // every row's window
         const bool full = (kt * BN + BN - 1 <= sp + wr_first / g) &&
                           (kt * BN >= tl_first_key(A, w_pos_hi) || kt * BN + BN <= keep);
-        if (full) softmax_step<BN / 8, false>(s, o, m, l, pos_r, lo_r, kt * BN, A.scale_log2, lane, 0, slope_p);
-        else      softmax_step<BN / 8, true>(s, o, m, l, pos_r, lo_r, kt * BN, A.scale_log2, lane, keep, slope_p);
+        if (full) softmax_step<BN / 8, false, CAP>(s, o, m, l, pos_r, lo_r, kt * BN, A.scale_log2, lane, 0, slope_p, A.cap_in, A.cap_out);
+        else      softmax_step<BN / 8, true, CAP>(s, o, m, l, pos_r, lo_r, kt * BN, A.scale_log2, lane, keep, slope_p, A.cap_in, A.cap_out);
         pv_tile<BN / 8>(o, s, sV + buf * BN * DP, 0, lane);
     }
     cp_async_wait<0>();
@@ -434,6 +441,7 @@ constexpr int DECODE_TAB_OFFSET = 16 * DP * 2 + (DECODE_KV_SMEM > DECODE_MERGE_S
 constexpr int DECODE_MAX_TAB = 1024;                    // table entries a block may copy (4 KB: head size 256 leaves no more)
 
 // grid (splits * m_tiles, nkv, B); 4 warps; each stage is 64 keys, 16 per warp.
+template <bool CAP>
 __global__ void __launch_bounds__(128) attn_decode_kernel(const AttnArgs A) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     bf16* sQ = reinterpret_cast<bf16*>(smem_raw);          // [16][DP]
@@ -528,8 +536,8 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const AttnArgs A) {
 #pragma unroll
         for (int nb = 0; nb < 2; ++nb) { s[nb][0] = s[nb][1] = s[nb][2] = s[nb][3] = 0.f; }
         qk_tile_regs<2>(s, qf, sK + buf * BN * DP, warp * 16, lane);
-        if (key0 + 16 <= len && (key0 >= lo || key0 + 16 <= keep)) softmax_step<2, false>(s, o, m, l, pos_r, lo_r, key0, A.scale_log2, lane, 0, slope_p);
-        else softmax_step<2, true>(s, o, m, l, pos_r, lo_r, key0, A.scale_log2, lane, keep, slope_p);
+        if (key0 + 16 <= len && (key0 >= lo || key0 + 16 <= keep)) softmax_step<2, false, CAP>(s, o, m, l, pos_r, lo_r, key0, A.scale_log2, lane, 0, slope_p, A.cap_in, A.cap_out);
+        else softmax_step<2, true, CAP>(s, o, m, l, pos_r, lo_r, key0, A.scale_log2, lane, keep, slope_p, A.cap_in, A.cap_out);
         pv_tile<2>(o, s, sV + buf * BN * DP, warp * 16, lane);
     }
     cp_async_wait<0>();
@@ -653,7 +661,7 @@ __device__ __forceinline__ float* cluster_peer_rw(float* p, int rank) {
 // partial results through distributed shared memory (every block finishes a slice of the head dimension), so
 // nothing goes through global memory and no combine kernel follows.  Needs 2 to 8 key ranges and at most 16
 // query heads per KV head (one row tile).  A block whose key range is empty takes part with weight zero.
-template <bool CLUSTER>
+template <bool CLUSTER, bool CAP>
 __global__ void __launch_bounds__(TMA_DEC_THREADS)
 attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                        const AttnArgs A, int* status) {
@@ -847,8 +855,8 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
             mma_bf16(s[0], qf[kb], bfr[0], bfr[1]);
             mma_bf16(s[1], qf[kb], bfr[2], bfr[3]);
         }
-        if (key0 + 16 <= k_end && key0 >= lo) softmax_step<2, false>(s, o, m, l, pos_r, lo_r, key0, A.scale_log2, lane);
-        else                                  softmax_step<2, true>(s, o, m, l, pos_r, lo_r, key0, A.scale_log2, lane);
+        if (key0 + 16 <= k_end && key0 >= lo) softmax_step<2, false, CAP>(s, o, m, l, pos_r, lo_r, key0, A.scale_log2, lane, 0, nullptr, A.cap_in, A.cap_out);
+        else                                  softmax_step<2, true, CAP>(s, o, m, l, pos_r, lo_r, key0, A.scale_log2, lane, 0, nullptr, A.cap_in, A.cap_out);
         uint32_t a[4];
         a[0] = pack_bf16(s[0][0], s[0][1]); a[1] = pack_bf16(s[0][2], s[0][3]);
         a[2] = pack_bf16(s[1][0], s[1][1]); a[3] = pack_bf16(s[1][2], s[1][3]);
@@ -1051,12 +1059,14 @@ int set_attrs() {
     const int dev = tl_device_index();
     if (dev < 0) return 1;
     if (g_attr_done[dev]) return 0;
-    cudaError_t e = cudaFuncSetAttribute(attn_prefill_kernel<32>, cudaFuncAttributeMaxDynamicSharedMemorySize, prefill_smem<32>());
-    if (e != cudaSuccess) return (int)e;
-    e = cudaFuncSetAttribute(attn_prefill_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, prefill_smem<64>());
-    if (e != cudaSuccess) return (int)e;
-    e = cudaFuncSetAttribute(attn_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, DECODE_SMEM_MAX);
-    if (e != cudaSuccess) return (int)e;
+    const struct { const void* kernel; int smem; } all[] = {
+        {(const void*)attn_prefill_kernel<32, false>, prefill_smem<32>()}, {(const void*)attn_prefill_kernel<32, true>, prefill_smem<32>()},
+        {(const void*)attn_prefill_kernel<64, false>, prefill_smem<64>()}, {(const void*)attn_prefill_kernel<64, true>, prefill_smem<64>()},
+        {(const void*)attn_decode_kernel<false>, DECODE_SMEM_MAX}, {(const void*)attn_decode_kernel<true>, DECODE_SMEM_MAX}};
+    for (const auto& k : all) {
+        const cudaError_t e = cudaFuncSetAttribute(k.kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, k.smem);
+        if (e != cudaSuccess) return (int)e;
+    }
     g_attr_done[dev] = true;
     return 0;
 }
@@ -1078,6 +1088,12 @@ TL_EXPORT int tl_attn_set_keep_first(int keep_first) { g_keep_first = keep_first
 static int g_seg = 0;
 static const float* g_slopes = nullptr;
 TL_EXPORT int tl_attn_set_distance(int seg, const float* slopes) { g_seg = seg > 0 ? seg : 0; g_slopes = slopes; return 0; }
+// A cap on the scores of the launches that follow, cap * tanh(score / cap); 0: none.  Set before every launch.
+static float g_cap = 0.f;
+TL_EXPORT int tl_attn_set_cap(float cap) { g_cap = cap > 0.f ? cap : 0.f; return 0; }
+namespace {
+void take_cap(AttnArgs& A, float scale) { if (g_cap > 0.f) { A.cap_in = scale / g_cap; A.cap_out = g_cap * LOG2E; } }
+}
 // 1 if this library was compiled as the checking build (-DTL_CHECK=1).
 TL_EXPORT int tl_check_build() { return TL_CHECKING; }
 // Block-table entries a decode block may copy: chunk / page_size of a decode call may not exceed it.
@@ -1107,8 +1123,14 @@ TL_EXPORT int tl_attn_prefill(const void* q, int q_stride, void* out, const void
     A.q_start = q_start; A.start_pos = start_pos; A.slots = slots;
     A.B = B; A.nq = nq; A.nkv = nkv; A.window = window; A.scale_log2 = scale * LOG2E;
     dim3 grid((unsigned)total_tiles * (unsigned)nkv);
-    if (page_size <= 32) attn_prefill_kernel<32><<<grid, 128, prefill_smem<32>(), stream>>>(A);
-    else                 attn_prefill_kernel<64><<<grid, 128, prefill_smem<64>(), stream>>>(A);
+    take_cap(A, scale);
+    if (g_cap > 0.f) {
+        if (page_size <= 32) attn_prefill_kernel<32, true><<<grid, 128, prefill_smem<32>(), stream>>>(A);
+        else                 attn_prefill_kernel<64, true><<<grid, 128, prefill_smem<64>(), stream>>>(A);
+    } else {
+        if (page_size <= 32) attn_prefill_kernel<32, false><<<grid, 128, prefill_smem<32>(), stream>>>(A);
+        else                 attn_prefill_kernel<64, false><<<grid, 128, prefill_smem<64>(), stream>>>(A);
+    }
     return tl_launch_status();
 }
 
@@ -1141,7 +1163,8 @@ TL_EXPORT int tl_attn_decode(const void* q, int q_stride, void* out, const void*
     if (grid.z > 65535) return 1;
     const int tab_entries = chunk / page_size;            // of the longest range a block can have
     if (tab_entries > DECODE_MAX_TAB) return 1;
-    e = launch_after_wait(attn_decode_kernel, grid, dim3(128), DECODE_TAB_OFFSET + tab_entries * 4, stream, A);
+    take_cap(A, scale);
+    e = launch_after_wait(g_cap > 0.f ? attn_decode_kernel<true> : attn_decode_kernel<false>, grid, dim3(128), DECODE_TAB_OFFSET + tab_entries * 4, stream, A);
     if (e || splits == 1) return e;
     dim3 cgrid(nq, B);
     return launch_after_wait(attn_combine_kernel, cgrid, dim3(D < 128 ? ((D + 31) / 32) * 32 : 128), 0, stream, A);
@@ -1204,14 +1227,16 @@ int decode_tma_impl(const void* q, int q_stride, void* out, const void* k_pages,
     const int dev_index = tl_device_index();
     if (dev_index < 0) return 1;
     if (!g_tma_attr_done[dev_index]) {
-        cudaError_t ce = cudaFuncSetAttribute(attn_decode_tma_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                              tma_tab_offset(TMA_MAX_RANGES) + DECODE_MAX_TAB * 4 + 1024);
-        if (ce == cudaSuccess)
-            ce = cudaFuncSetAttribute(attn_decode_tma_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                      tma_tab_offset(TMA_MAX_RANGES) + DECODE_MAX_TAB * 4 + 1024);
-        if (ce == cudaSuccess)                             // clusters of 9 to 16 blocks
-            ce = cudaFuncSetAttribute(attn_decode_tma_kernel<true>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
-        if (ce != cudaSuccess) return (int)ce;
+        const struct { const void* kernel; bool cluster; } all[] = {
+            {(const void*)attn_decode_tma_kernel<false, false>, false}, {(const void*)attn_decode_tma_kernel<true, false>, true},
+            {(const void*)attn_decode_tma_kernel<false, true>, false}, {(const void*)attn_decode_tma_kernel<true, true>, true}};
+        for (const auto& k : all) {
+            cudaError_t ce = cudaFuncSetAttribute(k.kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                                  tma_tab_offset(TMA_MAX_RANGES) + DECODE_MAX_TAB * 4 + 1024);
+            if (ce == cudaSuccess && k.cluster)            // clusters of 9 to 16 blocks
+                ce = cudaFuncSetAttribute(k.kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+            if (ce != cudaSuccess) return (int)ce;
+        }
         g_tma_attr_done[dev_index] = true;
     }
     int e = set_attrs();                                   // the combine kernel's library state
@@ -1230,6 +1255,7 @@ int decode_tma_impl(const void* q, int q_stride, void* out, const void* k_pages,
     A.chunk = chunk; A.splits = splits; A.part_o = part_o; A.part_ml = part_ml;
     A.lim = TlLimits{table_rows, (int)total_pages, fault};
     A.rope_inv_freq = R.inv_freq; A.rope_bias = R.bias; A.rope_bias_f32 = R.bias_f32; A.rope_write = R.write_kv;
+    take_cap(A, scale);
     A.trace = g_trace.take((unsigned)(splits * ((nq / nkv + 15) / 16) * nkv * B));
     A.k_pages_w = (bf16*)const_cast<void*>(k_pages); A.v_pages_w = (bf16*)const_cast<void*>(v_pages);
     const int g = nq / nkv, m_tiles = (g + 15) / 16;
@@ -1245,10 +1271,10 @@ int decode_tma_impl(const void* q, int q_stride, void* out, const void* k_pages,
         attr[1].val.programmaticStreamSerializationAllowed = 1;
         cfg.attrs = attr;
         cfg.numAttrs = tl_dependent_launch_enabled() ? 2 : 1;
-        const cudaError_t ce = cudaLaunchKernelEx(&cfg, attn_decode_tma_kernel<true>, mk, mv, A, status);
+        const cudaError_t ce = cudaLaunchKernelEx(&cfg, g_cap > 0.f ? attn_decode_tma_kernel<true, true> : attn_decode_tma_kernel<true, false>, mk, mv, A, status);
         return ce != cudaSuccess ? (int)ce : tl_launch_status();
     }
-    e = launch_after_wait(attn_decode_tma_kernel<false>, grid, dim3(TMA_DEC_THREADS), (size_t)smem, stream, mk, mv, A, status);
+    e = launch_after_wait(g_cap > 0.f ? attn_decode_tma_kernel<false, true> : attn_decode_tma_kernel<false, false>, grid, dim3(TMA_DEC_THREADS), (size_t)smem, stream, mk, mv, A, status);
     if (e || splits == 1) return e;
     dim3 cgrid(nq, B);
     return launch_after_wait(attn_combine_kernel, cgrid, dim3(D < 128 ? ((D + 31) / 32) * 32 : 128), 0, stream, A);
@@ -1375,7 +1401,7 @@ TL_EXPORT int tl_attn_decode_static(const void* q, int q_stride, void* out, cons
     const int g = nq / nkv, m_tiles = (g + 15) / 16;
     dim3 grid(splits * m_tiles, nkv, B);
     if (grid.z > 65535) return fail(err, err_len, 7, "tl_attn_decode_static: more than 65535 requests in one call");
-    attn_decode_kernel<<<grid, 128, DECODE_TAB_OFFSET + tab_entries * 4, stream>>>(A);
+    attn_decode_kernel<false><<<grid, 128, DECODE_TAB_OFFSET + tab_entries * 4, stream>>>(A);
     ce = cudaGetLastError();
     if (ce == cudaSuccess && splits > 1) {
         dim3 cgrid(nq, B);

@@ -75,6 +75,7 @@ struct TcAttnArgs {
     // slopes[h] * (p - j).
     int seg;
     const float* slopes;
+    float cap_in, cap_out;             // kernels with CAP: scores become cap_out tanh(dot * cap_in), in units of log2 e (see tl_cap_scores)
 };
 
 // First key a query at position `pos` reads: the start of its segment, of its window, or 0.
@@ -135,6 +136,8 @@ __device__ __forceinline__ void load_kv(uint32_t dst, const bf16* pages, const i
     }
 }
 
+// CAP: the scores pass cap * tanh(. / cap) before the mask (slopes, if any, come off the capped score).
+template <bool CAP>
 __global__ void __launch_bounds__(THREADS, 1) attn_tc_prefill_kernel(const TcAttnArgs A) {
     extern __shared__ unsigned char smem_raw[];
     unsigned char* base = reinterpret_cast<unsigned char*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
@@ -203,7 +206,7 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tc_prefill_kernel(const TcAtt
         // with distance slopes the scores are scaled where the slope is taken off, and the exponentials take them as they are
         const bool biased = A.slopes != nullptr;
         const float slope_r = (biased && R < rows_total) ? A.slopes[kh * g + R % g] * LOG2E : 0.f;
-        const float sc = biased ? 1.0f : A.scale_log2;
+        const float sc = biased || CAP ? 1.0f : A.scale_log2;
         const uint32_t lane_addr = tmem + ((uint32_t)(warp * 32) << 16);
         float m_ref = -INFINITY, l = 0.f;
         bool ok = true;
@@ -225,9 +228,11 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tc_prefill_kernel(const TcAtt
                 tmem_ld32(lane_addr + S_COL + sl * BN + c0, reinterpret_cast<float(&)[32]>(s[c0]));
             tmem_ld_wait();                                 // all parts in flight, one wait
             const int key0 = kt * BN;
+            if constexpr (CAP) tl_cap_scores(s, A.cap_in, A.cap_out);
             if (biased) {
+                const float pre = CAP ? 1.0f : A.scale_log2;
 #pragma unroll
-                for (int c = 0; c < BN; ++c) s[c] = fmaf(s[c], A.scale_log2, -slope_r * (float)(pos_r - (key0 + c)));
+                for (int c = 0; c < BN; ++c) s[c] = fmaf(s[c], pre, -slope_r * (float)(pos_r - (key0 + c)));
             }
             if (!(key0 + BN - 1 <= pos_r && (key0 >= lo_r || key0 + BN <= keep))) {   // not every key of the tile is visible to this row
 #pragma unroll
@@ -435,7 +440,8 @@ __device__ __forceinline__ void tmem_st32_nowait(uint32_t taddr, const uint32_t 
 // (32 of the slot's 64 columns), and O += P V takes P as its tensor-memory operand.  A key-tile step then moves 160 KB
 // through shared memory instead of 224 KB (the bound of this kernel: see the notes above).  The S slot of product i is
 // free again when P(i) V is complete, not when the softmax has read S(i): that is what the S issuer then waits for.
-template <bool P_TMEM>
+// CAP: the scores pass cap * tanh(. / cap) before the mask.
+template <bool P_TMEM, bool CAP>
 __global__ void __launch_bounds__(THREADS2, 1)
 attn_tc2_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, const TcAttnArgs A) {
     extern __shared__ unsigned char smem_raw[];
@@ -525,6 +531,7 @@ attn_tc2_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         const int lo_r = A.window > 0 ? max(0, pos_r - A.window + 1) : 0;
         const uint32_t lane_addr = tmem + ((uint32_t)((warp & 3) * 32) << 16);
         const int n_mine = kt_last[t] - kt_first[t] + 1;   // <= 0: this tile has no rows
+        const float sc = CAP ? 1.0f : A.scale_log2;        // capped scores are in base-2 units already
         // The two warps of a scheduler (one of each query tile) take turns at the exponentials.  Left alone they run
         // in step: both load and reduce (the special-function unit idle), then both want that unit at once, 2,060
         // cycles a key tile where the two phases side by side need 1,300.  Over the key tiles that both query tiles
@@ -555,6 +562,7 @@ attn_tc2_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
             for (int c0 = 0; c0 < BN; c0 += 32)
                 tmem_ld32(s_addr + c0, reinterpret_cast<float(&)[32]>(s[c0]));
             tmem_ld_wait();                                 // all parts in flight, one wait
+            if constexpr (CAP) tl_cap_scores(s, A.cap_in, A.cap_out);
             if (!(key0 + BN - 1 <= pos_r && key0 >= lo_r)) {   // not every key of the tile is visible to this row
 #pragma unroll
                 for (int c = 0; c < BN; ++c) {
@@ -562,7 +570,7 @@ attn_tc2_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
                     if (!(j <= pos_r && j >= lo_r)) s[c] = -INFINITY;
                 }
             }
-            const float mx = row_max(s) * A.scale_log2;
+            const float mx = row_max(s) * sc;
             const bool raise = mx > m_ref + RESCALE_THRESHOLD || (m_ref == -INFINITY && mx != -INFINITY);
             const float m_new = raise ? fmaxf(mx, m_ref) : m_ref;
             const bool fix_o = raise && i > 0 && m_ref != -INFINITY;        // O holds earlier tiles of this row
@@ -600,7 +608,7 @@ attn_tc2_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
                 float p[8];
 #pragma unroll
                 for (int e = 0; e < 8; ++e) {
-                    p[e] = fast_exp2(fmaf(s[j8 * 8 + e], A.scale_log2, -m_use));
+                    p[e] = fast_exp2(fmaf(s[j8 * 8 + e], sc, -m_use));
                     l4[e & 3] += p[e];
                 }
                 if constexpr (P_TMEM) {
@@ -1108,6 +1116,10 @@ TL_EXPORT int tl_attn_set_keep_first(int keep_first) { g_keep_first = keep_first
 static int g_seg = 0;
 static const float* g_slopes = nullptr;
 TL_EXPORT int tl_attn_set_distance(int seg, const float* slopes) { g_seg = seg > 0 ? seg : 0; g_slopes = slopes; return 0; }
+// A cap on the scores of the launches that follow, cap * tanh(score / cap); 0: none.  Set before every launch; the pair kernel
+// with key tiles of 128 turns such a launch down (code 2).
+static float g_cap = 0.f;
+TL_EXPORT int tl_attn_set_cap(float cap) { g_cap = cap > 0.f ? cap : 0.f; return 0; }
 // 1 if this library was compiled as the checking build (-DTL_CHECK=1).
 TL_EXPORT int tl_check_build() { return TL_CHECKING; }
 
@@ -1122,7 +1134,8 @@ TL_EXPORT int tl_attn_tc_prefill(const void* q, int q_stride, void* out, const v
     const int dev = tl_device_index();
     if (dev < 0) return 1;
     if (!g_attr_done[dev]) {
-        cudaError_t e = cudaFuncSetAttribute(attn_tc_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES);
+        cudaError_t e = cudaFuncSetAttribute(attn_tc_prefill_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_tc_prefill_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES);
         if (e != cudaSuccess) return (int)e;
         g_attr_done[dev] = true;
     }
@@ -1138,7 +1151,12 @@ TL_EXPORT int tl_attn_tc_prefill(const void* q, int q_stride, void* out, const v
     A.B = B; A.nq = nq; A.nkv = nkv; A.window = window; A.scale_log2 = scale * LOG2E; A.status = status; A.order = order;
     A.lim = TlLimits{table_rows, total_pages, fault};
     dim3 grid((unsigned)total_tiles * (unsigned)nkv);
-    attn_tc_prefill_kernel<<<grid, THREADS, SMEM_BYTES, stream>>>(A);
+    if (g_cap > 0.f) {
+        A.cap_in = scale / g_cap; A.cap_out = g_cap * LOG2E;
+        attn_tc_prefill_kernel<true><<<grid, THREADS, SMEM_BYTES, stream>>>(A);
+    } else {
+        attn_tc_prefill_kernel<false><<<grid, THREADS, SMEM_BYTES, stream>>>(A);
+    }
     return tl_launch_status();
 }
 
@@ -1190,8 +1208,10 @@ static int tc2_prefill_impl(const void* q, int q_stride, void* out, const void* 
     const int dev = tl_device_index();
     if (dev < 0) return 1;
     if (!g_attr2_done[dev]) {
-        cudaError_t e = cudaFuncSetAttribute(attn_tc2_prefill_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM2_BYTES);
-        if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_tc2_prefill_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM2_BYTES);
+        cudaError_t e = cudaFuncSetAttribute(attn_tc2_prefill_kernel<false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM2_BYTES);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_tc2_prefill_kernel<true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM2_BYTES);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_tc2_prefill_kernel<false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM2_BYTES);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_tc2_prefill_kernel<true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM2_BYTES);
         if (e != cudaSuccess) return (int)e;
         g_attr2_done[dev] = true;
     }
@@ -1211,8 +1231,14 @@ static int tc2_prefill_impl(const void* q, int q_stride, void* out, const void* 
     if (ksplit > 1 && (ksplit > 8 || !part_o || !part_ml || !merge_rows || tokens <= 0 || ((uintptr_t)part_o & 15) || ((uintptr_t)part_ml & 7))) return 1;
     A.ksplit = ksplit > 1 ? ksplit : 1; A.tokens = tokens; A.part_o = part_o; A.part_ml = part_ml;
     dim3 grid((unsigned)total_tiles * (unsigned)nkv * (unsigned)A.ksplit);
-    if (p_tmem) attn_tc2_prefill_kernel<true><<<grid, THREADS2, SMEM2_BYTES, stream>>>(mk, mv, A);
-    else        attn_tc2_prefill_kernel<false><<<grid, THREADS2, SMEM2_BYTES, stream>>>(mk, mv, A);
+    if (g_cap > 0.f) {
+        A.cap_in = scale / g_cap; A.cap_out = g_cap * LOG2E;
+        if (p_tmem) attn_tc2_prefill_kernel<true, true><<<grid, THREADS2, SMEM2_BYTES, stream>>>(mk, mv, A);
+        else        attn_tc2_prefill_kernel<false, true><<<grid, THREADS2, SMEM2_BYTES, stream>>>(mk, mv, A);
+    } else {
+        if (p_tmem) attn_tc2_prefill_kernel<true, false><<<grid, THREADS2, SMEM2_BYTES, stream>>>(mk, mv, A);
+        else        attn_tc2_prefill_kernel<false, false><<<grid, THREADS2, SMEM2_BYTES, stream>>>(mk, mv, A);
+    }
     int rc = tl_launch_status();
     if (rc || A.ksplit == 1 || n_merge_rows <= 0) return rc;
     constexpr int GROUPS = 256 / (D / 4);                  // (token, head) pairs a block of 256 threads
@@ -1268,7 +1294,7 @@ TL_EXPORT int tl_attn_tc3_prefill(const void* q, int q_stride, void* out, const 
                                   int* fault, cudaStream_t stream) {
 #if HEAD_DIM <= 128
     if (total_tiles <= 0 || B <= 0) return 0;
-    if (g_seg > 0 || g_slopes != nullptr) return 2;        // segments and distance slopes: the one-tile kernel
+    if (g_seg > 0 || g_slopes != nullptr || g_cap > 0.f) return 2;     // segments and distance slopes: the one-tile kernel; caps: the pair kernel above
     if (page_size < 8 || page_size > 64 || (page_size & (page_size - 1))) return 2;
     if (((uintptr_t)k_pages & 127) || ((uintptr_t)v_pages & 127)) return 2;
     if (nq % nkv || (q_stride & 7) || ((uintptr_t)q & 15)) return 1;

@@ -11,6 +11,7 @@
 // `gate` (float [T, nq], may be null): the finished row is multiplied by sigmoid(gate[t, h]).
 // `chunk` (> 0, instead of a window): the sequence is cut into chunks of that many positions counted from position 0, and
 // a query reads the keys of its own chunk only: lo = (p / chunk) * chunk.
+// `cap` (> 0): a score is cap * tanh(score / cap) before anything is taken off it.
 // `slopes` (float per query head, may be null): a key's score loses slopes[h] * (p - j), its distance from the query.
 //
 // Keys are taken in tiles of 32 aligned to absolute position 0, each lane owning one key of the
@@ -19,17 +20,16 @@
 // a position is bit-identical under every schedule.
 #include "common.cuh"
 
-#define ATT_MAX_D 512
-
-template <typename TA>
+// MAXD: the widest head the kernel's registers hold (512, or 1024 for the wide ones).
+template <typename TA, int MAXD>
 __global__ void attn_tokenwise_kernel(const TA* __restrict__ q, int q_stride, TA* __restrict__ out,
                                       const TA* __restrict__ k_pages, const TA* __restrict__ v_pages,
                                       const int* __restrict__ table, int max_pages, int page_size,
                                       const int* __restrict__ pos, const int* __restrict__ req_slot,
                                       int nq, int nkv, int d, int window, float scale,
                                       const float* __restrict__ sink, int keep_first, const float* __restrict__ gate,
-                                      int chunk, const float* __restrict__ slopes, const TlLimits L) {
-    __shared__ float qs[ATT_MAX_D];
+                                      int chunk, const float* __restrict__ slopes, float cap, const TlLimits L) {
+    __shared__ float qs[MAXD];
     const int t = blockIdx.x, h = blockIdx.y, lane = threadIdx.x;
     const int kh = h / (nq / nkv);
     const int p = pos[t];
@@ -40,7 +40,7 @@ __global__ void attn_tokenwise_kernel(const TA* __restrict__ q, int q_stride, TA
     for (int e = lane; e < d; e += 32) qs[e] = to_f<TA>(qrow[e]);
     __syncwarp();
 
-    constexpr int MAXC = ATT_MAX_D / 32;
+    constexpr int MAXC = MAXD / 32;
     float acc[MAXC];
 #pragma unroll
     for (int c = 0; c < MAXC; ++c) acc[c] = 0.f;
@@ -61,6 +61,7 @@ __global__ void attn_tokenwise_kernel(const TA* __restrict__ q, int q_stride, TA
             float dot = 0.f;
             for (int e = 0; e < d; ++e) dot = fmaf(qs[e], to_f<TA>(kr[e]), dot);
             s = dot * scale;
+            if (cap > 0.f) s = cap * tanhf(s / cap);
             if (slopes) s -= slope * (float)(p - j);
         }
         const float m_new = fmaxf(m, warp_max(s));
@@ -105,18 +106,16 @@ TL_EXPORT int tl_attn_tokenwise(const void* q, int q_stride, void* out, int act_
                                 const void* k_pages, const void* v_pages, const int* table, int max_pages,
                                 int page_size, const int* pos, const int* req_slot, int T, int nq, int nkv,
                                 int d, int window, float scale, const float* sink, int keep_first, const float* gate,
-                                int chunk, const float* slopes, int table_rows, int total_pages, int* fault, cudaStream_t stream) {
+                                int chunk, const float* slopes, float cap, int table_rows, int total_pages, int* fault, cudaStream_t stream) {
     const TlLimits L{table_rows, total_pages, fault};
     if (T <= 0) return 0;
-    if (d > ATT_MAX_D || nq % nkv || (chunk > 0 && window > 0) || chunk < 0) return 1;
+    if (d > 1024 || nq % nkv || (chunk > 0 && window > 0) || chunk < 0) return 1;
     dim3 grid(T, nq);
-    if (act_dtype == TL_F32)
-        attn_tokenwise_kernel<float><<<grid, 32, 0, stream>>>((const float*)q, q_stride, (float*)out,
-            (const float*)k_pages, (const float*)v_pages, table, max_pages, page_size, pos, req_slot,
-            nq, nkv, d, window, scale, sink, window > 0 ? keep_first : 0, gate, chunk, slopes, L);
-    else
-        attn_tokenwise_kernel<bf16><<<grid, 32, 0, stream>>>((const bf16*)q, q_stride, (bf16*)out,
-            (const bf16*)k_pages, (const bf16*)v_pages, table, max_pages, page_size, pos, req_slot,
-            nq, nkv, d, window, scale, sink, window > 0 ? keep_first : 0, gate, chunk, slopes, L);
+#define TOKENWISE(TA, MAXD) attn_tokenwise_kernel<TA, MAXD><<<grid, 32, 0, stream>>>((const TA*)q, q_stride, (TA*)out, \
+        (const TA*)k_pages, (const TA*)v_pages, table, max_pages, page_size, pos, req_slot, \
+        nq, nkv, d, window, scale, sink, window > 0 ? keep_first : 0, gate, chunk, slopes, cap, L)
+    if (act_dtype == TL_F32) { if (d <= 512) TOKENWISE(float, 512); else TOKENWISE(float, 1024); }
+    else                     { if (d <= 512) TOKENWISE(bf16, 512); else TOKENWISE(bf16, 1024); }
+#undef TOKENWISE
     return tl_launch_status();
 }

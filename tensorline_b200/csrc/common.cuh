@@ -76,6 +76,34 @@ __device__ __forceinline__ float tl_sink_term(const float* __restrict__ sink, in
     return sink ? exp2f(fmaf(sink[head], 1.4426950408889634f, -m)) : 0.f;
 }
 
+// Attention scores with a cap: cap * tanh(score / cap).  For kernels that keep scores in base-2 units; s holds raw dot products,
+// `in` = scale / cap and `out` = cap * log2(e), so s <- out * tanh(s * in).  Where every |s * in| of the warp is at most 1/2
+// (scores up to half the cap, the usual case) tanh(z) is z times a polynomial of degree 3 in z^2 (a least-maximum fit of
+// tanh(z) / z on [0, 1/2], relative error 6e-7), five multiply-adds a score; else 1 - 2 / (1 + e^(2 z)) with the
+// special-function unit's exponential and reciprocal (absolute error about 2e-7).  Called by whole warps.
+template <int N>
+__device__ __forceinline__ void tl_cap_scores(float (&s)[N], float in, float out) {
+    float big = 0.f;
+#pragma unroll
+    for (int i = 0; i < N; ++i) big = fmaxf(big, fabsf(s[i]));
+    if (!__any_sync(0xffffffffu, !(big * in <= 0.5f))) {
+        const float i2 = in * in, c0 = 0.99999945577f * (out * in), c1 = -0.33326317939f * (out * in) * i2,
+                    c2 = 0.13190296634f * (out * in) * i2 * i2, c3 = -0.04440222694f * (out * in) * i2 * i2 * i2;
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+            const float u = s[i] * s[i];
+            s[i] *= fmaf(fmaf(fmaf(c3, u, c2), u, c1), u, c0);
+        }
+    } else {
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+            float e;
+            asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(s[i] * in * 2.885390082f));      // e^(2 z)
+            s[i] = fmaf(-2.0f * out, __fdividef(1.0f, 1.0f + e), out);
+        }
+    }
+}
+
 static inline int tl_launch_status() { return (int)cudaGetLastError(); }
 
 // Host-side state that belongs to a device (kernel attributes that were set, addresses that were looked up) is
@@ -191,6 +219,10 @@ __device__ __forceinline__ float tl_relu_squared_rounded(float v) {
     const float r = fmaxf(__bfloat162float(__float2bfloat16_rn(v)), 0.f);
     return r * r;
 }
+
+// The epilogue activation of a product without a gate: `act` 1: the square of relu, 2: the tanh form of gelu (of the
+// accumulator itself).
+__device__ __forceinline__ float tl_plain_act(float v, int act) { return act == 2 ? tl_gelu_tanh(v) : tl_relu_squared_rounded(v); }
 
 // The clamped swish works on the pair: g' = min(g, limit), u' = clamp(u, -limit, limit); g' sigmoid(alpha g') (u' + 1).
 #define TL_ACT_SWISH_CLAMPED 3

@@ -333,15 +333,15 @@ __global__ void __launch_bounds__(256) post_norm_add_norm_kernel(float* __restri
         ss = fmaf(v, v, ss);
     }
     if (!out) return;
-    ss = block_sum(ss, red);
-    const float rstd = 1.0f / sqrtf(ss / (float)H + eps);
+    float rstd = 1.0f;
+    if (w_pre) { ss = block_sum(ss, red); rstd = 1.0f / sqrtf(ss / (float)H + eps); }
     for (int c = threadIdx.x; c < H; c += blockDim.x) {
         float v = xr[c];
         if (!write_x) {                                  // the same chain of operations as above
             if (a) v += to_f<TA>(a[src + c]) * ra * to_f<TW>(w_post[c]);
             if (extra) v += extra[c];
         }
-        out[(size_t)i * H + c] = from_f<TA>(v * rstd * to_f<TW>(w_pre[c]));
+        out[(size_t)i * H + c] = from_f<TA>(w_pre ? v * rstd * to_f<TW>(w_pre[c]) : v);
     }
 }
 
@@ -411,6 +411,14 @@ __global__ void post_norm_add_norm_vec_kernel(float* __restrict__ x, const TA* _
         }
     }
     if (!out) return;
+    if (!w_pre) {                                            // no second norm: the sum itself, rounded
+#pragma unroll
+        for (int k = 0; k < NV; ++k) {
+            const int c = threadIdx.x + k * blockDim.x;
+            if (c < nvec) Vec4<TA>::store(out + (size_t)i * H + 4 * c, v[k]);
+        }
+        return;
+    }
 #pragma unroll
     for (int k = 0; k < NV; ++k) {                           // the second norm's weights: the first one's are done with
         const int c = threadIdx.x + k * blockDim.x;
@@ -607,25 +615,27 @@ TL_EXPORT int tl_add_rmsnorm_pair(float* x, const void* a, const void* b, const 
 }
 
 // ------------------------------------------------------------------ a sigmoid gate per (token, head) on attention's output
-// o[t, h, :] *= sigmoid(gate[t, h]); gate float [T, nq].
+// o[t, h, :] *= sigmoid(gate[t, h]); gate float, rows of nq numbers `ldg` apart.
 template <typename TA>
-__global__ void head_gate_kernel(TA* __restrict__ o, const float* __restrict__ gate, int d, size_t total) {
+__global__ void head_gate_kernel(TA* __restrict__ o, const float* __restrict__ gate, int ldg, int nq, int d, size_t total) {
     grid_dependency_wait();
     grid_dependency_trigger();
     for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
-        const float g = 1.0f / (1.0f + expf(-gate[idx / d]));
+        const size_t row = idx / d, tok = row / nq;
+        const float g = 1.0f / (1.0f + expf(-gate[tok * ldg + (row - tok * nq)]));
         o[idx] = from_f<TA>(to_f<TA>(o[idx]) * g);
     }
 }
 
 // sixteen bytes a thread (eight bfloat16 or four floats of one head: d is a multiple of that many, o is 16-byte aligned)
 template <typename TA>
-__global__ void head_gate_vec_kernel(TA* __restrict__ o, const float* __restrict__ gate, int vecs_per_head, size_t vecs) {
+__global__ void head_gate_vec_kernel(TA* __restrict__ o, const float* __restrict__ gate, int ldg, int nq, int vecs_per_head, size_t vecs) {
     constexpr int N = 16 / sizeof(TA);
     grid_dependency_wait();
     grid_dependency_trigger();
     for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < vecs; idx += (size_t)gridDim.x * blockDim.x) {
-        const float g = 1.0f / (1.0f + expf(-gate[idx / vecs_per_head]));
+        const size_t row = idx / vecs_per_head, tok = row / nq;
+        const float g = 1.0f / (1.0f + expf(-gate[tok * ldg + (row - tok * nq)]));
         uint4 raw = reinterpret_cast<const uint4*>(o)[idx];
         TA* e = reinterpret_cast<TA*>(&raw);
 #pragma unroll
@@ -634,7 +644,7 @@ __global__ void head_gate_vec_kernel(TA* __restrict__ o, const float* __restrict
     }
 }
 
-TL_EXPORT int tl_head_gate(void* o, int act_dtype, const float* gate, int T, int nq, int d, cudaStream_t stream) {
+TL_EXPORT int tl_head_gate(void* o, int act_dtype, const float* gate, int ldg, int T, int nq, int d, cudaStream_t stream) {
     const size_t total = (size_t)T * nq * d;
     if (total == 0) return 0;
     const size_t cap = (size_t)tl_num_sms() * 16;
@@ -642,12 +652,12 @@ TL_EXPORT int tl_head_gate(void* o, int act_dtype, const float* gate, int T, int
     if (d % per == 0 && (reinterpret_cast<uintptr_t>(o) & 15) == 0) {
         const size_t vecs = total / per;
         const unsigned vb = (unsigned)((vecs + 255) / 256 < cap ? (vecs + 255) / 256 : cap);
-        if (act_dtype == TL_F32) launch_after_wait(head_gate_vec_kernel<float>, dim3(vb), dim3(256), 0, stream, (float*)o, gate, d / per, vecs);
-        else launch_after_wait(head_gate_vec_kernel<bf16>, dim3(vb), dim3(256), 0, stream, (bf16*)o, gate, d / per, vecs);
+        if (act_dtype == TL_F32) launch_after_wait(head_gate_vec_kernel<float>, dim3(vb), dim3(256), 0, stream, (float*)o, gate, ldg, nq, d / per, vecs);
+        else launch_after_wait(head_gate_vec_kernel<bf16>, dim3(vb), dim3(256), 0, stream, (bf16*)o, gate, ldg, nq, d / per, vecs);
         return tl_launch_status();
     }
     const unsigned blocks = (unsigned)((total + 255) / 256 < cap ? (total + 255) / 256 : cap);
-    if (act_dtype == TL_F32) launch_after_wait(head_gate_kernel<float>, dim3(blocks), dim3(256), 0, stream, (float*)o, gate, d, total);
-    else launch_after_wait(head_gate_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, (bf16*)o, gate, d, total);
+    if (act_dtype == TL_F32) launch_after_wait(head_gate_kernel<float>, dim3(blocks), dim3(256), 0, stream, (float*)o, gate, ldg, nq, d, total);
+    else launch_after_wait(head_gate_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, (bf16*)o, gate, ldg, nq, d, total);
     return tl_launch_status();
 }

@@ -128,7 +128,7 @@ struct GemmArgs {
     int gated;            // swap, one split: rows 0..63 of every 128-row tile of A are gate features, rows 64..127 the
                           // up features of the same 64 columns; out[b, 64 tile + j] = silu(gate) * up, [RB, RA / 2]
     float gate_limit, gate_alpha;   // gated = 3: the clamped swish's constants
-    int act;              // swap, bfloat16 out, one split or splits summed in a cluster: out = relu(.)^2
+    int act;              // swap, bfloat16 out, one split or splits summed in a cluster: 1: out = relu(.)^2, 2: out = gelu(.)
     long long wait_cycles;   // how long a wait on a barrier may take before the block gives up
     int drop_last_load;      // tests only: the copy thread leaves out its last stage, so the MMA thread's wait runs out
     // The residual add folded into the product that makes the addend (swap, cluster_reduce): the block that finishes a
@@ -435,7 +435,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                         const int b = b0 + c0 + j;
                         if (b < G.RB) {
                             if (G.out_f32) ((float*)G.out)[(size_t)b * G.ldo + a] = __uint_as_float(r[j]);
-                            else ((bf16*)G.out)[(size_t)b * G.ldo + a] = __float2bfloat16_rn(G.act ? tl_relu_squared_rounded(__uint_as_float(r[j])) : __uint_as_float(r[j]));
+                            else ((bf16*)G.out)[(size_t)b * G.ldo + a] = __float2bfloat16_rn(G.act ? tl_plain_act(__uint_as_float(r[j]), G.act) : __uint_as_float(r[j]));
                         }
                     }
                 } else {
@@ -536,8 +536,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                     continue;
                 }
                 if (G.act) {
-                    acc.x = tl_relu_squared_rounded(acc.x); acc.y = tl_relu_squared_rounded(acc.y);
-                    acc.z = tl_relu_squared_rounded(acc.z); acc.w = tl_relu_squared_rounded(acc.w);
+                    acc.x = tl_plain_act(acc.x, G.act); acc.y = tl_plain_act(acc.y, G.act);
+                    acc.z = tl_plain_act(acc.z, G.act); acc.w = tl_plain_act(acc.w, G.act);
                 }
                 const size_t o = (size_t)(b0 + tok) * G.ldo + a;
                 if (wide && a + 3 < G.RA) {
@@ -732,7 +732,7 @@ int gemm_impl(const void* x, const void* w, void* y, int out_f32, int ldo, int T
     const int per = (k_tiles + splits - 1) / splits;
     splits = (k_tiles + per - 1) / per;                                                  // no empty split
     if (y == nullptr && splits < 2) return 1;
-    const int act = gated == 4;                                                          // no gate: the square of relu over every output
+    const int act = gated == 4 ? 1 : gated == 5 ? 2 : 0;                                 // no gate: the square of relu, gelu over every output
     if (act) {
         gated = 0;
         if (!swap || out_f32 || y == nullptr || adds || (splits > 1 && !cluster_reduce)) return 1;

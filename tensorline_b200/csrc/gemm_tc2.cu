@@ -121,7 +121,7 @@ struct Gemm2Args {
     int T, N, K;
     int m_tiles, n_tiles;  // tiles of 256 rows and 256 columns
     int out_f32, gated;
-    int act;               // plain epilogue, bf16 out: y = relu(y)^2
+    int act;               // plain epilogue, bf16 out: 1: y = relu(y)^2, 2: y = gelu(y)
     float gate_limit, gate_alpha;   // gated = 3: the clamped swish's constants
     int* status;
 };
@@ -282,7 +282,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant
                             } else {
                                 float v[16];
 #pragma unroll
-                                for (int j = 0; j < 16; ++j) v[j] = G.act ? tl_relu_squared_rounded(__uint_as_float(r[j])) : __uint_as_float(r[j]);
+                                for (int j = 0; j < 16; ++j) v[j] = G.act ? tl_plain_act(__uint_as_float(r[j]), G.act) : __uint_as_float(r[j]);
                                 store16_bf16((bf16*)G.out + (size_t)t * G.ldo + col, v, G.N - col);
                             }
                         }
@@ -359,7 +359,7 @@ TL_EXPORT int tl_gemm_tc2(const void* x, const void* w, void* y, int out_f32, in
                           int* status, int max_pairs, cudaStream_t stream) {
     if (T <= 0 || N <= 0) return 0;
     if (K <= 0 || (K & 7) || ((uintptr_t)x & 15) || ((uintptr_t)w & 15) || y == nullptr || status == nullptr) return 1;
-    const int act = gated == 4;                            // no gate: the square of relu over every output
+    const int act = gated == 4 ? 1 : gated == 5 ? 2 : 0;   // no gate: the square of relu, gelu over every output
     if (act) { gated = 0; if (out_f32) return 1; }
     if (gated && (out_f32 || (N & 127))) return 1;
     if (!g_encode) {

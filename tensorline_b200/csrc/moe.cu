@@ -489,6 +489,35 @@ __global__ void relu_square_vec8_kernel(uint4* __restrict__ u, size_t n8) {
     }
 }
 
+// u = gelu(u) in place, the tanh form
+template <typename TA>
+__global__ void gelu_kernel(TA* __restrict__ u, size_t n) {
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) u[i] = from_f<TA>(tl_gelu_tanh(to_f<TA>(u[i])));
+}
+__global__ void gelu_vec8_kernel(uint4* __restrict__ u, size_t n8) {
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n8; i += (size_t)gridDim.x * blockDim.x) {
+        uint4 v = u[i];
+        __nv_bfloat162* p = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) p[e] = __floats2bfloat162_rn(tl_gelu_tanh(__low2float(p[e])), tl_gelu_tanh(__high2float(p[e])));
+        u[i] = v;
+    }
+}
+
+TL_EXPORT int tl_gelu(void* u, int act_dtype, long long n, cudaStream_t stream) {
+    if (n <= 0) return 0;
+    if (act_dtype == TL_BF16 && n % 8 == 0 && (((uintptr_t)u) & 15) == 0) {
+        const long long n8 = n / 8, most = (long long)tl_num_sms() * 32;
+        gelu_vec8_kernel<<<(int)((n8 + 255) / 256 < most ? (n8 + 255) / 256 : most), 256, 0, stream>>>((uint4*)u, (size_t)n8);
+        return tl_launch_status();
+    }
+    const long long most = (long long)tl_num_sms() * 16;
+    const int blocks = (int)((n + 255) / 256 < most ? (n + 255) / 256 : most);
+    if (act_dtype == TL_F32) gelu_kernel<float><<<blocks, 256, 0, stream>>>((float*)u, (size_t)n);
+    else gelu_kernel<bf16><<<blocks, 256, 0, stream>>>((bf16*)u, (size_t)n);
+    return tl_launch_status();
+}
+
 TL_EXPORT int tl_relu_square(void* u, int act_dtype, long long n, cudaStream_t stream) {
     if (n <= 0) return 0;
     if (act_dtype == TL_BF16 && n % 8 == 0 && (((uintptr_t)u) & 15) == 0) {

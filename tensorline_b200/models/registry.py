@@ -19,6 +19,7 @@ from ..config.dekerax import DekeraxConfig
 from ..config.sumuvik import SumuvikConfig
 from ..config.tenalorn import TenalornConfig
 from ..config.zosurax import ZosuraxConfig
+from ..config.fimolix import FimolixConfig
 from ..parts import Runtime
 from ..weights import load_weights
 from .qwen2 import describe_qwen2
@@ -27,6 +28,7 @@ from .dekerax import describe_dekerax
 from .sumuvik import describe_sumuvik
 from .tenalorn import describe_tenalorn
 from .zosurax import describe_zosurax
+from .fimolix import describe_fimolix
 from .spec import Model
 
 
@@ -60,6 +62,7 @@ register_architecture("Dekerax", DekeraxConfig, describe_dekerax)
 register_architecture("Sumuvik", SumuvikConfig, describe_sumuvik)
 register_architecture("Tenalorn", TenalornConfig, describe_tenalorn)
 register_architecture("Zosurax", ZosuraxConfig, describe_zosurax)
+register_architecture("Fimolix", FimolixConfig, describe_fimolix)
 
 
 def load_config(folder):

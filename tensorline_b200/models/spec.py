@@ -14,6 +14,7 @@ from dataclasses import dataclass
 
 import torch
 
+from ..cache import PagedKV
 from ..parts import BLOCKS, EMBEDDINGS, HEADS, NORMS, POSITION_ENCODINGS, KVCacheView, PartSpec, Runtime, TensorSpec
 from ..parts.linear import with_base, with_row
 
@@ -124,6 +125,12 @@ class Model:
                         needs[(i, name)] = n
                 elif need is not None:
                     needs[i] = need
+        for e in self.spec.run:                          # a cache keeps what the entries that read it can see as well
+            need = self.blocks[e.layer].cache_need() if e.reads_cache_of is not None else None
+            for name, n in (need.items() if isinstance(need, dict) else ((None, need),)):
+                cid = e.reads_cache_of if name is None else (e.reads_cache_of, name)
+                if isinstance(n, PagedKV) and isinstance(needs.get(cid), PagedKV):
+                    needs[cid] = needs[cid].widened(n)
         return needs
 
     def _cache_of(self, i: int, caches: dict):

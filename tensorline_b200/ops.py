@@ -16,7 +16,7 @@ from .csrc.build import CHECK_BUILD, load_library
 
 CORE_SOURCES = ["elementwise.cu", "rope_kv.cu", "attn_tokenwise.cu", "gemm_f32.cu", "sampling.cu", "recurrent.cu", "moe.cu",
                 "delta.cu", "latent.cu", "rglru.cu", "streams.cu", "stream_norm.cu", "attn_mixed_tokenwise.cu",
-                "channel_scan.cu"]
+                "channel_scan.cu", "differential.cu"]
 
 _P, _I, _F = ctypes.c_void_p, ctypes.c_int, ctypes.c_float
 
@@ -25,11 +25,11 @@ _SIGNATURES = {
     "tl_add_rmsnorm": [_P, _P, _P, _I, _P, _I, _P, _I, _I, _F, _I, _P, _I, ctypes.c_longlong, _F, _I, _P],
     "tl_silu_mul": [_P, _P, _I, _I, _I, _I, _I, _F, _F, _P],
     "tl_add_rmsnorm_pair": [_P, _P, _P, _P, _P, _I, _P, _P, _I, _P, _I, _I, _F, _P],
-    "tl_head_gate": [_P, _I, _P, _I, _I, _I, _P],
+    "tl_head_gate": [_P, _I, _P, _I, _I, _I, _I, _P],
     "tl_post_norm_add_norm": [_P, _P, _P, _P, _P, _I, _P, _I, _P, _I, _I, _F, _I, _P],
     "tl_rope_kv_write": [_P, _I, _P, _I, _P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _P, _P, _I, _I, _P, _I, ctypes.c_longlong,
                          _I, _P, _P, _F, _I, _I, _I, _I, _P, _P],
-    "tl_attn_tokenwise": [_P, _I, _P, _I, _P, _P, _P, _I, _I, _P, _P, _I, _I, _I, _I, _I, _F, _P, _I, _P, _I, _P, _I, _I, _P, _P],
+    "tl_attn_tokenwise": [_P, _I, _P, _I, _P, _P, _P, _I, _I, _P, _P, _I, _I, _I, _I, _I, _F, _P, _I, _P, _I, _P, _F, _I, _I, _P, _P],
     "tl_gemm_f32": [_P, _I, _P, _I, _I, _P, _P, _I, _I, _I, _I, _P],
     "tl_argmax": [_P, _I, _I, _I, _P, _P, _P],
     "tl_sample": [_P, _I, _I, _I, _P, _P, _P, _P, _P],
@@ -53,6 +53,7 @@ _SIGNATURES = {
     "tl_moe_sort": [_P, _I, _I, _P, _P, _P, _P],
     "tl_moe_gather": [_P, _I, _P, _P, _P, _I, _P, _I, _I, _I, _I, _P, _P],
     "tl_relu_square": [_P, _I, ctypes.c_longlong, _P],
+    "tl_gelu": [_P, _I, ctypes.c_longlong, _P],
     "tl_moe_combine": [_P, _I, _P, _P, _P, _I, _P, _P, _I, _I, _I, _P, _P, _I, _P],
     "tl_conv_prep": [_P, _I, _I, _P, _I, _I, _P, ctypes.c_longlong, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _F, _P],
     "tl_delta_scan": [_P, _I, _I, _I, _I, _P, _I, _P, _P, _P, ctypes.c_longlong, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
@@ -68,6 +69,9 @@ _SIGNATURES = {
     "tl_attn_mixed_tokenwise": [_P, _I, _P, _I, _P, _P, _P, _I, _I, _P, _P, _I, _I, _I, _I, _F, _P, _I, _I, _P, _P],
     "tl_softcap": [_P, ctypes.c_longlong, _F, _P],
     "tl_sigmoid_gate": [_P, _P, _I, _P, _I, _I, _I, _P],
+    "tl_conv_heads": [_P, _I, _I, _P, _I, _I, _P, ctypes.c_longlong, _P, _P, _P, _P, _I, _I, _P, _P, _F, _P, _P, _P, _I, _I, _I, _I, _I, _I,
+                      _I, _I, _I, _I, _P, _P],
+    "tl_map_difference": [_P, _P, _I, _I, _I, _I, _I, _F, _F, _F, _P],
     "tl_head_matmul": [_P, _I, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _P],
 }
 
@@ -501,12 +505,13 @@ def add_rmsnorm_pair(x: torch.Tensor, a: torch.Tensor | None, b: torch.Tensor | 
 
 
 def head_gate(o: torch.Tensor, gate: torch.Tensor, nq: int, d: int) -> None:
-    """o[t, h, :] *= sigmoid(gate[t, h]) in place; o [T, nq * d] of the activation type, gate float32 [T, nq]."""
+    """o[t, h, :] *= sigmoid(gate[t, h]) in place; o [T, nq * d] of the activation type, gate float32 [T, nq] (a column range
+    of a wider tensor may be passed)."""
     T = o.shape[0]
-    if o.shape != (T, nq * d) or gate.shape != (T, nq) or gate.dtype != torch.float32:
+    if o.shape != (T, nq * d) or gate.shape != (T, nq) or gate.dtype != torch.float32 or gate.stride(1) != 1:
         raise KernelError("head_gate: o [T, nq d], gate float32 [T, nq]")
-    _contig(o, "o"); _contig(gate, "gate")
-    _check(core().tl_head_gate(_ptr(o), dtype_code(o.dtype), _ptr(gate), T, nq, d, _stream()), "head_gate")
+    _contig(o, "o")
+    _check(core().tl_head_gate(_ptr(o), dtype_code(o.dtype), _ptr(gate), gate.stride(0), T, nq, d, _stream()), "head_gate")
 
 
 def post_norm_add_norm(x: torch.Tensor, a: torch.Tensor | None, w_post: torch.Tensor | None, w_pre: torch.Tensor | None,
@@ -514,11 +519,11 @@ def post_norm_add_norm(x: torch.Tensor, a: torch.Tensor | None, w_post: torch.Te
                        rows: torch.Tensor | None = None) -> None:
     """x += a / rms(a) * w_post (+ extra, float32 [H], once a row); out = x / rms(x) * w_pre; float to the end.
     x float32 [*, H]; a (or None: no addend) and out (or None: the sum only) of the activation type; the two weights of
-    one type.  `rows` picks the rows that are produced (x is then left alone)."""
+    one type.  out without w_pre: the sum itself, rounded to out's type.  `rows` picks the rows that are produced (x is then left alone)."""
     H = x.shape[-1]
     if x.dtype != torch.float32 or not x.is_contiguous():
         raise KernelError("post_norm_add_norm: x must be contiguous float32")
-    if (a is None) != (w_post is None) or (out is None) != (w_pre is None):
+    if (a is None) != (w_post is None) or (out is None and w_pre is not None):
         raise KernelError("post_norm_add_norm: an addend comes with its weight, an output with its weight")
     ws = [w for w in (w_post, w_pre) if w is not None]
     if any(w.numel() != H or not w.is_contiguous() or w.dtype != ws[0].dtype for w in ws):
@@ -592,17 +597,18 @@ def attn_tokenwise(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_pages: t
                    table: torch.Tensor, page_size: int, pos: torch.Tensor, req_slot: torch.Tensor,
                    nq: int, nkv: int, d: int, window: int | None, scale: float, sink: torch.Tensor | None = None,
                    keep_first: int = 0, gate: torch.Tensor | None = None, chunk: int | None = None,
-                   slopes: torch.Tensor | None = None) -> None:
+                   slopes: torch.Tensor | None = None, cap: float | None = None) -> None:
     """Exact-order paged attention; q rows `q_stride` elements apart, out [T, nq*d].  `sink` (float32 [nq]): one more
     term exp(sink[h]) in every softmax denominator of head h.  `keep_first` (with a window): the keys at positions below
     it stay visible beside the window.  `gate` (float32 [T, nq]): the row of (t, h) is multiplied by sigmoid(gate[t, h]).
     `chunk` (instead of a window): a query reads the keys of its own chunk of that many positions, counted from position 0.
-    `slopes` (float32 [nq]): the score of key j seen from position p loses slopes[h] * (p - j)."""
+    `slopes` (float32 [nq]): the score of key j seen from position p loses slopes[h] * (p - j).  `cap`: a score is
+    cap * tanh(score / cap) before a slope comes off it."""
     T = out.shape[0]
     if out.shape[1] != nq * d or out.dtype != q.dtype or k_pages.dtype != q.dtype:
         raise KernelError("attn_tokenwise: out must be [T, nq*d] and all tensors of one type")
-    if d > 512:
-        raise KernelError(f"attn_tokenwise: head_dim {d} > 512 is not supported")
+    if d > 1024:
+        raise KernelError(f"attn_tokenwise: head_dim {d} > 1024 is not supported")
     _contig(out, "out"); _contig(k_pages, "k_pages"); _contig(v_pages, "v_pages")
     _ints(pos, "pos"); _ints(req_slot, "req_slot"); _ints(table, "table")
     _sink(sink, nq, "attn_tokenwise")
@@ -616,7 +622,7 @@ def attn_tokenwise(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_pages: t
     _check(core().tl_attn_tokenwise(_ptr(q), q_stride, _ptr(out), dtype_code(q.dtype), _ptr(k_pages), _ptr(v_pages),
                                     _ptr(table), table.shape[1], page_size, _ptr(pos), _ptr(req_slot), T, nq, nkv, d,
                                     int(window or 0), float(scale), _ptr(sink), int(keep_first), _ptr(gate), int(chunk or 0),
-                                    _ptr(slopes), table.shape[0], k_pages.shape[0], fault_words(out.device), _stream()),
+                                    _ptr(slopes), float(cap or 0.0), table.shape[0], k_pages.shape[0], fault_words(out.device), _stream()),
            "attn_tokenwise")
 
 
@@ -972,6 +978,12 @@ def relu_square(u: torch.Tensor) -> None:
     _check(core().tl_relu_square(_ptr(u), dtype_code(u.dtype), u.numel(), _stream()), "relu_square")
 
 
+def gelu(u: torch.Tensor) -> None:
+    """u = 0.5 u (1 + tanh(sqrt(2/pi) (u + 0.044715 u^3))) in place."""
+    _contig(u, "u")
+    _check(core().tl_gelu(_ptr(u), dtype_code(u.dtype), u.numel(), _stream()), "gelu")
+
+
 def moe_combine(rows: torch.Tensor, place_of: torch.Tensor, idx: torch.Tensor, offsets: torch.Tensor, wts: torch.Tensor | None,
                 y: torch.Tensor, cap: int = 0, extra: torch.Tensor | None = None, extra_gate: torch.Tensor | None = None) -> None:
     """y[t] = sum_j wts[t, j] * rows[row of place_of[t * top + j]] (+ sigmoid(extra_gate[t]) * extra[t]); rows laid out as
@@ -1124,6 +1136,60 @@ def head_matmul(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, H: int, K: in
     _contig(w, "w")
     _check(core().tl_head_matmul(_ptr(x), x.stride(0), x_head_stride, _ptr(w), dtype_code(w.dtype), _ptr(y), y.stride(0),
                                  y_head_stride, T, H, K, N, dtype_code(x.dtype), _stream()), "head_matmul")
+
+
+# ---------------------------------------------------------------------------------------------
+# Heads made of maps behind a short convolution (csrc/differential.cu)
+
+def conv_heads(proj: torch.Tensor, taps_w: torch.Tensor, state: torch.Tensor | None, ctx, table: torch.Tensor, page_size: int,
+               q_out: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, *, nq: int, nkv: int, maps: int, dim: int, dv: int,
+               q_norm: torch.Tensor | None = None, k_norm: torch.Tensor | None = None, eps: float = 0.0) -> None:
+    """proj [T, C] holds q [nq, maps, dim], k [nkv, maps, dim], v [nkv, dv] of every token.  Every channel passes a causal
+    convolution over its request's tokens (taps_w [C, taps], the last tap on the current token; the taps - 1 rows before the step
+    come from `state[slot]`, [taps - 1, C] of proj's type, zeros for a new request, which is then brought up to date); every map of
+    q and k is RMS-normalised over its dim channels with q_norm / k_norm (float32 [dim], both or neither).  q_out [T, nq maps d]: map m
+    of a head in columns [m dim, (m + 1) dim) of its row of d, zeros elsewhere; k_pages, v_pages [pages, nkv, page, d]: a key's maps
+    side by side, a value in front, zeros behind."""
+    T = proj.shape[0]
+    C = (nq + nkv) * maps * dim + nkv * dv
+    taps = taps_w.shape[1]
+    d = k_pages.shape[-1]
+    if proj.shape != (T, C) or taps_w.shape != (C, taps) or q_out.shape != (T, nq * maps * d) or q_out.dtype != proj.dtype:
+        raise KernelError("conv_heads: proj [T, C], taps_w [C, taps], q_out [T, nq maps d] of proj's type")
+    for name, pages in (("k_pages", k_pages), ("v_pages", v_pages)):
+        if pages.dtype != proj.dtype or tuple(pages.shape[1:]) != (nkv, page_size, d):
+            raise KernelError(f"conv_heads: {name} must be [pages, nkv, page, d] of proj's type")
+        _contig(pages, name)
+    if maps * dim > d or dv > d:
+        raise KernelError(f"conv_heads: rows of {d} hold neither {maps} x {dim} nor {dv} columns")
+    if (q_norm is None) != (k_norm is None):
+        raise KernelError("conv_heads: q_norm and k_norm come together")
+    for name, w in (("q_norm", q_norm), ("k_norm", k_norm)):
+        if w is not None and (w.dtype != torch.float32 or w.numel() != dim or not w.is_contiguous()):
+            raise KernelError(f"conv_heads: {name} must be float32 [dim]")
+    slot_stride = 0
+    if taps > 1:
+        if state is None or state.dtype != proj.dtype or not state.is_contiguous() or state[0].numel() != (taps - 1) * C:
+            raise KernelError("conv_heads: state must be [slots, taps - 1, C] of proj's type")
+        slot_stride = state[0].numel()
+    _contig(proj, "proj"); _contig(taps_w, "taps_w"); _contig(q_out, "q_out")
+    _ints(ctx.q_start, "q_start"); _ints(ctx.slots, "slots"); _ints(ctx.start_pos, "start_pos"); _ints(table, "table")
+    _check(core().tl_conv_heads(_ptr(proj), dtype_code(proj.dtype), proj.stride(0), _ptr(taps_w), dtype_code(taps_w.dtype), taps,
+                                _ptr(state) if taps > 1 else None, slot_stride, _ptr(ctx.q_start), _ptr(ctx.slots), _ptr(ctx.start_pos),
+                                _ptr(table), table.shape[1], page_size, _ptr(q_norm), _ptr(k_norm), float(eps), _ptr(q_out), _ptr(k_pages),
+                                _ptr(v_pages), nq, nkv, maps, dim, dv, d, int(ctx.B), int(ctx.max_q_len), table.shape[0], k_pages.shape[0],
+                                fault_words(proj.device), _stream()), "conv_heads")
+
+
+def map_difference(a: torch.Tensor, y: torch.Tensor, H: int, dv: int, weight: float, eps: float, out_scale: float) -> None:
+    """y[t, h] = out_scale * o / rms(o), o = a[t, h, 0, :dv] - weight * a[t, h, 1, :dv]; a [T, H * 2 * d], y [T, H * dv] of one type."""
+    T = a.shape[0]
+    d = a.shape[1] // (2 * H)
+    if a.shape != (T, 2 * H * d) or y.shape != (T, H * dv) or y.dtype != a.dtype or dv > d:
+        raise KernelError("map_difference: a [T, H 2 d], y [T, H dv] of one type, dv <= d")
+    _contig(a, "a"); _contig(y, "y")
+    _check(core().tl_map_difference(_ptr(a), _ptr(y), dtype_code(a.dtype), T, H, d, dv, float(weight), float(eps), float(out_scale),
+                                    _stream()), "map_difference")
 
 
 # ---------------------------------------------------------------------------------------------

@@ -49,6 +49,8 @@ def attn_lib(head_dim: int):
         lib.tl_attn_set_keep_first.restype = ctypes.c_int
         lib.tl_attn_set_distance.argtypes = [_I, _P]
         lib.tl_attn_set_distance.restype = ctypes.c_int
+        lib.tl_attn_set_cap.argtypes = [_F]
+        lib.tl_attn_set_cap.restype = ctypes.c_int
         if lib.tl_attn_decode_max_table() != DECODE_MAX_TABLE_ENTRIES:
             raise KernelError(f"the attention library copies {lib.tl_attn_decode_max_table()} block-table entries a block, "
                               f"the split planner assumes {DECODE_MAX_TABLE_ENTRIES}")
@@ -91,12 +93,18 @@ def attn_tc_lib(head_dim: int):
         lib.tl_attn_set_keep_first.restype = ctypes.c_int
         lib.tl_attn_set_distance.argtypes = [_I, _P]
         lib.tl_attn_set_distance.restype = ctypes.c_int
+        lib.tl_attn_set_cap.argtypes = [_F]
+        lib.tl_attn_set_cap.restype = ctypes.c_int
         _tc_libs[head_dim] = lib
     return lib
 
 
-def _set_distance(lib, chunk, slopes, nq: int, window) -> None:
-    """Chunks and distance slopes of the library's launches that follow (None: none).  Set before every launch."""
+def _set_distance(lib, chunk, slopes, nq: int, window, cap: float | None = None) -> None:
+    """Chunks, distance slopes and the cap on the scores of the library's launches that follow (None: none).  Set before every
+    launch."""
+    if cap is not None and not cap > 0:
+        raise KernelError("attention: a cap on the scores is positive")
+    lib.tl_attn_set_cap(float(cap or 0.0))
     if chunk and window:
         raise KernelError("attention: a window or chunks, not both")
     if slopes is not None and (slopes.dtype != torch.float32 or slopes.numel() != nq or not slopes.is_contiguous() or not slopes.is_cuda):
@@ -118,10 +126,11 @@ def tc_min_page(head_dim: int) -> int:
 
 
 def prefill_tc(q, q_stride, out, k_pages, v_pages, table, page_size, q_start, start_pos, slots, h_q_start,
-               nq, nkv, d, window, scale, order=None, sink=None, keep_first: int = 0, chunk: int | None = None, slopes=None) -> None:
+               nq, nkv, d, window, scale, order=None, sink=None, keep_first: int = 0, chunk: int | None = None, slopes=None,
+               cap: float | None = None) -> None:
     """Prompt-portion attention on tcgen05: 128 query rows per block, S and O in tensor memory.  `keep_first` (with a
     window): the keys at positions below it stay visible to every later row; a block walks their key tiles first.
-    `chunk` (instead of a window) and `slopes`: as `prefill` takes them."""
+    `chunk` (instead of a window), `slopes` and `cap`: as `prefill` takes them."""
     from .ops_gemm import status_word
     if page_size < tc_min_page(d) or page_size > KEY_TILE or page_size & (page_size - 1):
         raise KernelError(f"page size {page_size}: the tcgen05 attention kernel for head size {d} takes powers of two "
@@ -132,7 +141,7 @@ def prefill_tc(q, q_stride, out, k_pages, v_pages, table, page_size, q_start, st
     if order is not None:
         tiles = order.numel()                           # the array may leave requests out
     _set_sink(attn_tc_lib(d), sink, nq)
-    _set_distance(attn_tc_lib(d), chunk, slopes, nq, window)
+    _set_distance(attn_tc_lib(d), chunk, slopes, nq, window, cap)
     attn_tc_lib(d).tl_attn_set_keep_first(int(keep_first) if window else 0)
     _check(attn_tc_lib(d).tl_attn_tc_prefill(_ptr(q), q_stride, _ptr(out), _ptr(k_pages), _ptr(v_pages), _ptr(table),
                                              table.shape[1], page_size, _ptr(q_start), _ptr(start_pos), _ptr(slots), B,
@@ -181,7 +190,8 @@ TC_P_IN_TMEM = {"0": False, "1": True}.get(os.environ.get("TENSORLINE_B200_TC_P_
 
 
 def prefill_tc_pair(q, q_stride, out, k_pages, v_pages, table, page_size, q_start, start_pos, slots, h_q_start,
-                    nq, nkv, d, window, scale, order=None, p_in_tmem=None, ksplit: int = 1, merge_rows=None, sink=None) -> bool:
+                    nq, nkv, d, window, scale, order=None, p_in_tmem=None, ksplit: int = 1, merge_rows=None, sink=None,
+                    cap: float | None = None) -> bool:
     """Prompt-portion attention on tcgen05 with two query tiles (256 rows) per block and K, V by TMA.
     `p_in_tmem` (None: as the switch says): "64": P kept in tensor memory, key tiles of 64; False: P through shared
     memory; True: key tiles of 128 and P in tensor memory.  Head sizes 64 and 128, pages of 8 to 64 tokens; returns
@@ -200,7 +210,7 @@ def prefill_tc_pair(q, q_stride, out, k_pages, v_pages, table, page_size, q_star
         tiles = order.numel()
     lib = attn_tc_lib(d)
     _set_sink(lib, sink, nq)
-    _set_distance(lib, None, None, nq, window)             # the pair kernels take neither chunks nor slopes
+    _set_distance(lib, None, None, nq, window, cap)        # the pair kernels take neither chunks nor slopes
     if ksplit > 1 and p_in_tmem is not True:
         T = out.shape[0]
         if merge_rows is None:
@@ -265,15 +275,16 @@ def plan_splits(batch: int, nkv: int, group: int, span: int, head_dim: int = 128
 
 
 def prefill(q, q_stride, out, k_pages, v_pages, table, page_size, q_start, start_pos, slots, h_q_start,
-            nq, nkv, d, window, scale, order=None, sink=None, keep_first: int = 0, chunk: int | None = None, slopes=None) -> None:
+            nq, nkv, d, window, scale, order=None, sink=None, keep_first: int = 0, chunk: int | None = None, slopes=None,
+            cap: float | None = None) -> None:
     """Prompt-portion attention on mma.sync tiles of 64 query rows.  `keep_first` (with a window): the keys at positions below
     it stay visible beside the window; the kernel walks their tiles in front of the window's.  `chunk` (instead of a
     window): a query reads the keys of its own chunk of that many positions only; `slopes` (float32 [nq]): the score of key
-    j seen from position p loses slopes[h] * (p - j)."""
+    j seen from position p loses slopes[h] * (p - j).  `cap`: scores are cap * tanh(score / cap)."""
     g = nq // nkv
     B = len(h_q_start) - 1
     _set_sink(attn_lib(d), sink, nq)
-    _set_distance(attn_lib(d), chunk, slopes, nq, window)
+    _set_distance(attn_lib(d), chunk, slopes, nq, window, cap)
     attn_lib(d).tl_attn_set_keep_first(int(keep_first) if window else 0)
     tiles = sum(-(-(h_q_start[i + 1] - h_q_start[i]) * g // KEY_TILE) for i in range(B))
     if order is not None:
@@ -305,7 +316,7 @@ def decode_takes_rope(B: int, d: int, page_size: int) -> bool:
 def decode(q, q_stride, out, k_pages, v_pages, table, page_size, q_start, start_pos, slots, B,
            nq, nkv, d, window, scale, chunk, splits, part_o=None, part_ml=None, tma: bool | None = None,
            cluster: bool | None = None, rope: dict | None = None, sink=None, keep_first: int = 0, mask_chunk: int | None = None,
-           slopes=None) -> None:
+           slopes=None, cap: float | None = None) -> None:
     """Split-KV decode attention.  `tma`: load K and V by TMA (head sizes that are multiples of 64, pages of
     8..64 tokens); None = wherever that applies.  `cluster` (TMA path, 2..8 key ranges, groups of at most 16
     heads): the ranges of a request merge inside a thread-block cluster, no partials, no second kernel;
@@ -316,7 +327,7 @@ def decode(q, q_stride, out, k_pages, v_pages, table, page_size, q_start, start_
     if KEY_TILE % page_size:
         raise KernelError(f"page size {page_size} must divide {KEY_TILE}")
     _set_sink(attn_lib(d), sink, nq)
-    _set_distance(attn_lib(d), mask_chunk, slopes, nq, window)      # `mask_chunk`: the chunks of the mask (`chunk` is a block's key range)
+    _set_distance(attn_lib(d), mask_chunk, slopes, nq, window, cap)      # `mask_chunk`: the chunks of the mask (`chunk` is a block's key range)
     keep_first = int(keep_first) if window else 0
     attn_lib(d).tl_attn_set_keep_first(keep_first)
     # kept first keys beside a window are two runs of keys: the cp.async kernel walks them (`chunk` and `splits` then count
@@ -376,7 +387,7 @@ def kept_span(keep_first: int) -> int:
 
 
 def attend_bf16(qkv, o, ctx, k_pages, v_pages, table, nq, nkv, d, window, scale, rope: dict | None = None, sink=None,
-                keep_first: int = 0, chunk: int | None = None, slopes=None) -> None:
+                keep_first: int = 0, chunk: int | None = None, slopes=None, cap: float | None = None) -> None:
     """`rope`: only for decode-only steps that `decode_takes_rope` accepted (see `decode`).  `sink`: float32 [nq], one more
     term exp(sink[h]) in the softmax denominators of head h (every kernel adds it once, where a row is finished)."""
     if qkv.dtype != torch.bfloat16 or k_pages.dtype != torch.bfloat16:
@@ -391,7 +402,7 @@ def attend_bf16(qkv, o, ctx, k_pages, v_pages, table, nq, nkv, d, window, scale,
             span = min(span, window + KEY_TILE - 1 + kept_span(keep_first))
         if chunk:
             span = min(span, chunk + KEY_TILE - 1)
-        dist = {"mask_chunk": chunk, "slopes": slopes}
+        dist = {"mask_chunk": chunk, "slopes": slopes, "cap": cap}
         chunk, splits = plan_splits(ctx.B, nkv, nq // nkv, span, d, page_size=ctx.page_size)
         part_o = part_ml = None
         if splits > 1:
@@ -402,7 +413,7 @@ def attend_bf16(qkv, o, ctx, k_pages, v_pages, table, nq, nkv, d, window, scale,
                **dist)
     else:
         g = nq // nkv
-        dist = {"mask_chunk": chunk, "slopes": slopes}
+        dist = {"mask_chunk": chunk, "slopes": slopes, "cap": cap}
         mask_chunk = chunk
         singles = _single_token_requests(ctx, qkv.device, g, nkv)
         skip = singles["set"] if singles else frozenset()
@@ -477,17 +488,17 @@ def attend_bf16(qkv, o, ctx, k_pages, v_pages, table, nq, nkv, d, window, scale,
             if rows_key not in ctx.scratch:
                 rows = [t for i in rest for t in range(ctx.h_q_start[i], ctx.h_q_start[i + 1])]
                 ctx.scratch[rows_key] = torch.tensor(rows, dtype=torch.int32).to(qkv.device, non_blocking=True)
-            if not prefill_tc_pair(*args, order(2 * TC_QUERY_TILE), ksplit=ksplit, merge_rows=ctx.scratch[rows_key], sink=sink):
+            if not prefill_tc_pair(*args, order(2 * TC_QUERY_TILE), ksplit=ksplit, merge_rows=ctx.scratch[rows_key], sink=sink, cap=cap):
                 ksplit = 1
         if ksplit >= 2:
             pass
         elif use_tc and TC_PAIR and not keep_first and not distant and one_tile_blocks > ops.num_sms() and \
-                prefill_tc_pair(*args, order(2 * TC_QUERY_TILE), sink=sink):
+                prefill_tc_pair(*args, order(2 * TC_QUERY_TILE), sink=sink, cap=cap):
             pass
         elif use_tc:
-            prefill_tc(*args, order(TC_QUERY_TILE), sink=sink, keep_first=keep_first, chunk=mask_chunk, slopes=slopes)
+            prefill_tc(*args, order(TC_QUERY_TILE), sink=sink, keep_first=keep_first, chunk=mask_chunk, slopes=slopes, cap=cap)
         else:
-            prefill(*args, order(KEY_TILE), sink=sink, keep_first=keep_first, chunk=mask_chunk, slopes=slopes)
+            prefill(*args, order(KEY_TILE), sink=sink, keep_first=keep_first, chunk=mask_chunk, slopes=slopes, cap=cap)
         if singles and joined is not None:
             torch.cuda.current_stream(qkv.device).wait_event(joined)
 

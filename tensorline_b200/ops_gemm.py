@@ -82,7 +82,7 @@ def gemm_tc(x, w: torch.Tensor, out_dtype: torch.dtype = torch.bfloat16, *, swap
     consumer that adds them up itself) instead of the product.
     `gated`: w holds gate and up rows interleaved in blocks of 64 (N % 128 == 0); the result is
     silu(gate) * up, [T, N / 2] bfloat16, formed in the epilogue (few tokens, one split only:
-    check `can_gate` first); "relu_squared": no gate, relu(.)^2 of every output, [T, N] (check `can_act`).
+    check `can_gate` first); a name of `PLAIN_ACTS`: no gate, that activation of every output, [T, N] (check `can_act`).
     `x` may be a `parts.linear.NormedInput` (few-token order): the activations are then the RMS norm of rows of the
     float32 residual stream, made inside the kernel from the stream, the rows' partial sums of squares and the norm weight.
     `residual` (float32 [T, N], check `can_add_residual` first): the result, rounded to bfloat16, is added into it in
@@ -131,9 +131,9 @@ def gemm_tc(x, w: torch.Tensor, out_dtype: torch.dtype = torch.bfloat16, *, swap
         if residual.dtype != torch.float32 or residual.shape != (T, N) or residual.stride(1) != 1 or residual.stride(0) % 4:
             raise KernelError("gemm_tc: residual must be float32 [T, N] with unit inner stride")
         ssq = torch.empty((T, -(-N // 128)), dtype=torch.float32, device=dev)
-    if gated == "relu_squared":                          # no gate: an activation over every output
+    if gated in PLAIN_ACTS:                              # no gate: an activation over every output
         if not swap or residual is not None or pieces or (splits > 1 and not use_cluster) or out_dtype != torch.bfloat16:
-            raise KernelError("gemm_tc: the square of relu needs the few-token order, ranges of K summed in a cluster, bfloat16 (see can_act)")
+            raise KernelError("gemm_tc: an activation without a gate needs the few-token order, ranges of K summed in a cluster, bfloat16 (see can_act)")
         if out is None:
             out = torch.empty((T, N), dtype=out_dtype, device=dev)
     elif gated:
@@ -152,7 +152,7 @@ def gemm_tc(x, w: torch.Tensor, out_dtype: torch.dtype = torch.bfloat16, *, swap
     partial = torch.empty((splits, T, N), dtype=torch.float32, device=dev) if splits > 1 and not use_cluster else None
     st = status_word(dev)
     ldo = N if out is None else out.stride(0)
-    name = (f"gemm_tc<{bn}>" + ("+relu2" if gated == "relu_squared" else "+gated" if gated else "") + ("+cluster" if use_cluster else "") + ("+pieces" if pieces else "")
+    name = (f"gemm_tc<{bn}>" + (PLAIN_ACTS[gated][1] if gated in PLAIN_ACTS else "+gated" if gated else "") + ("+cluster" if use_cluster else "") + ("+pieces" if pieces else "")
             + ("" if swap else "+rows") + ("+normed" if normed is not None else "") + ("+residual" if residual is not None else ""))
     launches = 1 if (splits == 1 or fused_reduce or pieces or use_cluster) else 2
     counters = (st.data_ptr() + 4) if fused_reduce else None
@@ -195,7 +195,7 @@ def gemm_tc2(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype = torch.bf
              out: torch.Tensor | None = None, max_pairs: int = 0) -> torch.Tensor:
     """x [T, K] times w [N, K]^T on pairs of thread blocks (256 x 256 tiles, persistent, double-buffered
     accumulators).  `gated`: w holds gate and up rows interleaved in blocks of 64 (N % 128 == 0); the result is
-    silu(gate) * up, [T, N / 2] bfloat16, formed in the epilogue; "relu_squared": no gate, relu(.)^2, [T, N]."""
+    silu(gate) * up, [T, N / 2] bfloat16, formed in the epilogue; a name of `PLAIN_ACTS`: no gate, that activation, [T, N]."""
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
         raise KernelError("gemm_tc2: bfloat16 operands only")
     T, K = x.shape
@@ -206,7 +206,7 @@ def gemm_tc2(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype = torch.bf
         raise KernelError(f"gemm_tc2: K = {K} must be a multiple of 8 (TMA needs 16-byte rows)")
     if out_dtype not in (torch.bfloat16, torch.float32):
         raise KernelError("gemm_tc2: output is bfloat16 or float32")
-    plain_act = gated == "relu_squared"                  # no gate: an activation over every output
+    plain_act = gated in PLAIN_ACTS                      # no gate: an activation over every output
     if gated and ((N % 128 and not plain_act) or out_dtype != torch.bfloat16):
         raise KernelError("gemm_tc2: the gated epilogue needs N % 128 == 0 and bfloat16 output")
     cols = N // 2 if gated and not plain_act else N
@@ -218,8 +218,12 @@ def gemm_tc2(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype = torch.bf
     if isinstance(gated, tuple):
         lib2().tl_gemm_tc2_set_gate(float(gated[1]), float(gated[2]))
     _check(lib2().tl_gemm_tc2(_ptr(x), _ptr(w), _ptr(out), int(out_dtype == torch.float32), out.stride(0), T, N, K,
-                              _gate_code(gated), _ptr(st), int(max_pairs), _stream()), "gemm_tc2" + ("+relu2" if gated == "relu_squared" else "+gated" if gated else ""))
+                              _gate_code(gated), _ptr(st), int(max_pairs), _stream()), "gemm_tc2" + (PLAIN_ACTS[gated][1] if gated in PLAIN_ACTS else "+gated" if gated else ""))
     return out
+
+
+# activations of products without a gate: name -> (code of the kernels, suffix of the launch's name)
+PLAIN_ACTS = {"relu_squared": (4, "+relu2"), "plain_gelu_tanh": (5, "+gelu")}
 
 
 def _gate_code(gated) -> int:
@@ -233,8 +237,8 @@ def _gate_code(gated) -> int:
         return 1
     if gated == "gelu_tanh":
         return 2
-    if gated == "relu_squared":                          # no gate at all
-        return 4
+    if gated in PLAIN_ACTS:                              # no gate at all
+        return PLAIN_ACTS[gated][0]
     raise KernelError(f"a gated epilogue applies 'silu', 'gelu_tanh' or ('swish_clamped', limit, alpha), not {gated!r}")
 
 
@@ -245,7 +249,7 @@ def can_gate(T: int, N: int, K: int) -> bool:
 
 
 def can_act(T: int, N: int, K: int) -> bool:
-    """Whether the plan for these sizes allows the square of relu in the epilogue (`gated` "relu_squared")."""
+    """Whether the plan for these sizes allows an activation without a gate in the epilogue (`PLAIN_ACTS`)."""
     swap, _, splits = plan(T, N, K)
     k_tiles = -(-K // 64)
     splits = -(-k_tiles // -(-k_tiles // min(splits, k_tiles)))

@@ -36,6 +36,8 @@ result, instead of a rounding to the activation type before the weight.
 
 `head_mix` (tensor `head_mix`, [query heads, query heads]): the heads' softmax weights are mixed before they meet the values
 (Shazeer et al., "Talking-Heads Attention"): head h applies sum_g mix[h, g] P_g to the values of its own KV head.
+
+`score_cap`: a score is cap * tanh(score / cap), after the scale and before a distance slope comes off it.
 """
 from __future__ import annotations
 
@@ -71,7 +73,7 @@ class PagedAttention(Part):
                  qk_norm_eps: float | None = None, v_head_dim: int | None = None, sink: bool = False,
                  names: dict | None = None, keep_first: int = 0, sink_value: float | None = None, head_gate: bool = False,
                  chunk: int | None = None, distance_slopes=None, qk_norm_weight: bool = True, qk_norm_cast: bool = True,
-                 head_mix: bool = False):
+                 head_mix: bool = False, score_cap: float | None = None):
         super().__init__(rt)
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} query heads are not a multiple of {num_kv_heads} KV heads")
@@ -86,6 +88,9 @@ class PagedAttention(Part):
             d += d & 1                                    # the kernel that writes the pages works on pairs of dimensions
         if head_mix and (window is not None or chunk is not None or sink or sink_value is not None or head_gate or distance_slopes is not None):
             raise ValueError("heads whose weights are mixed see every earlier key, without a sink, a gate or distance slopes")
+        if head_mix and score_cap is not None:
+            raise ValueError("heads whose weights are mixed take no cap on their scores")
+        self.score_cap = score_cap
         self.has_mix, self.qk_norm_cast = bool(head_mix), bool(qk_norm_cast)
         if chunk is not None and (window is not None or chunk < 1):
             raise ValueError("chunks are positive and stand instead of a window")

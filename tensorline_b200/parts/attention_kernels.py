@@ -19,6 +19,7 @@ def attend(mixer, qkv, o, ctx, cache, table, rope=None, gate=None) -> None:
     sink = getattr(mixer, "sink", None)
     keep_first = getattr(mixer, "keep_first", 0) if mixer.window else 0
     chunk, slopes = getattr(mixer, "chunk", None), getattr(mixer, "slopes", None)
+    cap = getattr(mixer, "score_cap", None)
     from .. import ops_attention, ops_attention_mix
     if getattr(mixer, "mix", None) is not None:              # the heads' weights are mixed: kernels of their own
         if mixer.mix_pad is not None and qkv.dtype == torch.bfloat16 and not ctx.force_exact_attention and \
@@ -33,9 +34,9 @@ def attend(mixer, qkv, o, ctx, cache, table, rope=None, gate=None) -> None:
             ((chunk or slopes is not None) and not ops_attention.TAKES_CHUNKS):   # heads wider than the tensor-core kernels take
         ops.attn_tokenwise(qkv, qkv.shape[1], o, cache.k, cache.v, table, ctx.page_size, ctx.pos, ctx.req_slot,
                            nq, nkv, d, mixer.window, mixer.scale, sink=sink, keep_first=keep_first, gate=gate, chunk=chunk,
-                           slopes=slopes)
+                           slopes=slopes, cap=cap)
         return
     ops_attention.attend_bf16(qkv, o, ctx, cache.k, cache.v, table, nq, nkv, d, mixer.window, mixer.scale, rope=rope, sink=sink,
-                              keep_first=keep_first, chunk=chunk, slopes=slopes)
+                              keep_first=keep_first, chunk=chunk, slopes=slopes, cap=cap)
     if gate is not None:
         ops.head_gate(o, gate, nq, d)

@@ -9,6 +9,7 @@ first norm (or the model's last) as `pending`.
 from __future__ import annotations
 
 from .base import FEED_FORWARDS, MIXERS, NORMS, Part, PartSpec, Runtime, register_block
+from .norm import read_stream
 from .linear import PairSum, PostNormed, Scaled, StreamSum, StreamUpdate, resolve
 
 
@@ -143,6 +144,24 @@ class SandwichNormBlock(PreNormBlock):
             return a
         h = self.norm2.add_norm(x, a)
         return PostNormed(self.ff.forward(h, ctx), self.post2.weight, self.post2.eps)
+
+
+@register_block("post_norm")
+class PostNormBlock(PreNormBlock):
+    """A block that normalises its sub-blocks' outputs and nothing else; they read the stream itself:
+
+        x += norm1(mixer(x));   x += norm2(feed_forward(x))
+
+    A sub-block's output travels as a `PostNormed` addend: its norm, the residual sum and the rounding of the stream for the
+    next sub-block are one kernel in float32 (`read_stream`)."""
+
+    def forward(self, x, pending, ctx, cache):
+        h = read_stream(x, pending, self.rt)
+        a = PostNormed(self.mixer.forward(h, ctx, cache), self.norm1.weight, self.norm1.eps)
+        if self.ff is None:
+            return a
+        h = read_stream(x, a, self.rt)
+        return PostNormed(self.ff.forward(h, ctx), self.norm2.weight, self.norm2.eps)
 
 
 @register_block("hyper_connections")

@@ -15,7 +15,10 @@ products per head (`ops.head_matmul`).  Norm statistics, angles, scores and soft
 Options: `q_rank` None: the queries are one projection of the input (tensor `uq` [H (dk + dr), hidden]), there is no query
 latent; the position encoding may pair (i, i + rot/2) or (2i, 2i + 1); `out_gate`: the heads' outputs, side by side, are
 multiplied element by element by sigmoid(Wg h) (tensor `g` [H dv, hidden], float32 pre-activations: its rows ride in the
-down product) before the output projection.
+down product) before the output projection; `head_gate`: head a's output is multiplied by the one number sigmoid(Wg h)_a (tensor
+`g` [H, hidden]); `sink` (tensor `sink` [H]): every softmax denominator of head a also holds exp(sink_a), a term without key or
+value that is not scaled; `score_cap`: scores are cap * tanh(score / cap); `reads_latent`: the mixer has no Wdkv, its run entry reads
+what another entry's cache holds (`RunEntry.reads_cache_of`) with a Wuk, a Wuv and queries of its own.
 """
 from __future__ import annotations
 
@@ -30,7 +33,7 @@ from .linear import matmul, resolve
 HEAD_PRODUCT_LIBRARY_MIN_TOKENS = 64
 
 _NAMES = {"dq": "dq", "dq_norm": "dq.norm", "uq": "uq", "dkv": "dkv", "dkv_norm": "dkv.norm", "uk": "uk", "uv": "uv", "o": "o",
-          "g": "g"}
+          "g": "g", "sink": "sink"}
 
 
 @register_mixer("latent_attention")
@@ -39,17 +42,24 @@ class LatentAttention(Part):
 
     def __init__(self, rt: Runtime, hidden: int, num_heads: int, head_dim: int, rot_dim: int, v_head_dim: int, q_rank: int | None,
                  kv_rank: int, scale: float, norm_eps: float, position: PartSpec, window: int | None = None,
-                 names: dict | None = None, out_gate: bool = False):
+                 names: dict | None = None, out_gate: bool = False, head_gate: bool = False, sink: bool = False,
+                 score_cap: float | None = None, reads_latent: bool = False):
         super().__init__(rt)
+        if out_gate and head_gate:
+            raise ValueError("a gate is either one number a head or one a column")
+        if reads_latent and (q_rank or out_gate):
+            raise ValueError("a mixer without a down projection has neither a query latent nor a gate that rides in it")
         self.hidden, self.H, self.dk, self.dr, self.dv = hidden, num_heads, head_dim, rot_dim, v_head_dim
         self.qr, self.rank, self.scale, self.eps, self.window = int(q_rank or 0), kv_rank, float(scale), float(norm_eps), window
-        self.out_gate = bool(out_gate)
+        self.out_gate, self.head_gate, self.has_sink, self.reads_latent = bool(out_gate), bool(head_gate), bool(sink), bool(reads_latent)
+        self.score_cap = score_cap
         d = kv_rank + rot_dim
         self.d = d if rt.exact else -(-d // 16) * 16     # the bfloat16 attention kernels take multiples of 16
         self.position = POSITION_ENCODINGS.build(position, rt, head_dim=rot_dim)
         self.names = {**_NAMES, **(names or {})}
         # what `attention_kernels.attend` reads of a mixer
         self.nq, self.nkv, self.sink = num_heads, 1, None
+        self.w_gate = None
         self.w_down = self.w_uq = self.w_uk = self.w_uv = self.w_o = self.n_q = self.n_kv = None
 
     def cache_need(self):
@@ -59,9 +69,14 @@ class LatentAttention(Part):
         n = {k: f"{prefix}.{v}" for k, v in self.names.items()}
         W, H = self.hidden, self.H
         out = {n["uq"]: TensorSpec((H * (self.dk + self.dr), self.qr or W)),
-               n["dkv"]: TensorSpec((self.rank + self.dr, W)), n["dkv_norm"]: TensorSpec((self.rank,), init="ones"),
                n["uk"]: TensorSpec((H * self.dk, self.rank)), n["uv"]: TensorSpec((H * self.dv, self.rank)),
                n["o"]: TensorSpec((W, H * self.dv))}
+        if not self.reads_latent:
+            out.update({n["dkv"]: TensorSpec((self.rank + self.dr, W)), n["dkv_norm"]: TensorSpec((self.rank,), init="ones")})
+        if self.has_sink:
+            out[n["sink"]] = TensorSpec((H,))
+        if self.head_gate:
+            out[n["g"]] = TensorSpec((H, W))
         if self.qr:
             out.update({n["dq"]: TensorSpec((self.qr, W)), n["dq_norm"]: TensorSpec((self.qr,), init="ones")})
         if self.out_gate:
@@ -72,13 +87,19 @@ class LatentAttention(Part):
         n = {k: f"{prefix}.{v}" for k, v in self.names.items()}
         H = self.H
         # the down product's float32 accumulators are kept as they are: they feed two norms
-        down = ([weights[n["dq"]]] if self.qr else []) + [weights[n["dkv"]]] + ([weights[n["g"]]] if self.out_gate else [])
-        self.w_down = self._compute_copy(torch.cat(down, dim=0))
+        if not self.reads_latent:
+            down = ([weights[n["dq"]]] if self.qr else []) + [weights[n["dkv"]]] + \
+                ([weights[n["g"]]] if self.out_gate or self.head_gate else [])
+            self.w_down = self._compute_copy(torch.cat(down, dim=0))
+            self.n_kv = weights[n["dkv_norm"]].contiguous()
+        elif self.head_gate:
+            self.w_gate = weights[n["g"]].contiguous()          # stored type; the gate's product accumulates in float32
+        if self.has_sink:
+            self.sink = weights[n["sink"]].float().contiguous()
         self.w_uq = self._compute_copy(weights[n["uq"]])
         self.w_uk = self._compute_copy(weights[n["uk"]].view(H, self.dk, self.rank))                       # [H, K = dk, N = rank]
         self.w_uv = self._compute_copy(weights[n["uv"]].view(H, self.dv, self.rank).transpose(1, 2))       # [H, K = rank, N = dv]
         self.w_o = self._compute_copy(weights[n["o"]])
-        self.n_kv = weights[n["dkv_norm"]].contiguous()
         self.n_q = weights[n["dq_norm"]].to(self.n_kv.dtype).contiguous() if self.qr else None
 
     def forward(self, h, ctx, cache):
@@ -90,10 +111,17 @@ class LatentAttention(Part):
             rotary = Rotary(*rotary)
         table = ctx.tables[cache.group]
         h = resolve(h)
-        down = self._down(h)
-        cq = torch.empty((T, self.qr), dtype=act, device=down.device) if self.qr else None
-        ops.latent_prep(down, self.qr, rank, dr, self.n_q, self.n_kv, self.eps, rotary.inv_freq, rotary.rot, ctx.pos, ctx.req_slot,
-                        table, ctx.page_size, cq, cache.k, write_kv=cache.owner, pairing=rotary.pairing)
+        cq = torch.empty((T, self.qr), dtype=act, device=h.device) if self.qr else None
+        gate = None
+        if not self.reads_latent:
+            down = self._down(h)
+            ops.latent_prep(down, self.qr, rank, dr, self.n_q, self.n_kv, self.eps, rotary.inv_freq, rotary.rot, ctx.pos, ctx.req_slot,
+                            table, ctx.page_size, cq, cache.k, write_kv=cache.owner, pairing=rotary.pairing)
+            if self.out_gate or self.head_gate:
+                gate = down[:, self.qr + rank + dr:]
+        elif self.head_gate:
+            gate = torch.empty((T, H), dtype=torch.float32, device=h.device)
+            ops.small_proj(h, self.w_gate, None, gate)
         q = resolve(matmul(cq if self.qr else h, self.w_uq))
         qa = torch.empty((T, H * d), dtype=act, device=q.device)
         self._per_head(q, self.w_uk, qa, dk, rank, dk + dr, d, ctx)
@@ -104,7 +132,9 @@ class LatentAttention(Part):
         ov = torch.empty((T, H * self.dv), dtype=act, device=q.device)
         self._per_head(o, self.w_uv, ov, rank, self.dv, d, self.dv, ctx)
         if self.out_gate:
-            ops.sigmoid_gate(ov, down[:, self.qr + rank + dr:], ov)
+            ops.sigmoid_gate(ov, gate, ov)
+        elif gate is not None:
+            ops.head_gate(ov, gate, H, self.dv)
         return matmul(ov, self.w_o)
 
     def _per_head(self, x, w, y, K, N, xs, ys, ctx):
@@ -119,5 +149,5 @@ class LatentAttention(Part):
         ops.mark("library product")
 
     def _down(self, h):
-        """[Wdq; Wdkv; Wg] h as float32 [T, qr + rank + dr (+ H dv)]."""
+        """[Wdq; Wdkv; Wg] h as float32 [T, qr + rank + dr (+ H dv or H)]."""
         return resolve(matmul(resolve(h), self.w_down, out_dtype=torch.float32))

@@ -80,16 +80,17 @@ class GatedMLP(Part):
 
 @register_feed_forward("plain_mlp")
 class PlainMLP(Part):
-    """y = act(h Wu^T) Wd^T, no gate and no biases; act = the square of relu (`relu_squared`), in the epilogue of the tcgen05
-    products (steps of few tokens, long steps), a kernel of its own in between."""
+    """y = act(h Wu^T) Wd^T, no gate and no biases; act = the square of relu (`relu_squared`) or the tanh form of gelu
+    (`gelu_tanh`), in the epilogue of the tcgen05 products (steps of few tokens, long steps), a kernel of its own in between."""
     graph_capturable = True
 
     def __init__(self, rt: Runtime, hidden: int, intermediate: int, activation: str = "relu_squared", names: dict | None = None):
         """`names`: the two tensors' names under the part's prefix (keys up, down)."""
         super().__init__(rt)
-        if activation != "relu_squared":
-            raise ValueError(f"plain_mlp runs 'relu_squared', not {activation!r}")
+        if activation not in ("relu_squared", "gelu_tanh"):
+            raise ValueError(f"plain_mlp runs 'relu_squared' or 'gelu_tanh', not {activation!r}")
         self.hidden, self.intermediate, self.activation = hidden, intermediate, activation
+        self.act = "relu_squared" if activation == "relu_squared" else "plain_gelu_tanh"      # the products' name of it
         self.names = {"up": "up_proj.weight", "down": "down_proj.weight", **(names or {})}
         self.w_up = self.w_down = None
 
@@ -110,9 +111,9 @@ class PlainMLP(Part):
         if h.dtype == torch.bfloat16 and h.is_cuda and h.is_contiguous():
             from .. import ops_gemm
             if use_tc(T, I, H) and ops_gemm.can_act(T, I, H):
-                return ops_gemm.gemm_tc(h, self.w_up, gated="relu_squared")
+                return ops_gemm.gemm_tc(h, self.w_up, gated=self.act)
             if use_pair_product(T, I, H):
-                return ops_gemm.gemm_tc2(h, self.w_up, gated="relu_squared")
+                return ops_gemm.gemm_tc2(h, self.w_up, gated=self.act)
         m = resolve(matmul(h, self.w_up))
-        ops.relu_square(m)
+        (ops.relu_square if self.activation == "relu_squared" else ops.gelu)(m)
         return m

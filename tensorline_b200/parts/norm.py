@@ -105,7 +105,7 @@ class RMSNorm(Part):
             else:
                 return self.add_norm_pair(x, pending, None, rows=rows)[0]
         if isinstance(pending, PostNormed):              # x += value / rms(value) * its weight (+ a row), then this norm
-            if self.cast_first or self.one_plus or pending.eps != self.eps or \
+            if self.cast_first or pending.eps != self.eps or \
                     (pending.weight is not None and pending.weight.dtype != self.weight.dtype):
                 if rows is not None:
                     raise NotImplementedError("a normalised addend before a norm of picked rows needs this norm's float form")
@@ -143,3 +143,24 @@ class RMSNorm(Part):
             pending = pending.sum()
         ops.add_rmsnorm(x, pending, self.weight, h, self.eps, rows=rows)
         return h
+
+
+def read_stream(x, pending, rt: Runtime):
+    """x += pending, and x itself as a sublayer without a norm in front reads it: rounded to the activation type (the 32-bit
+    engine's sublayers read the stream where it lies)."""
+    if isinstance(pending, StreamSum):
+        pending = pending.write_into(x)
+    if isinstance(pending, (StreamUpdate,)):
+        raise TypeError("a sublayer without a norm reads one stream, not several copies")
+    post = pending if isinstance(pending, PostNormed) else None
+    if post is None and pending is not None and not isinstance(pending, StreamSum):
+        x.add_(resolve(pending).float())
+    if rt.exact:
+        if post is not None:
+            post.add_into(x)
+        return x
+    h = torch.empty(x.shape, dtype=rt.act_dtype, device=x.device)
+    value = post.value if post is not None else None
+    ops.post_norm_add_norm(x, value, post.weight if value is not None else None, None, h, post.eps if post is not None else 0.0,
+                           extra=post.extra if post is not None else None)
+    return h
