@@ -640,10 +640,31 @@ def _zosurax_sizes(z):
             "layers": [rec, attention("attention", z["head"] // 2), attention("attention_2", z["head"])]}
 
 
+def _fimolix_sizes(z):
+    """Four layers: differential attention (as many query, key and value columns as the other arm's attention: two maps of half a
+    head over values of a whole one) behind a convolution of four taps, with capped scores; attention through a latent over a window
+    of 1,024 keys, the latent as wide as the widest head the tensor-core attention takes; differential attention again; attention over
+    2,048 keys through the latents of the second layer.  A plain feed-forward with as many active weights a token as the routed one
+    of the other arm."""
+    mlp = {"kind": "dense", "ff": 3 * z["top"] * z["ff"] // 2 // 64 * 64}
+    diff = {"type": "attention", "mlp": mlp, "mixer": {
+        "heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["head"] // 2, "vdim": z["head"], "scale": (z["head"] // 2) ** -0.5,
+        "softcap": 50.0, "diff": 0.5, "conv": 4}}
+
+    def latent(window, **more):
+        return {"type": "latent_attention", "mlp": mlp, "mixer": dict({
+            "heads": z["heads"], "dim": z["head"], "rot_dim": 64, "rot": {"base": 500000.0, "dims": 64}, "vdim": z["head"], "kv_rank": 192,
+            "scale": (z["head"] + 64) ** -0.5, "mask": {"size": window}}, **more)}
+    order = [diff, latent(1024), diff, latent(2048, kv_from=1)]
+    return {"architecture": "Fimolix", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5},
+            "layers": [order[i] if i < 4 else diff for i in range(z["layers"])]}
+
+
 def run_design(a):
     import torch
     from tensorline_b200 import Engine, Qwen2Config
     from tensorline_b200.config.dekerax import DekeraxConfig
+    from tensorline_b200.config.fimolix import FimolixConfig
     from tensorline_b200.config.sumuvik import SumuvikConfig
     from tensorline_b200.config.tenalorn import TenalornConfig
     from tensorline_b200.config.vutesun import VutesunConfig
@@ -670,6 +691,8 @@ def run_design(a):
             arms = {"tenalorn": TenalornConfig.from_dict(_tenalorn_sizes(z)), "vutesun": arms["vutesun"]}
         if a.design == "zosurax":                                        # its closest: a matrix memory in the scan kernel, rotated attention
             arms = {"zosurax": ZosuraxConfig.from_dict(_zosurax_sizes(z)), "vutesun": arms["vutesun"]}
+        if a.design == "fimolix":                                        # its closest: attention through a latent over a window, norms of sub-blocks' outputs
+            arms = {"fimolix": FimolixConfig.from_dict(_fimolix_sizes(z)), "dekerax": DekeraxConfig.from_dict(_dekerax_sizes(z))}
         out[tag] = {"sizes": dict(z, dense_intermediate=dense)}
         for name, cfg in arms.items():
             weights = random_weights(cfg, device)
@@ -693,7 +716,8 @@ def run_design(a):
             import gc
             gc.collect(); torch.cuda.empty_cache()
     first = out[sorted(out)[0]]
-    beside = {"vutesun": "Qwen2", "dekerax": "Vutesun", "sumuvik": "Dekerax", "tenalorn": "Vutesun", "zosurax": "Vutesun"}[a.design]
+    beside = {"vutesun": "Qwen2", "dekerax": "Vutesun", "sumuvik": "Dekerax", "tenalorn": "Vutesun", "zosurax": "Vutesun",
+              "fimolix": "Dekerax"}[a.design]
     print(json.dumps({"metric": f"decode tok/s of the {a.design.capitalize()} decoder beside {beside} at equal layer sizes (bf16, batch {batch}, context {context})",
                       "value": first[a.design][f"decode_b{batch}_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": K, "warmup": W,
                       "ms_per_step": first[a.design][f"decode_b{batch}_ms"], "higher_is_better": True, "scaling": "weak",
@@ -732,9 +756,9 @@ def main(argv=None):
     ap.add_argument("--timeline", action="store_true",
                     help="print the time line of one captured decode step from the kernels' own stamps (needs TENSORLINE_B200_TRACE=1)")
     ap.add_argument("--no-warm-mix", dest="warm_mix", action="store_false", help="mix: time the first pass (graph capture included)")
-    ap.add_argument("--design", choices=["vutesun", "dekerax", "sumuvik", "tenalorn", "zosurax"], default=None,
+    ap.add_argument("--design", choices=["vutesun", "dekerax", "sumuvik", "tenalorn", "zosurax", "fimolix"], default=None,
                     help="instead of the default workload: this design beside the closest other one at equal layer sizes "
-                         "(vutesun beside Qwen2, dekerax beside vutesun, sumuvik beside dekerax, tenalorn beside vutesun, zosurax beside vutesun; "
+                         "(vutesun beside Qwen2, dekerax beside vutesun, sumuvik beside dekerax, tenalorn beside vutesun, zosurax beside vutesun, fimolix beside dekerax; "
                          "prefill, decode, --profile)")
     ap.add_argument("--design-size", default="", help="--design: which of the sizes (2k, 4k; commas between them; default all)")
     a = ap.parse_args(argv)

@@ -35,20 +35,20 @@ class DifferentialAttention(Part):
     graph_capturable = True
 
     def __init__(self, rt: Runtime, hidden: int, num_heads: int, num_kv_heads: int, head_dim: int, v_head_dim: int, scale: float,
-                 init: float, norm_eps: float, taps: int = 1, qk_norm: bool = True, score_cap: float | None = None,
+                 init: float, norm_eps: float, taps: int | None = None, qk_norm: bool = True, score_cap: float | None = None,
                  window: int | None = None, names: dict | None = None):
-        """`taps` 1: no convolution.  `init`: the constant part of lambda, also 1 - the outputs' factor.  `norm_eps`: of the q/k
+        """`taps` None: no convolution (one tap is a factor a channel, without state).  `init`: the constant part of lambda, also 1 - the outputs' factor.  `norm_eps`: of the q/k
         norms and of the outputs' norm."""
         super().__init__(rt)
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} query heads are not a multiple of {num_kv_heads} KV heads")
-        if taps < 1:
+        if taps is not None and taps < 1:
             raise ValueError(f"a convolution of {taps} taps")
         d = max(MAPS * head_dim, v_head_dim)
         if not rt.exact:
             d = -(-d // 16) * 16                          # the bfloat16 attention kernels take multiples of 16
         self.hidden, self.H, self.G, self.dk, self.dv, self.d = hidden, num_heads, num_kv_heads, head_dim, v_head_dim, d
-        self.taps, self.init, self.eps, self.qk_norm = taps, float(init), float(norm_eps), bool(qk_norm)
+        self.has_conv, self.taps, self.init, self.eps, self.qk_norm = taps is not None, taps or 1, float(init), float(norm_eps), bool(qk_norm)
         self.C = (num_heads + num_kv_heads) * MAPS * head_dim + num_kv_heads * v_head_dim
         self.names = {**_NAMES, **(names or {})}
         # what `attention_kernels.attend` reads of a mixer
@@ -69,7 +69,7 @@ class DifferentialAttention(Part):
         n = {k: f"{prefix}.{v}" for k, v in self.names.items()}
         out = {n[k]: TensorSpec((rows, self.hidden)) for k, rows in self._heads()}
         out[n["o"]] = TensorSpec((self.hidden, self.H * self.dv))
-        if self.taps > 1:
+        if self.has_conv:
             out.update({n[k + "_conv"]: TensorSpec((rows, self.taps)) for k, rows in self._heads()})
         if self.qk_norm:
             out.update({n["q_norm"]: TensorSpec((self.dk,), init="ones"), n["k_norm"]: TensorSpec((self.dk,), init="ones")})
@@ -80,7 +80,7 @@ class DifferentialAttention(Part):
         n = {k: f"{prefix}.{v}" for k, v in self.names.items()}
         self.w_qkv = self._compute_copy(torch.cat([weights[n[k]] for k, _ in self._heads()], dim=0))
         self.w_o = self._compute_copy(weights[n["o"]])
-        if self.taps > 1:
+        if self.has_conv:
             self.taps_w = torch.cat([weights[n[k + "_conv"]] for k, _ in self._heads()], dim=0).contiguous()
         else:
             self.taps_w = torch.ones((self.C, 1), dtype=torch.bfloat16, device=self.w_o.device)
