@@ -81,19 +81,27 @@ __device__ __forceinline__ float tl_sink_term(const float* __restrict__ sink, in
 // (scores up to half the cap, the usual case) tanh(z) is z times a polynomial of degree 3 in z^2 (a least-maximum fit of
 // tanh(z) / z on [0, 1/2], relative error 6e-7), five multiply-adds a score; else 1 - 2 / (1 + e^(2 z)) with the
 // special-function unit's exponential and reciprocal (absolute error about 2e-7).  Called by whole warps.
-template <int N>
+template <int N>                                          // N even
 __device__ __forceinline__ void tl_cap_scores(float (&s)[N], float in, float out) {
     float big = 0.f;
 #pragma unroll
     for (int i = 0; i < N; ++i) big = fmaxf(big, fabsf(s[i]));
     if (!__any_sync(0xffffffffu, !(big * in <= 0.5f))) {
+        // two scores an instruction: the pairs of float multiply-adds of this architecture
         const float i2 = in * in, c0 = 0.99999945577f * (out * in), c1 = -0.33326317939f * (out * in) * i2,
                     c2 = 0.13190296634f * (out * in) * i2 * i2, c3 = -0.04440222694f * (out * in) * i2 * i2 * i2;
 #pragma unroll
-        for (int i = 0; i < N; ++i) {
-            const float u = s[i] * s[i];
-            s[i] *= fmaf(fmaf(fmaf(c3, u, c2), u, c1), u, c0);
-        }
+        for (int i = 0; i < N; i += 2)
+            asm("{\n\t.reg .b64 x, u, r, k0, k1, k2, k3;\n\t"
+                "mov.b64 x, {%0, %1};\n\t"
+                "mov.b64 k0, {%2, %2};\n\tmov.b64 k1, {%3, %3};\n\tmov.b64 k2, {%4, %4};\n\tmov.b64 k3, {%5, %5};\n\t"
+                "mul.rn.f32x2 u, x, x;\n\t"
+                "fma.rn.f32x2 r, k3, u, k2;\n\t"
+                "fma.rn.f32x2 r, r, u, k1;\n\t"
+                "fma.rn.f32x2 r, r, u, k0;\n\t"
+                "mul.rn.f32x2 x, x, r;\n\t"
+                "mov.b64 {%0, %1}, x;\n\t}"
+                : "+f"(s[i]), "+f"(s[i + 1]) : "f"(c0), "f"(c1), "f"(c2), "f"(c3));
     } else {
 #pragma unroll
         for (int i = 0; i < N; ++i) {
@@ -220,9 +228,26 @@ __device__ __forceinline__ float tl_relu_squared_rounded(float v) {
     return r * r;
 }
 
-// The epilogue activation of a product without a gate: `act` 1: the square of relu, 2: the tanh form of gelu (of the
-// accumulator itself).
-__device__ __forceinline__ float tl_plain_act(float v, int act) { return act == 2 ? tl_gelu_tanh(v) : tl_relu_squared_rounded(v); }
+// The tanh form of gelu in the bfloat16 engine: (1 + tanh(u)) / 2 = 1 / (1 + e^(-2 u)) with the special-function unit's
+// exponential and reciprocal, nine instructions (an epilogue with tanhf took longer than its product's tiles).
+__device__ __forceinline__ float tl_gelu_tanh_bf16(float z) {
+    float e;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(-2.302208198f * z * fmaf(0.044715f * z, z, 1.0f)));      // 2 sqrt(2 / pi) log2(e)
+    return __fdividef(z, 1.0f + e);
+}
+
+// The epilogue activation of a product without a gate, `act` 0: none, 1: the square of relu, 2: the tanh form of gelu (of the
+// accumulator itself).  The choice stands outside the loops: the elements' chains overlap.
+template <int N>
+__device__ __forceinline__ void tl_plain_act(float (&v)[N], int act) {
+    if (act == 2) {
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] = tl_gelu_tanh_bf16(v[i]);
+    } else if (act == 1) {
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] = tl_relu_squared_rounded(v[i]);
+    }
+}
 
 // The clamped swish works on the pair: g' = min(g, limit), u' = clamp(u, -limit, limit); g' sigmoid(alpha g') (u' + 1).
 #define TL_ACT_SWISH_CLAMPED 3

@@ -91,10 +91,11 @@ __global__ void __launch_bounds__(128) conv_heads_kernel(const ConvHeads A, int 
     }
 }
 
-// bfloat16, dim 8 .. 256 a power of two, dv and d multiples of 8, weights in bfloat16.  A thread owns eight channels and walks TT
-// tokens of a request: every row of the tile and the TAPS - 1 rows in front of it are loaded at once (16 bytes each), a map's
-// sum of squares is finished by shuffles over the dim / 8 lanes that share it.  The thread of a request's first tile holds the
-// slot's rows in registers before it overwrites them.  The sums are those of the kernel above, in its order but for the squares.
+// bfloat16, dim 8 .. 256 a power of two, dv and d multiples of 8, weights in bfloat16.  A thread owns eight channels and walks
+// `tiles` tiles of TT tokens of a request: the TAPS - 1 rows in front of a tile are carried along, the next tile's rows (16 bytes
+// each) are on their way while a tile is worked through, a map's sum of squares is finished by shuffles over the dim / 8 lanes
+// that share it.  The thread of a request's first tile holds the slot's rows in registers before it overwrites them.  The sums
+// are those of the kernel above, in its order but for the squares.
 __device__ __forceinline__ void conv_unpack(const uint4 x, float (&v)[8]) {
     const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&x);
 #pragma unroll
@@ -102,7 +103,8 @@ __device__ __forceinline__ void conv_unpack(const uint4 x, float (&v)[8]) {
 }
 
 template <int TAPS, int TT>
-__global__ void __launch_bounds__(128) conv_heads_vec_kernel(const ConvHeads A) {
+__global__ void __launch_bounds__(128) conv_heads_vec_kernel(const ConvHeads A, int tiles) {
+    __shared__ size_t place[TT == 1 ? 1 : 128];              // the block's tokens: row of head 0 in the pages
     const int b = blockIdx.x, nqm = A.nq * A.maps, nkm = A.nkv * A.maps;
     const int n8 = A.C >> 3, mine = blockIdx.z * blockDim.x + threadIdx.x, c8 = min(mine, n8 - 1), c = c8 * 8;      // whole warps: the lanes exchange
     const int qk8 = (nqm + nkm) * A.dim >> 3;
@@ -130,63 +132,89 @@ __global__ void __launch_bounds__(128) conv_heads_vec_kernel(const ConvHeads A) 
     grid_dependency_wait();
     grid_dependency_trigger();
     const int t0 = A.q_start[b], t1 = A.q_start[b + 1], n = t1 - t0, slot = A.slots[b], p0 = A.start_pos[b];
-    const int first = blockIdx.y * TT, count = min(TT, n - first);                 // the tile's place in the step
+    const int first = blockIdx.y * TT * tiles, count = min(TT * tiles, n - first);             // the block's place in the step
     if (count <= 0) return;
+    for (int i = threadIdx.x; i < count; i += blockDim.x) {
+        const int p = p0 + first + i;
+        const int* tab = A.table + (size_t)tl_checked(slot, A.lim.table_rows, A.lim, TL_K_ROPE) * A.max_pages;
+        const int page = tl_checked(tab[tl_checked(p / A.page_size, A.max_pages, A.lim, TL_K_ROPE)], A.lim.total_pages, A.lim, TL_K_ROPE);
+        place[i] = (size_t)page * A.nkv * A.page_size + p % A.page_size;
+    }
     const bf16* proj = (const bf16*)A.proj + (size_t)t0 * A.stride + c;
     bf16* st = (bf16*)A.state + (size_t)slot * A.slot_stride + c;
-    uint4 rows[TT + TAPS - 1], last[TAPS > 1 ? TAPS - 1 : 1];
+    auto row_at = [&](int src) {                             // a row of the step, or what the request left in front of it
+        if (src < 0) return *reinterpret_cast<const uint4*>(st + (size_t)(TAPS - 1 + src) * A.C);
+        if (src < n) return *reinterpret_cast<const uint4*>(proj + (size_t)src * A.stride);
+        return make_uint4(0, 0, 0, 0);
+    };
+    uint4 next[TT], last[TAPS > 1 ? TAPS - 1 : 1];
+    float back[TAPS > 1 ? TAPS - 1 : 1][8];                  // the TAPS - 1 rows in front of the tile
 #pragma unroll
-    for (int i = 0; i < TT + TAPS - 1; ++i) {
-        const int src = first + i - (TAPS - 1);
-        rows[i] = make_uint4(0, 0, 0, 0);
-        if (src < 0) rows[i] = *reinterpret_cast<const uint4*>(st + (size_t)(TAPS - 1 + src) * A.C);
-        else if (src < n) rows[i] = *reinterpret_cast<const uint4*>(proj + (size_t)src * A.stride);
-    }
+    for (int j = 0; j < TAPS - 1; ++j) conv_unpack(row_at(first + j - (TAPS - 1)), back[j]);
+#pragma unroll
+    for (int i = 0; i < TT; ++i) next[i] = row_at(first + i);
     if (first == 0 && TAPS > 1) {                            // the slot's rows after the step: loaded before any is written
 #pragma unroll
         for (int j = 0; j < TAPS - 1; ++j) {
             const int src = n - (TAPS - 1) + j;
-            last[j] = src >= 0 ? *reinterpret_cast<const uint4*>(proj + (size_t)src * A.stride)
-                               : *reinterpret_cast<const uint4*>(st + (size_t)(TAPS - 1 + src) * A.C);
+            last[j] = row_at(src);
         }
     }
     const int lanes = A.dim >> 3;
+    const int head = is_q ? unit : qk ? (unit - nqm) / A.maps : unit - nqm - nkm;
+    bf16* const pages = (bf16*)(qk ? A.k_pages : A.v_pages) + (size_t)head * A.page_size * A.d;
+    bf16* const queries = (bf16*)A.q_out + ((size_t)(t0 + first) * nqm + unit) * A.d;
+    __syncthreads();
+    for (int at = 0; at < count; at += TT) {
+        float u[TAPS - 1 + TT][8];
 #pragma unroll
-    for (int i = 0; i < TT; ++i) {
-        if (i >= count) break;                               // the same for the whole block
-        float y[8];
+        for (int j = 0; j < TAPS - 1; ++j)
 #pragma unroll
-        for (int k = 0; k < 8; ++k) y[k] = 0.f;
+            for (int k = 0; k < 8; ++k) u[j][k] = back[j][k];
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j) {
-            float u[8];
-            conv_unpack(rows[i + j], u);
+        for (int i = 0; i < TT; ++i) conv_unpack(next[i], u[TAPS - 1 + i]);
+        if (TT > 1) {
 #pragma unroll
-            for (int k = 0; k < 8; ++k) y[k] = fmaf(w[k][j], u[k], y[k]);
+            for (int i = 0; i < TT; ++i) if (at + TT < count) next[i] = row_at(first + at + TT + i);
         }
-        float ss = 0.f;
 #pragma unroll
-        for (int k = 0; k < 8; ++k) ss = fmaf(y[k], y[k], ss);
-        for (int o = 1; o < lanes; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);      // values join in and ignore the sum
-        if (nw) {
-            const float rstd = 1.0f / sqrtf(ss / (float)A.dim + A.eps);
+        for (int i = 0; i < TT; ++i) {
+            if (at + i >= count) break;                      // the same for the whole block
+            float y[8];
 #pragma unroll
-            for (int k = 0; k < 8; ++k) y[k] = y[k] * rstd * g[k];
-        }
-        if (mine >= n8) continue;
-        uint4 out;
-        __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&out);
+            for (int k = 0; k < 8; ++k) y[k] = 0.f;
 #pragma unroll
-        for (int k = 0; k < 4; ++k) o2[k] = __floats2bfloat162_rn(y[2 * k], y[2 * k + 1]);
-        bf16* row = conv_heads_row<bf16>(A, unit, t0 + first + i, p0 + first + i, slot);
-        *reinterpret_cast<uint4*>(row + map * A.dim + e0) = out;
-        const uint4 zero = make_uint4(0, 0, 0, 0);
-        if (is_q) {                                          // a query's other maps
-            for (int m = 0; m < A.maps; ++m) if (m != map) *reinterpret_cast<uint4*>(row + m * A.dim + e0) = zero;
+            for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+                for (int k = 0; k < 8; ++k) y[k] = fmaf(w[k][j], u[i + j][k], y[k]);
+            float ss = 0.f;
+#pragma unroll
+            for (int k = 0; k < 8; ++k) ss = fmaf(y[k], y[k], ss);
+            for (int o = 1; o < lanes; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);      // values join in and ignore the sum
+            if (nw) {
+                const float rstd = 1.0f / sqrtf(ss / (float)A.dim + A.eps);
+#pragma unroll
+                for (int k = 0; k < 8; ++k) y[k] = y[k] * rstd * g[k];
+            }
+            if (mine >= n8) continue;
+            uint4 out;
+            __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&out);
+#pragma unroll
+            for (int k = 0; k < 4; ++k) o2[k] = __floats2bfloat162_rn(y[2 * k], y[2 * k + 1]);
+            bf16* row = is_q ? queries + (size_t)(at + i) * nqm * A.d : pages + place[at + i] * A.d;
+            *reinterpret_cast<uint4*>(row + map * A.dim + e0) = out;
+            const uint4 zero = make_uint4(0, 0, 0, 0);
+            if (is_q) {                                      // a query's other maps
+                for (int m = 0; m < A.maps; ++m) if (m != map) *reinterpret_cast<uint4*>(row + m * A.dim + e0) = zero;
+            }
+            if (is_q || !qk || map == A.maps - 1) {          // behind the last map, behind a value
+                for (int e = (qk ? A.maps * A.dim : A.dv) + e0; e < A.d; e += width) *reinterpret_cast<uint4*>(row + e) = zero;
+            }
         }
-        if (is_q || !qk || map == A.maps - 1) {              // behind the last map, behind a value
-            for (int e = (qk ? A.maps * A.dim : A.dv) + e0; e < A.d; e += width) *reinterpret_cast<uint4*>(row + e) = zero;
-        }
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; ++j)
+#pragma unroll
+            for (int k = 0; k < 8; ++k) back[j][k] = u[TT + j][k];
     }
     if (first == 0 && TAPS > 1 && mine < n8) {
 #pragma unroll
@@ -194,7 +222,7 @@ __global__ void __launch_bounds__(128) conv_heads_vec_kernel(const ConvHeads A) 
     }
 }
 
-constexpr int CONV_HEADS_TT = 8;
+constexpr int CONV_HEADS_TT = 4, CONV_HEADS_TILES = 4;       // tokens a tile, tiles a block in long steps (128 tokens at most)
 
 TL_EXPORT int tl_conv_heads(const void* proj, int act_dtype, int stride, const void* taps_w, int w_dtype, int taps, void* state,
                             long long slot_stride, const int* q_start, const int* slots, const int* start_pos, const int* table,
@@ -211,10 +239,13 @@ TL_EXPORT int tl_conv_heads(const void* proj, int act_dtype, int stride, const v
         (d & 7) == 0 && (stride & 7) == 0 && (slot_stride & 7) == 0 && (bases & 15) == 0) {
         const int n8 = A.C >> 3;
         const bool one = max_q_len == 1;
-        const dim3 grid(B, one ? 1 : (max_q_len + CONV_HEADS_TT - 1) / CONV_HEADS_TT, (n8 + 127) / 128);
+        // a few tiles a block once the blocks of single tiles would fill the GPU more than twice
+        const long long single_tiles = (long long)B * ((max_q_len + CONV_HEADS_TT - 1) / CONV_HEADS_TT) * ((n8 + 127) / 128);
+        const int tiles = one || single_tiles < 8LL * tl_num_sms() ? 1 : CONV_HEADS_TILES;
+        const dim3 grid(B, one ? 1 : (max_q_len + CONV_HEADS_TT * tiles - 1) / (CONV_HEADS_TT * tiles), (n8 + 127) / 128);
         if (grid.y > 65535 || grid.z > 65535) return 1;
-#define CH(TAPS) (one ? launch_after_wait(conv_heads_vec_kernel<TAPS, 1>, grid, dim3(128), 0, stream, A) \
-                      : launch_after_wait(conv_heads_vec_kernel<TAPS, CONV_HEADS_TT>, grid, dim3(128), 0, stream, A))
+#define CH(TAPS) (one ? launch_after_wait(conv_heads_vec_kernel<TAPS, 1>, grid, dim3(128), 0, stream, A, tiles) \
+                      : launch_after_wait(conv_heads_vec_kernel<TAPS, CONV_HEADS_TT>, grid, dim3(128), 0, stream, A, tiles))
         const int e = taps == 1 ? CH(1) : taps == 2 ? CH(2) : taps == 3 ? CH(3) : CH(4);
 #undef CH
         return e ? e : tl_launch_status();

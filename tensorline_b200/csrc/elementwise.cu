@@ -615,27 +615,27 @@ TL_EXPORT int tl_add_rmsnorm_pair(float* x, const void* a, const void* b, const 
 }
 
 // ------------------------------------------------------------------ a sigmoid gate per (token, head) on attention's output
-// o[t, h, :] *= sigmoid(gate[t, h]); gate float, rows of nq numbers `ldg` apart.
-template <typename TA>
-__global__ void head_gate_kernel(TA* __restrict__ o, const float* __restrict__ gate, int ldg, int nq, int d, size_t total) {
+// o[t, h, :] *= sigmoid(gate[t, h]); gate float or of o's type, rows of nq numbers `ldg` apart.
+template <typename TA, typename TG>
+__global__ void head_gate_kernel(TA* __restrict__ o, const TG* __restrict__ gate, int ldg, int nq, int d, size_t total) {
     grid_dependency_wait();
     grid_dependency_trigger();
     for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
         const size_t row = idx / d, tok = row / nq;
-        const float g = 1.0f / (1.0f + expf(-gate[tok * ldg + (row - tok * nq)]));
+        const float g = 1.0f / (1.0f + expf(-to_f<TG>(gate[tok * ldg + (row - tok * nq)])));
         o[idx] = from_f<TA>(to_f<TA>(o[idx]) * g);
     }
 }
 
 // sixteen bytes a thread (eight bfloat16 or four floats of one head: d is a multiple of that many, o is 16-byte aligned)
-template <typename TA>
-__global__ void head_gate_vec_kernel(TA* __restrict__ o, const float* __restrict__ gate, int ldg, int nq, int vecs_per_head, size_t vecs) {
+template <typename TA, typename TG>
+__global__ void head_gate_vec_kernel(TA* __restrict__ o, const TG* __restrict__ gate, int ldg, int nq, int vecs_per_head, size_t vecs) {
     constexpr int N = 16 / sizeof(TA);
     grid_dependency_wait();
     grid_dependency_trigger();
     for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < vecs; idx += (size_t)gridDim.x * blockDim.x) {
         const size_t row = idx / vecs_per_head, tok = row / nq;
-        const float g = 1.0f / (1.0f + expf(-gate[tok * ldg + (row - tok * nq)]));
+        const float g = 1.0f / (1.0f + expf(-to_f<TG>(gate[tok * ldg + (row - tok * nq)])));
         uint4 raw = reinterpret_cast<const uint4*>(o)[idx];
         TA* e = reinterpret_cast<TA*>(&raw);
 #pragma unroll
@@ -644,20 +644,23 @@ __global__ void head_gate_vec_kernel(TA* __restrict__ o, const float* __restrict
     }
 }
 
-TL_EXPORT int tl_head_gate(void* o, int act_dtype, const float* gate, int ldg, int T, int nq, int d, cudaStream_t stream) {
+TL_EXPORT int tl_head_gate(void* o, int act_dtype, const void* gate, int gate_dtype, int ldg, int T, int nq, int d, cudaStream_t stream) {
     const size_t total = (size_t)T * nq * d;
     if (total == 0) return 0;
+    if (act_dtype == TL_F32 && gate_dtype != TL_F32) return 1;
     const size_t cap = (size_t)tl_num_sms() * 16;
     const int per = act_dtype == TL_F32 ? 4 : 8;
     if (d % per == 0 && (reinterpret_cast<uintptr_t>(o) & 15) == 0) {
         const size_t vecs = total / per;
         const unsigned vb = (unsigned)((vecs + 255) / 256 < cap ? (vecs + 255) / 256 : cap);
-        if (act_dtype == TL_F32) launch_after_wait(head_gate_vec_kernel<float>, dim3(vb), dim3(256), 0, stream, (float*)o, gate, ldg, nq, d / per, vecs);
-        else launch_after_wait(head_gate_vec_kernel<bf16>, dim3(vb), dim3(256), 0, stream, (bf16*)o, gate, ldg, nq, d / per, vecs);
+        if (act_dtype == TL_F32) launch_after_wait(head_gate_vec_kernel<float, float>, dim3(vb), dim3(256), 0, stream, (float*)o, (const float*)gate, ldg, nq, d / per, vecs);
+        else if (gate_dtype == TL_F32) launch_after_wait(head_gate_vec_kernel<bf16, float>, dim3(vb), dim3(256), 0, stream, (bf16*)o, (const float*)gate, ldg, nq, d / per, vecs);
+        else launch_after_wait(head_gate_vec_kernel<bf16, bf16>, dim3(vb), dim3(256), 0, stream, (bf16*)o, (const bf16*)gate, ldg, nq, d / per, vecs);
         return tl_launch_status();
     }
     const unsigned blocks = (unsigned)((total + 255) / 256 < cap ? (total + 255) / 256 : cap);
-    if (act_dtype == TL_F32) launch_after_wait(head_gate_kernel<float>, dim3(blocks), dim3(256), 0, stream, (float*)o, gate, ldg, nq, d, total);
-    else launch_after_wait(head_gate_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, (bf16*)o, gate, ldg, nq, d, total);
+    if (act_dtype == TL_F32) launch_after_wait(head_gate_kernel<float, float>, dim3(blocks), dim3(256), 0, stream, (float*)o, (const float*)gate, ldg, nq, d, total);
+    else if (gate_dtype == TL_F32) launch_after_wait(head_gate_kernel<bf16, float>, dim3(blocks), dim3(256), 0, stream, (bf16*)o, (const float*)gate, ldg, nq, d, total);
+    else launch_after_wait(head_gate_kernel<bf16, bf16>, dim3(blocks), dim3(256), 0, stream, (bf16*)o, (const bf16*)gate, ldg, nq, d, total);
     return tl_launch_status();
 }

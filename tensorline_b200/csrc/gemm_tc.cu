@@ -430,12 +430,16 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                         if (b < G.RB) part[G.swap ? (size_t)b * G.RA + a : (size_t)a * G.RB + b] = __uint_as_float(r[j]);
                     }
                 } else if (G.swap) {
+                    float v[16];
+#pragma unroll
+                    for (int j = 0; j < 16; ++j) v[j] = __uint_as_float(r[j]);
+                    if (G.act) tl_plain_act(v, G.act);
 #pragma unroll
                     for (int j = 0; j < 16; ++j) {
                         const int b = b0 + c0 + j;
                         if (b < G.RB) {
-                            if (G.out_f32) ((float*)G.out)[(size_t)b * G.ldo + a] = __uint_as_float(r[j]);
-                            else ((bf16*)G.out)[(size_t)b * G.ldo + a] = __float2bfloat16_rn(G.act ? tl_plain_act(__uint_as_float(r[j]), G.act) : __uint_as_float(r[j]));
+                            if (G.out_f32) ((float*)G.out)[(size_t)b * G.ldo + a] = v[j];
+                            else ((bf16*)G.out)[(size_t)b * G.ldo + a] = __float2bfloat16_rn(v[j]);
                         }
                     }
                 } else {
@@ -536,8 +540,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                     continue;
                 }
                 if (G.act) {
-                    acc.x = tl_plain_act(acc.x, G.act); acc.y = tl_plain_act(acc.y, G.act);
-                    acc.z = tl_plain_act(acc.z, G.act); acc.w = tl_plain_act(acc.w, G.act);
+                    float v[4] = {acc.x, acc.y, acc.z, acc.w};
+                    tl_plain_act(v, G.act);
+                    acc = make_float4(v[0], v[1], v[2], v[3]);
                 }
                 const size_t o = (size_t)(b0 + tok) * G.ldo + a;
                 if (wide && a + 3 < G.RA) {

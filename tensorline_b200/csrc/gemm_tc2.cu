@@ -282,7 +282,8 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant
                             } else {
                                 float v[16];
 #pragma unroll
-                                for (int j = 0; j < 16; ++j) v[j] = G.act ? tl_plain_act(__uint_as_float(r[j]), G.act) : __uint_as_float(r[j]);
+                                for (int j = 0; j < 16; ++j) v[j] = __uint_as_float(r[j]);
+                                if (G.act) tl_plain_act(v, G.act);
                                 store16_bf16((bf16*)G.out + (size_t)t * G.ldo + col, v, G.N - col);
                             }
                         }

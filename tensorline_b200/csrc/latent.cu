@@ -74,15 +74,15 @@ TL_EXPORT int tl_latent_prep(const float* down, int ld, int qr, int rank, int dr
     return tl_launch_status();
 }
 
-// q: [T, H, dk + dr] (plain part, then the part to rotate); qa: [T, H, d]: columns [rank, rank + dr) get the rotated part,
-// columns from rank + dr on zeros.
+// q: rows `ldq` apart of [H, dk + dr] (plain part, then the part to rotate); qa: [T, H, d]: columns [rank, rank + dr) get the
+// rotated part, columns from rank + dr on zeros.
 template <typename TA>
-__global__ void latent_qrot_kernel(const TA* __restrict__ q, int dk, int dr, const float* __restrict__ inv_freq, int rot,
+__global__ void latent_qrot_kernel(const TA* __restrict__ q, int ldq, int dk, int dr, const float* __restrict__ inv_freq, int rot,
                                    const int* __restrict__ pos, TA* __restrict__ qa, int rank, int d, int H, int interleaved) {
     const int t = blockIdx.x, h = blockIdx.y;
     grid_dependency_wait();
     grid_dependency_trigger();
-    const TA* src = q + ((size_t)t * H + h) * (dk + dr) + dk;
+    const TA* src = q + (size_t)t * ldq + (size_t)h * (dk + dr) + dk;
     TA* dst = qa + ((size_t)t * H + h) * d + rank;
     const int p = pos[t], rhalf = rot >> 1;
     for (int i = threadIdx.x; i < rhalf; i += blockDim.x) {
@@ -95,12 +95,70 @@ __global__ void latent_qrot_kernel(const TA* __restrict__ q, int dk, int dr, con
     for (int i = dr + threadIdx.x; i < d - rank; i += blockDim.x) dst[i] = from_f<TA>(0.f);
 }
 
-TL_EXPORT int tl_latent_qrot(const void* q, int dk, int dr, const float* inv_freq, int rot, const int* pos, void* qa, int rank, int d,
+// bfloat16, every size a multiple of eight: a block a token, its angles once for all heads, eight values a thread and step.
+template <bool INTERLEAVED>
+__global__ void latent_qrot_vec_kernel(const bf16* __restrict__ q, int ldq, int dk, int dr, const float* __restrict__ inv_freq, int rot,
+                                       const int* __restrict__ pos, bf16* __restrict__ qa, int rank, int d, int H) {
+    extern __shared__ float cs[];                        // cos [rot / 2], sin [rot / 2]
+    const int t = blockIdx.x, p = pos[t], rhalf = rot >> 1, per_head = (d - rank) >> 3;
+    for (int i = threadIdx.x; i < rhalf; i += blockDim.x) {
+        float sn, c;
+        sincosf(__fmul_rn((float)p, inv_freq[i]), &sn, &c);
+        cs[i] = c; cs[rhalf + i] = sn;
+    }
+    grid_dependency_wait();
+    grid_dependency_trigger();
+    __syncthreads();
+    for (int item = threadIdx.x; item < H * per_head; item += blockDim.x) {
+        const int h = item / per_head, e0 = (item - h * per_head) * 8;
+        uint4 out = make_uint4(0, 0, 0, 0);
+        if (e0 < dr) {
+            const bf16* src = q + (size_t)t * ldq + (size_t)h * (dk + dr) + dk;
+            out = *reinterpret_cast<const uint4*>(src + e0);
+            if (e0 < rot) {
+                __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&out);
+                if (INTERLEAVED) {
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) {
+                        const float a = __low2float(o2[k]), b = __high2float(o2[k]), c = cs[(e0 >> 1) + k], sn = cs[rhalf + (e0 >> 1) + k];
+                        o2[k] = __floats2bfloat162_rn(__fmul_rn(a, c) - __fmul_rn(b, sn), __fmul_rn(b, c) + __fmul_rn(a, sn));
+                    }
+                } else {
+                    const bool low = e0 < rhalf;
+                    const int i0 = low ? e0 : e0 - rhalf;
+                    const uint4 other = *reinterpret_cast<const uint4*>(src + (low ? e0 + rhalf : i0));
+                    const __nv_bfloat162* p2 = reinterpret_cast<const __nv_bfloat162*>(&other);
+                    float v[8];
+#pragma unroll
+                    for (int k = 0; k < 8; ++k) {
+                        const float mine = k & 1 ? __high2float(o2[k >> 1]) : __low2float(o2[k >> 1]);
+                        const float far = k & 1 ? __high2float(p2[k >> 1]) : __low2float(p2[k >> 1]);
+                        const float c = cs[i0 + k], sn = cs[rhalf + i0 + k];
+                        v[k] = low ? __fmul_rn(mine, c) - __fmul_rn(far, sn) : __fmul_rn(mine, c) + __fmul_rn(far, sn);
+                    }
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) o2[k] = __floats2bfloat162_rn(v[2 * k], v[2 * k + 1]);
+                }
+            }
+        }
+        *reinterpret_cast<uint4*>(qa + ((size_t)t * H + h) * d + rank + e0) = out;
+    }
+}
+
+TL_EXPORT int tl_latent_qrot(const void* q, int ldq, int dk, int dr, const float* inv_freq, int rot, const int* pos, void* qa, int rank, int d,
                              int H, int T, int act_dtype, int interleaved, cudaStream_t stream) {
     if (T <= 0 || H <= 0) return 0;
-    if ((rot & 1) || rot > dr || rank + dr > d || H > 65535) return 1;
-    if (act_dtype == TL_F32) launch_after_wait(latent_qrot_kernel<float>, dim3(T, H), dim3(64), 0, stream, (const float*)q, dk, dr, inv_freq, rot, pos, (float*)qa, rank, d, H, interleaved);
-    else launch_after_wait(latent_qrot_kernel<bf16>, dim3(T, H), dim3(64), 0, stream, (const bf16*)q, dk, dr, inv_freq, rot, pos, (bf16*)qa, rank, d, H, interleaved);
+    if ((rot & 1) || rot > dr || rank + dr > d || H > 65535 || ldq < H * (dk + dr)) return 1;
+    if (act_dtype == TL_BF16 && ((ldq | dk | dr | rank | d) & 7) == 0 && (rot & (interleaved ? 7 : 15)) == 0 && ((((uintptr_t)q | (uintptr_t)qa) & 15) == 0)) {
+        const int items = H * ((d - rank) >> 3), threads = items < 256 ? (items + 31) / 32 * 32 : 256;
+        if (items == 0) return 0;
+        const size_t smem = (size_t)rot * sizeof(float);
+#define QV(I) launch_after_wait(latent_qrot_vec_kernel<I>, dim3(T), dim3(threads), smem, stream, (const bf16*)q, ldq, dk, dr, inv_freq, rot, pos, (bf16*)qa, rank, d, H)
+        return interleaved ? QV(true) : QV(false);
+#undef QV
+    }
+    if (act_dtype == TL_F32) launch_after_wait(latent_qrot_kernel<float>, dim3(T, H), dim3(64), 0, stream, (const float*)q, ldq, dk, dr, inv_freq, rot, pos, (float*)qa, rank, d, H, interleaved);
+    else launch_after_wait(latent_qrot_kernel<bf16>, dim3(T, H), dim3(64), 0, stream, (const bf16*)q, ldq, dk, dr, inv_freq, rot, pos, (bf16*)qa, rank, d, H, interleaved);
     return tl_launch_status();
 }
 
@@ -162,6 +220,81 @@ __global__ void __launch_bounds__(128) head_matmul_kernel(const TA* __restrict__
             }
         }
     }
+}
+
+// The same in the bfloat16 engine, bfloat16 weights: a block is 32 columns x HB_S slices of k, a lane a column; a slice is short
+// enough that its weights are all in flight at once, the first of them before the wait for the kernel in front (nobody writes
+// them).  NT: tokens a block, at most HM_T.  `gate` (float or bfloat16, rows `ldg` apart, may be null): y[t, h, :] is multiplied
+// by sigmoid(gate[t, h]) before it is rounded.  Slices are added in order: as above, one fixed chain a result.
+constexpr int HB_S = 8, HB_AHEAD = 8;
+template <int NT, typename TG>
+__global__ void __launch_bounds__(32 * HB_S) head_matmul_bf16_kernel(const bf16* __restrict__ x, int ldx, int hx, const bf16* __restrict__ w,
+                                                                     bf16* __restrict__ y, int ldy, int hy, int T, int K, int N,
+                                                                     const TG* __restrict__ gate, int ldg) {
+    extern __shared__ float xs[];                        // [NT][K], then the slices' sums [HB_S][NT][32]
+    float* part = xs + NT * K;
+    const int col = threadIdx.x & 31, slice = threadIdx.x >> 5;
+    const int t0 = blockIdx.x * NT, h = blockIdx.y, n = blockIdx.z * 32 + col;
+    const int per = (K + HB_S - 1) / HB_S, k0 = slice * per, k1 = min(K, k0 + per);
+    const bf16* wh = w + (size_t)h * K * N + min(n, N - 1);
+    bf16 ahead[HB_AHEAD];
+#pragma unroll
+    for (int u = 0; u < HB_AHEAD; ++u) ahead[u] = k0 + u < k1 ? wh[(size_t)(k0 + u) * N] : __float2bfloat16_rn(0.f);
+    grid_dependency_wait();
+    grid_dependency_trigger();
+    const int nt = min(NT, T - t0);
+    for (int i = threadIdx.x; i < NT * K; i += blockDim.x) {
+        const int t = i / K, k = i - t * K;
+        xs[i] = t < nt ? __bfloat162float(x[(size_t)(t0 + t) * ldx + (size_t)h * hx + k]) : 0.f;
+    }
+    __syncthreads();
+    float acc[NT];
+#pragma unroll
+    for (int t = 0; t < NT; ++t) acc[t] = 0.f;
+    for (int k = k0; k < k1; k += HB_AHEAD) {
+        bf16 now[HB_AHEAD];
+#pragma unroll
+        for (int u = 0; u < HB_AHEAD; ++u) {
+            now[u] = ahead[u];
+            ahead[u] = k + HB_AHEAD + u < k1 ? wh[(size_t)(k + HB_AHEAD + u) * N] : __float2bfloat16_rn(0.f);
+        }
+#pragma unroll
+        for (int u = 0; u < HB_AHEAD; ++u) {
+            if (k + u < k1) {                            // the same for the whole warp
+                const float wv = __bfloat162float(now[u]);
+#pragma unroll
+                for (int t = 0; t < NT; ++t) acc[t] = fmaf(xs[t * K + k + u], wv, acc[t]);
+            }
+        }
+    }
+#pragma unroll
+    for (int t = 0; t < NT; ++t) part[(slice * NT + t) * 32 + col] = acc[t];
+    __syncthreads();
+    for (int i = threadIdx.x; i < NT * 32; i += blockDim.x) {
+        const int t = i >> 5, c = i & 31, nn = blockIdx.z * 32 + c;
+        if (t >= nt || nn >= N) continue;
+        float v = 0.f;
+#pragma unroll
+        for (int s = 0; s < HB_S; ++s) v += part[(s * NT + t) * 32 + c];
+        if (gate) v *= 1.0f / (1.0f + expf(-to_f<TG>(gate[(size_t)(t0 + t) * ldg + h])));
+        y[(size_t)(t0 + t) * ldy + (size_t)h * hy + nn] = __float2bfloat16_rn(v);
+    }
+}
+
+TL_EXPORT int tl_head_matmul_bf16(const void* x, int ldx, int hx, const void* w, void* y, int ldy, int hy, int T, int H, int K, int N,
+                                  const void* gate, int gate_dtype, int ldg, cudaStream_t stream) {
+    if (T <= 0 || H <= 0 || N <= 0) return 0;
+    const int nt = T >= 8 ? 8 : T >= 4 ? 4 : T >= 2 ? 2 : 1;
+    const size_t smem = ((size_t)nt * K + (size_t)HB_S * nt * 32) * sizeof(float);
+    if (smem > 48 * 1024 || H > 65535 || (N + 31) / 32 > 65535) return 1;
+    const dim3 grid((T + nt - 1) / nt, H, (N + 31) / 32);
+#define HB(NT, TG) launch_after_wait(head_matmul_bf16_kernel<NT, TG>, grid, dim3(32 * HB_S), smem, stream, (const bf16*)x, ldx, hx, (const bf16*)w, \
+        (bf16*)y, ldy, hy, T, K, N, (const TG*)gate, ldg)
+#define HBG(NT) (gate && gate_dtype == TL_BF16 ? HB(NT, bf16) : HB(NT, float))
+    const int e = nt == 8 ? HBG(8) : nt == 4 ? HBG(4) : nt == 2 ? HBG(2) : HBG(1);
+#undef HBG
+#undef HB
+    return e ? e : tl_launch_status();
 }
 
 TL_EXPORT int tl_head_matmul(const void* x, int ldx, int hx, const void* w, int w_dtype, void* y, int ldy, int hy, int T, int H, int K,

@@ -499,7 +499,7 @@ __global__ void gelu_vec8_kernel(uint4* __restrict__ u, size_t n8) {
         uint4 v = u[i];
         __nv_bfloat162* p = reinterpret_cast<__nv_bfloat162*>(&v);
 #pragma unroll
-        for (int e = 0; e < 4; ++e) p[e] = __floats2bfloat162_rn(tl_gelu_tanh(__low2float(p[e])), tl_gelu_tanh(__high2float(p[e])));
+        for (int e = 0; e < 4; ++e) p[e] = __floats2bfloat162_rn(tl_gelu_tanh_bf16(__low2float(p[e])), tl_gelu_tanh_bf16(__high2float(p[e])));
         u[i] = v;
     }
 }

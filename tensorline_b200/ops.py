@@ -25,7 +25,7 @@ _SIGNATURES = {
     "tl_add_rmsnorm": [_P, _P, _P, _I, _P, _I, _P, _I, _I, _F, _I, _P, _I, ctypes.c_longlong, _F, _I, _P],
     "tl_silu_mul": [_P, _P, _I, _I, _I, _I, _I, _F, _F, _P],
     "tl_add_rmsnorm_pair": [_P, _P, _P, _P, _P, _I, _P, _P, _I, _P, _I, _I, _F, _P],
-    "tl_head_gate": [_P, _I, _P, _I, _I, _I, _I, _P],
+    "tl_head_gate": [_P, _I, _P, _I, _I, _I, _I, _I, _P],
     "tl_post_norm_add_norm": [_P, _P, _P, _P, _P, _I, _P, _I, _P, _I, _I, _F, _I, _P],
     "tl_rope_kv_write": [_P, _I, _P, _I, _P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _P, _P, _I, _I, _P, _I, ctypes.c_longlong,
                          _I, _P, _P, _F, _I, _I, _I, _I, _P, _P],
@@ -60,7 +60,7 @@ _SIGNATURES = {
     "tl_delta_state_floats": [_I, _I],
     "tl_delta_columns": [],
     "tl_latent_prep": [_P, _I, _I, _I, _I, _P, _P, _I, _F, _P, _I, _P, _P, _P, _I, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P],
-    "tl_latent_qrot": [_P, _I, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _P],
+    "tl_latent_qrot": [_P, _I, _I, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _P],
     "tl_embed_streams": [_P, _P, _I, _P, _I, _I, _F, _I, _P, _I, _I, _I, _P, _P, _P, _P],
     "tl_remember_last": [_P, _P, _P, _I, _P, _P],
     "tl_stream_step": [_P, _I, _I, _P, _F, _P, _F, _I, _P, _P, _P, _P, _I, _F, _P, _P, _P, _I, _I, _P],
@@ -72,6 +72,7 @@ _SIGNATURES = {
     "tl_conv_heads": [_P, _I, _I, _P, _I, _I, _P, ctypes.c_longlong, _P, _P, _P, _P, _I, _I, _P, _P, _F, _P, _P, _P, _I, _I, _I, _I, _I, _I,
                       _I, _I, _I, _I, _P, _P],
     "tl_map_difference": [_P, _P, _I, _I, _I, _I, _I, _F, _F, _F, _P],
+    "tl_head_matmul_bf16": [_P, _I, _I, _P, _P, _I, _I, _I, _I, _I, _I, _P, _I, _I, _P],
     "tl_head_matmul": [_P, _I, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _P],
 }
 
@@ -505,13 +506,20 @@ def add_rmsnorm_pair(x: torch.Tensor, a: torch.Tensor | None, b: torch.Tensor | 
 
 
 def head_gate(o: torch.Tensor, gate: torch.Tensor, nq: int, d: int) -> None:
-    """o[t, h, :] *= sigmoid(gate[t, h]) in place; o [T, nq * d] of the activation type, gate float32 [T, nq] (a column range
-    of a wider tensor may be passed)."""
+    """o[t, h, :] *= sigmoid(gate[t, h]) in place; o [T, nq * d] of the activation type, gate [T, nq] float32 or of o's type (a
+    column range of a wider tensor may be passed)."""
     T = o.shape[0]
-    if o.shape != (T, nq * d) or gate.shape != (T, nq) or gate.dtype != torch.float32 or gate.stride(1) != 1:
-        raise KernelError("head_gate: o [T, nq d], gate float32 [T, nq]")
+    _head_gates(gate, o, T, nq, "head_gate")
+    if o.shape != (T, nq * d):
+        raise KernelError("head_gate: o [T, nq d]")
     _contig(o, "o")
-    _check(core().tl_head_gate(_ptr(o), dtype_code(o.dtype), _ptr(gate), gate.stride(0), T, nq, d, _stream()), "head_gate")
+    _check(core().tl_head_gate(_ptr(o), dtype_code(o.dtype), _ptr(gate), dtype_code(gate.dtype), gate.stride(0), T, nq, d, _stream()),
+           "head_gate")
+
+
+def _head_gates(gate: torch.Tensor, o: torch.Tensor, T: int, nq: int, who: str) -> None:
+    if gate.shape != (T, nq) or gate.dtype not in (torch.float32, o.dtype) or gate.stride(1) != 1:
+        raise KernelError(f"{who}: the gates must be [T, heads], float32 or of the output's type")
 
 
 def post_norm_add_norm(x: torch.Tensor, a: torch.Tensor | None, w_post: torch.Tensor | None, w_pre: torch.Tensor | None,
@@ -1115,25 +1123,36 @@ def _pairing(pairing: str, who: str) -> bool:
 def latent_qrot(q: torch.Tensor, dk: int, dr: int, inv_freq: torch.Tensor, rot: int, pos: torch.Tensor, qa: torch.Tensor,
                 rank: int, H: int, pairing: str = "half") -> None:
     """qa[t, h, rank : rank + dr] = q[t, h, dk : dk + dr] with its first `rot` dimensions rotated by position; the columns of
-    qa behind them are set to zero.  q [T, H (dk + dr)], qa [T, H d]."""
+    qa behind them are set to zero.  q [T, H (dk + dr) or more], qa [T, H d]."""
     T = q.shape[0]
     d = qa.shape[1] // H
-    if q.shape != (T, H * (dk + dr)) or qa.shape != (T, H * d) or qa.dtype != q.dtype or rank + dr > d:
-        raise KernelError("latent_qrot: q [T, H (dk + dr)], qa [T, H d] of one type, d >= rank + dr")
-    _contig(q, "q"); _contig(qa, "qa"); _ints(pos, "pos")
-    _check(core().tl_latent_qrot(_ptr(q), dk, dr, _ptr(inv_freq), int(rot), _ptr(pos), _ptr(qa), rank, d, H, T, dtype_code(q.dtype),
+    if q.shape[1] < H * (dk + dr) or q.stride(1) != 1 or qa.shape != (T, H * d) or qa.dtype != q.dtype or rank + dr > d:
+        raise KernelError("latent_qrot: q [T, H (dk + dr) or more], qa [T, H d] of one type, d >= rank + dr")
+    _contig(qa, "qa"); _ints(pos, "pos")
+    _check(core().tl_latent_qrot(_ptr(q), q.stride(0), dk, dr, _ptr(inv_freq), int(rot), _ptr(pos), _ptr(qa), rank, d, H, T, dtype_code(q.dtype),
                                  int(_pairing(pairing, "latent_qrot")), _stream()), "latent_qrot")
 
 
 def head_matmul(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, H: int, K: int, N: int, x_head_stride: int,
-                y_head_stride: int) -> None:
-    """y[t, h, :N] = x[t, h, :K] w[h]; w [H, K, N]; head h of row t starts at x[t, h * x_head_stride] (y alike); float sums."""
+                y_head_stride: int, gate: torch.Tensor | None = None) -> None:
+    """y[t, h, :N] = x[t, h, :K] w[h]; w [H, K, N]; head h of row t starts at x[t, h * x_head_stride] (y alike); float sums.
+    `gate` ([T, H], float32 or of y's type; bfloat16 x, w and y only): the result is multiplied by sigmoid(gate[t, h]) before it
+    is rounded."""
     T = x.shape[0]
     if w.shape != (H, K, N) or x.dtype != y.dtype or y.shape[0] != T or x.stride(1) != 1 or y.stride(1) != 1:
         raise KernelError("head_matmul: w [H, K, N], x and y of one type with unit inner stride")
     if (H - 1) * x_head_stride + K > x.shape[1] or (H - 1) * y_head_stride + N > y.shape[1]:
         raise KernelError("head_matmul: the heads do not lie inside the rows")
     _contig(w, "w")
+    if gate is not None:
+        _head_gates(gate, y, T, H, "head_matmul")
+    if x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16:
+        _check(core().tl_head_matmul_bf16(_ptr(x), x.stride(0), x_head_stride, _ptr(w), _ptr(y), y.stride(0), y_head_stride, T, H, K, N,
+                                          _ptr(gate), dtype_code(gate.dtype) if gate is not None else 0,
+                                          gate.stride(0) if gate is not None else 0, _stream()), "head_matmul")
+        return
+    if gate is not None:
+        raise KernelError("head_matmul: gates go with bfloat16 tensors")
     _check(core().tl_head_matmul(_ptr(x), x.stride(0), x_head_stride, _ptr(w), dtype_code(w.dtype), _ptr(y), y.stride(0),
                                  y_head_stride, T, H, K, N, dtype_code(x.dtype), _stream()), "head_matmul")
 

@@ -59,7 +59,6 @@ class LatentAttention(Part):
         self.names = {**_NAMES, **(names or {})}
         # what `attention_kernels.attend` reads of a mixer
         self.nq, self.nkv, self.sink = num_heads, 1, None
-        self.w_gate = None
         self.w_down = self.w_uq = self.w_uk = self.w_uv = self.w_o = self.n_q = self.n_kv = None
 
     def cache_need(self):
@@ -92,11 +91,13 @@ class LatentAttention(Part):
                 ([weights[n["g"]]] if self.out_gate or self.head_gate else [])
             self.w_down = self._compute_copy(torch.cat(down, dim=0))
             self.n_kv = weights[n["dkv_norm"]].contiguous()
-        elif self.head_gate:
-            self.w_gate = weights[n["g"]].contiguous()          # stored type; the gate's product accumulates in float32
         if self.has_sink:
             self.sink = weights[n["sink"]].float().contiguous()
-        self.w_uq = self._compute_copy(weights[n["uq"]])
+        uq = weights[n["uq"]]
+        if self.head_gate and self.reads_latent:               # no down product: the gate's rows ride in the queries', padded to whole 16 bytes
+            g = weights[n["g"]].to(uq.dtype)
+            uq = torch.cat([uq, g, torch.zeros((-(uq.shape[0] + g.shape[0]) % 8, g.shape[1]), dtype=uq.dtype, device=uq.device)])
+        self.w_uq = self._compute_copy(uq)
         self.w_uk = self._compute_copy(weights[n["uk"]].view(H, self.dk, self.rank))                       # [H, K = dk, N = rank]
         self.w_uv = self._compute_copy(weights[n["uv"]].view(H, self.dv, self.rank).transpose(1, 2))       # [H, K = rank, N = dv]
         self.w_o = self._compute_copy(weights[n["o"]])
@@ -119,10 +120,9 @@ class LatentAttention(Part):
                             table, ctx.page_size, cq, cache.k, write_kv=cache.owner, pairing=rotary.pairing)
             if self.out_gate or self.head_gate:
                 gate = down[:, self.qr + rank + dr:]
-        elif self.head_gate:
-            gate = torch.empty((T, H), dtype=torch.float32, device=h.device)
-            ops.small_proj(h, self.w_gate, None, gate)
         q = resolve(matmul(cq if self.qr else h, self.w_uq))
+        if self.head_gate and self.reads_latent:
+            gate = q[:, H * (dk + dr):H * (dk + dr) + H]
         qa = torch.empty((T, H * d), dtype=act, device=q.device)
         self._per_head(q, self.w_uk, qa, dk, rank, dk + dr, d, ctx)
         ops.latent_qrot(q, dk, dr, rotary.inv_freq, rotary.rot, ctx.pos, qa, rank, H, pairing=rotary.pairing)
@@ -130,23 +130,28 @@ class LatentAttention(Part):
         from . import attention_kernels
         attention_kernels.attend(self, qa, o, ctx, KVCacheView(cache.k, cache.k, cache.group, cache.owner), table)
         ov = torch.empty((T, H * self.dv), dtype=act, device=q.device)
-        self._per_head(o, self.w_uv, ov, rank, self.dv, d, self.dv, ctx)
+        self._per_head(o, self.w_uv, ov, rank, self.dv, d, self.dv, ctx, gate=gate if self.head_gate else None)
         if self.out_gate:
             ops.sigmoid_gate(ov, gate, ov)
-        elif gate is not None:
-            ops.head_gate(ov, gate, H, self.dv)
         return matmul(ov, self.w_o)
 
-    def _per_head(self, x, w, y, K, N, xs, ys, ctx):
-        """y[t, h, :N] = x[t, h, :K] w[h] with the heads xs (ys) columns apart: the package's kernel, or for long bfloat16 steps
-        one batched library product (as the engine's other long products are the library's)."""
+    def _per_head(self, x, w, y, K, N, xs, ys, ctx, gate=None):
+        """y[t, h, :N] = x[t, h, :K] w[h] (times sigmoid(gate[t, h])) with the heads xs (ys) columns apart: the package's kernel, or
+        for long bfloat16 steps one batched library product that writes where it belongs (as the engine's other long products are
+        the library's)."""
         T, H = x.shape[0], self.H
-        if x.dtype != torch.bfloat16 or T < HEAD_PRODUCT_LIBRARY_MIN_TOKENS or ctx.graph_max_ctx:
-            ops.head_matmul(x, w, y, H, K, N, xs, ys)
+        few = T < HEAD_PRODUCT_LIBRARY_MIN_TOKENS or ctx.graph_max_ctx
+        if x.dtype == torch.bfloat16 and few and w.dtype == torch.bfloat16:
+            ops.head_matmul(x, w, y, H, K, N, xs, ys, gate=gate)
             return
-        out = torch.matmul(x.view(T, H, xs)[:, :, :K].transpose(0, 1), w)          # [H, T, N]
-        y.view(T, H, ys)[:, :, :N].copy_(out.transpose(0, 1))
-        ops.mark("library product")
+        if x.dtype != torch.bfloat16 or few:
+            ops.head_matmul(x, w, y, H, K, N, xs, ys)
+        else:
+            heads = x.as_strided((H, T, K), (xs, x.stride(0), 1))
+            torch.bmm(heads, w, out=y.as_strided((H, T, N), (ys, y.stride(0), 1)))
+            ops.mark("library product")
+        if gate is not None:
+            ops.head_gate(y, gate, H, N)
 
     def _down(self, h):
         """[Wdq; Wdkv; Wg] h as float32 [T, qr + rank + dr (+ H dv or H)]."""
