@@ -8,6 +8,7 @@ build must record the violation (kernel, value, limit), send the access to the s
 pages beyond the stated pool untouched.  Prints one line per case and `ok` at the end.
 """
 import sys
+from types import SimpleNamespace
 
 import torch
 
@@ -53,6 +54,18 @@ def main() -> int:
     expect("position beyond the table's width", "rotary",
            lambda: ops.rope_kv_write(qkv.clone(), None, i32([8, 40, 3]), i32([0, 0, 1]), good, ps, inv_freq, d, nq, nkv, d, k, v))
     assert bool((real_k[POOL + 1:] == 3.0).all())
+    # the convolution of heads and its page write, in both forms (eight channels a thread; 24 channels a map: the plain one)
+    for dim in (32, 24):
+        proj = torch.randn(T, (nq + nkv) * 2 * dim + nkv * 48, device=dev).to(torch.bfloat16)
+        step = SimpleNamespace(q_start=i32([0, 2, 3]), slots=i32([0, 1]), start_pos=i32([8, 3]), B=2, max_q_len=2)
+        taps, state = torch.ones(proj.shape[1], 2, device=dev).to(torch.bfloat16), torch.zeros(3, 1, proj.shape[1], dtype=torch.bfloat16, device=dev)
+        q_out = torch.zeros(T, nq * 2 * d, dtype=torch.bfloat16, device=dev)
+        sizes = dict(nq=nq, nkv=nkv, maps=2, dim=dim, dv=48)
+        ops.conv_heads(proj, taps, state, step, good, ps, q_out, k, v, **sizes)
+        ops.check_device_status()
+        expect(f"page number beyond the pool, convolution of heads of {dim}", "rotary",
+               lambda: ops.conv_heads(proj, taps, state, step, bad_page, ps, q_out, k, v, **sizes))
+        assert bool((real_k[POOL + 1:] == 3.0).all()) and bool((real_v[POOL + 1:] == -3.0).all()), "a page beyond the pool was written"
     # attention kernels reading through the bad entry
     out = torch.zeros(T, nq * d, dtype=torch.bfloat16, device=dev)
     expect("exact-order attention", "exact-order",

@@ -23,7 +23,7 @@ def test_checker_catches_entries_outside_its_bounds_and_redirects_them():
     proc = run(["tests/check_build_cases.py"])
     assert proc.returncode == 0, proc.stdout[-3000:] + proc.stderr[-3000:]
     lines = proc.stdout.splitlines()
-    assert lines[-1] == "ok" and sum(l.startswith("caught:") for l in lines) == 8, proc.stdout
+    assert lines[-1] == "ok" and sum(l.startswith("caught:") for l in lines) == 10, proc.stdout
 
 
 def test_replay_schedules_and_kernel_tests_report_nothing_under_the_checking_build():
