@@ -262,6 +262,10 @@ def plan_splits(batch: int, nkv: int, group: int, span: int, head_dim: int = 128
         # few requests: sixteen ranges in a cluster of sixteen blocks (no parts in memory, no combine kernel, which alone
         # cost 5 us a layer at batch 1)
         splits = min(splits, 16)
+        if base > BIG_CLUSTERS_AT_ONCE and decode_blocks_per_sm(head_dim) == 1:
+            # heads whose block fills an SM: a group of SMs holds two clusters of nine but one larger one, and the eighth waits
+            # for a second round (8 requests, one head of 256, 2,048 keys: 24.9 us with eleven ranges, 14.5 with nine)
+            splits = min(splits, 9)
     elif 8 < splits <= 16:
         # eight ranges merge inside a cluster; measured at batch 8, 8 k to 32 k keys: 27 / 46 / 86 against 30 / 49 / 88 us
         # with nine; at batch 2 and 4, context 4,090, against sixteen ranges and the combine kernel: 2.768 / 2.793 against
@@ -298,6 +302,7 @@ def prefill(q, q_stride, out, k_pages, v_pages, table, page_size, q_start, start
                                        ops.fault_words(q.device), _stream()), "attn_prefill")
 
 
+BIG_CLUSTERS_AT_ONCE = 7            # clusters of 10 to 16 blocks that are placed at once where a block fills an SM (measured)
 CLUSTER16_MAX = int(os.environ.get("TENSORLINE_B200_CLUSTER16_MAX", "12"))   # (request, KV head) pairs up to which 16 ranges merge in a cluster; 0: never
 TMA_DECODE = os.environ.get("TENSORLINE_B200_TMA_DECODE", "1") != "0"   # 0: cp.async loads only (A/B timing)
 TMA_DECODE_MIN_BATCH = int(os.environ.get("TENSORLINE_B200_TMA_DECODE_MIN_BATCH", "1"))   # fewer requests: cp.async loads
