@@ -74,6 +74,14 @@ def test_a_cache_keeps_what_its_readers_see():
     cm.check()
 
 
+def test_ranges_of_keys_for_heads_whose_block_fills_an_sm():
+    """One key/value head of 256: clusters of more than nine blocks only while at most seven of them run."""
+    from tensorline_b200.ops_attention import plan_splits
+    assert plan_splits(7, 1, 16, 2111, 256, sms=148) == (192, 11) and plan_splits(8, 1, 16, 2111, 256, sms=148) == (256, 9)
+    assert plan_splits(12, 1, 16, 2111, 256, sms=148)[1] <= 9
+    assert plan_splits(2, 4, 7, 4096, 128, sms=148)[1] == 16             # narrower heads: two blocks an SM, as they were
+
+
 @pytest.mark.parametrize("path,value,word", [
     (("layers", 1, "type"), "hgrn2", "type"), (("layers", 1, "mixer", "kv_heads"), 4, "kv_heads"), (("layers", 0, "mixer", "rot", "dims"), 3, "dims"),
     (("layers", 0, "mlp", "kind"), "moe", "kind"), (("layers", 0, "mixer", "mask", "size"), 0, "size"), (("layers", 1, "mixer", "softcap"), 0.0, "softcap"),
